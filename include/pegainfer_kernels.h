@@ -211,6 +211,7 @@ int pk_b200_gemm_plan(int M, int N, int K, int swiglu, int sms);
  *   x_mode 3: Qwen3.5 variant of x_mode 1: hidden_out = bf16(hidden + residual) and the norm runs on that ROUNDED sum with
  *             (1 + w) weights (add_batch + rms_norm_batch_offset of pegainfer-qwen35-4b/src/batch_decode.rs:241-253).
  *   epi 4:    like epi 1 with SiLU rounded to bf16 before the multiply (silu_mul_triton_aot_cuda, elementwise.cu:36-41).
+ *   epi 5:    like epi 1 with ReLU in the place of SiLU.
  *   Tensor parallel, GEMV fused with its all-reduce over NVLink peer memory (no collective launch):
  *   epi 2:    the bf16 partial rows are pushed into every rank's staging slot and the grid's last CTA
  *             publishes the sequence flag (release.sys); Y is not written.
@@ -423,7 +424,8 @@ int pk_res32_skinny_proj(const void* W, const float* x, float* out, int M, int K
 /* the same projection for many tokens from the bf16 copy of the residual, on the tensor cores, fp32 accumulation and output;
  * -2: K not a multiple of 8 or misaligned */
 int pk_proj_rows_f32out(const void* W, const void* xa, float* out, int M, int K, int tokens, pk_stream st);
-/* kind 0: out[t][f] = silu(in[t][f]) * in[t][F + f] (in [tokens, 2F]);  kind 1: out[t][f] = relu(in[t][f])^2 (in [tokens, F]) */
+/* kind 0: out[t][f] = silu(in[t][f]) * in[t][F + f] (in [tokens, 2F]);  kind 1: out[t][f] = relu(in[t][f])^2 (in [tokens, F]);
+ * kind 2: out[t][f] = relu(in[t][f]) * in[t][F + f] (in [tokens, 2F]) */
 int pk_act(const void* in, void* out, int F, int tokens, int kind, int f32, pk_stream st);
 int pk_convert(const void* in, int in_f32, void* out, int out_f32, long n, pk_stream st);
 /* Strided batched product in plain FMA arithmetic: C[b][i][j] = f(row_scale[i*ld_scale + b]) * sum_k A[b*bsA + i*lda + k] * B[b*bsB + k*sbk + j*sbn],
@@ -610,6 +612,53 @@ int pk_moe_up_act_p(const void* xa, const void* w_up, const int* ids, void* hid,
 int pk_moe_grouped_act_p(const void* xa, const void* w_up, const void* w_down, const int* ids, const float* weights, const void* shared,
                          const float* shared_gate, float* y, void* workspace, int tokens, int top, int experts, int width, int ff, int act, float p0,
                          float p1, pk_stream st);
+
+/* =============== residual in parallel streams, score-mixing attention with logistic weights, more recurrences ===============
+ * The residual is `streams` rows per token, x [tokens, streams, width] fp32.  A sublayer reads rms(sum_s w_in[s] x_s) * w and its result y returns to
+ * every stream at once: x_t <- sum_s mix[s * streams + t] x_s + w_out[t] y.  mix, w_in, w_out are float arrays on the device; streams <= 16. */
+/* x[t][s] = float(embed[ids[t]]) for every stream s;  h[t] = rms(sum_s w_in[s] x[t][s]) * w_next in the element type, h32 (may be NULL) unrounded
+ * (w_next NULL: no h) */
+int pk_res32_streams_embed(const void* embed, const int* token_ids, const float* w_in, float* x, const void* w_next, void* h, float* h32, int width,
+                           int streams, float eps, int tokens, int f32, pk_stream st);
+/* the write of one sublayer's result y (element type) and the read of the next sublayer (h / h32 as above) */
+int pk_res32_streams_step(const void* y, const float* mix, const float* w_out, const float* w_in, float* x, const void* w_next, void* h, float* h32,
+                          int width, int streams, float eps, int tokens, int f32, pk_stream st);
+/* out[r] = rms(sum_s x[rows[r]][s]) * w in the element type (rows NULL: every row);  w NULL: out32[r] = the sum of the streams */
+int pk_res32_streams_rows(const float* x, const int* rows, const void* w, void* out, float* out32, int width, int streams, float eps, int n_rows, int f32,
+                          pk_stream st);
+/* Grouped-query attention with mixed scores and logistic weights (gqa_mixed_attention.cu), cache as for pk_gqa_attention:
+ * s_h(j) = scale * q[t,h] . k_j;  z_h = sum_g score_mix[h * heads + g] s_g + head_bias[h] (score_mix element type, NULL: z_h = s_h + bias; head_bias float,
+ * may be NULL);  out[t,h] = out_scale * logistic(gate[t * gate_ld + h]) * sum_{j <= positions[t]} logistic(z_h(j)) v_j, not normalised over keys.
+ * gate: fp32 pre-activations, may be NULL.  out has rows of stride out_ld.  max_kv_len: longest context of the step (0: unknown), a hint for
+ * splitting the key axis. */
+int pk_gqa_mixed_attention(const void* q, const void* cache, const void* score_mix, const float* head_bias, const float* gate, int gate_ld,
+                           const int* positions, const int* req, const int* page_off, const int* pages, void* out, int out_ld, float out_scale,
+                           long page_stride, int page_size, int tokens, int heads, int kv_heads, int dim, int vdim, float scale, int max_kv_len, int f32,
+                           pk_stream st);
+/* Short causal convolution per channel of in + in_bias, plus bias, act 0: none / 1: SiLU (either bias may be NULL); the slot's state keeps the last
+ * taps - 1 biased inputs [taps-1][channels] and is updated by the same launch. */
+int pk_causal_conv(const void* in, int ld_in, const void* in_bias, const void* w, const void* bias, int act, float* state, long slot_stride,
+                   const int* slot, const int* row0, const int* len, void* out, int ld_out, int channels, int taps, int tokens, int entries, int f32,
+                   pk_stream st);
+/* pk_gated_delta_seq with one decay per head and key channel: decay [tokens, ld_decay] fp32 holds its pre-activation at h * dim + d,
+ * g = exp(-exp(a_log[h]) * softplus(decay + dt_bias[h * dim + d])). */
+int pk_channel_delta_seq(const void* qkv, int ld, int q_off, int k_off, int v_off, const float* z, int ldz, int beta_off, const float* decay, int ld_decay,
+                         const float* a_log, const float* dt_bias, float* state, long slot_stride, const int* slot, const int* row0, const int* len,
+                         float* out, int heads, int kv_heads, int dim, int vdim, int entries, int f32, pk_stream st);
+/* Real-gated linear recurrent unit, one scalar of state per channel: r = logistic(z_r + r_bias), i = logistic(z_i + i_bias), log a = -rate * r * softplus(lam),
+ * S <- a S + sqrt(1 - a^2) i u,  out = S * gelu_tanh(y + y_bias) (y_bias element type, may be NULL).  z [tokens, ldz] fp32: block b of n = channels / blocks
+ * channels has z_r at b * 2n + j and z_i at b * 2n + n + j. */
+int pk_lru_seq(const void* u, int ld_u, const float* z, int ldz, const float* r_bias, const float* i_bias, const float* lam, float rate, int blocks,
+               const void* y, int ld_y, const void* y_bias, float* state, long slot_stride, const int* slot, const int* row0, const int* len, void* out,
+               int ld_out, int channels, int tokens, int entries, int f32, pk_stream st);
+/* pk_head_norm_gate with rows of stride ld_out, the result multiplied by `factor` before it is rounded */
+int pk_head_norm_gate_ex(const float* o, const float* den, const void* w, int w_stride, const void* gate, int ld_gate, int gate_off, void* out, int ld_out,
+                         float factor, int tokens, int heads, int vdim, float eps, int act, int f32, pk_stream st);
+/* Strided batched product with fp32 results, both operands contraction-major: C[b*bsC + i*ldc + j] = sum_k A[b*bsA + i*lda + k] * B[b*bsB + j*ldb + k] */
+int pk_gemm_strided_f32out(const void* A, const void* B, float* C, int rows, int cols, int K, long lda, long ldb, long ldc, int batch, long bsA, long bsB,
+                           long bsC, int f32, pk_stream st);
+/* pk_b200_gemm_swiglu with a choice of the gate's activation: act 0 SiLU, 1 ReLU (pk_b200_gemv_args.epi 5 is the same for a few tokens) */
+int pk_b200_gemm_gated(const pk_bf16* W, const pk_bf16* X, pk_bf16* Y, int M, int N, int K, int act, pk_stream stream);
 
 #ifdef __cplusplus
 }

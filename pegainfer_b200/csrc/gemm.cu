@@ -440,9 +440,13 @@ extern "C" int pk_b200_gemm_segments(const pk_bf16* W, const pk_bf16* X, pk_bf16
 // Y[tok][M] = bf16(silu(bf16(gate.x)) * bf16(up.x)) -- gemm + silu_mul_fused_cuda of the reference in one launch, same
 // rounding points.  Returns -2 when the CTA-pair kernel cannot take the shape (caller runs the two-kernel sequence).
 extern "C" int pk_b200_gemm_swiglu(const pk_bf16* W, const pk_bf16* X, pk_bf16* Y, int M, int N, int K, pk_stream stream) {
-  if (!W || !X || !Y || M <= 0 || N <= 0 || K <= 0) return -1;
+  return pk_b200_gemm_gated(W, X, Y, M, N, K, 0, stream);
+}
+// the same with a choice of the gate's activation: 0 SiLU, 1 ReLU
+extern "C" int pk_b200_gemm_gated(const pk_bf16* W, const pk_bf16* X, pk_bf16* Y, int M, int N, int K, int act, pk_stream stream) {
+  if (!W || !X || !Y || M <= 0 || N <= 0 || K <= 0 || act < 0 || act > 1) return -1;
   if (!pk::gemm_pair_enabled() || pk::gemm_impl_mode() != 0) return -2;
-  return pk::launch_gemm_pair((const pk::bf16*)W, (const pk::bf16*)X, (pk::bf16*)Y, (pk::bf16*)Y, (pk::bf16*)Y, M, M, M, N, K, 1, stream);
+  return pk::launch_gemm_pair((const pk::bf16*)W, (const pk::bf16*)X, (pk::bf16*)Y, (pk::bf16*)Y, (pk::bf16*)Y, M, M, M, N, K, 1 + act, stream);
 }
 
 // Same dispatch as gemm_graphsafe_cuda (gemv.cu): N <= 4 streams the weights (HBM-bound GEMV), larger N runs on the

@@ -91,7 +91,7 @@ struct G2Args {
   bf16 *Y, *Y1, *Y2;
   int e0, e1;     // output segments (the fused q|k|v projection): features [0,e0) -> Y, [e0,e1) -> Y1, rest -> Y2
   int M, N, K;    // features, tokens, reduction
-  int swiglu;     // 1: W = [gate (M rows); up (M rows)], Y[tok][M] = silu(gate) * up
+  int swiglu;     // 1: W = [gate (M rows); up (M rows)], Y[tok][M] = silu(gate) * up; 2: relu(gate) * up
 };
 
 // A pair tile is 256 tokens x (NSUB * BN) features: NSUB accumulators of BN columns side by side in TMEM, one
@@ -224,7 +224,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant
             for (int j = 0; j < 32; ++j) {
               const float g = round_bf16(__uint_as_float(gv[j]));  // gate_up_out is bf16 in the reference
               const float u = round_bf16(__uint_as_float(uv[j]));
-              r[j] = g / (1.0f + expf(-g)) * u;
+              r[j] = (a.swiglu == 2 ? fmaxf(g, 0.f) : g / (1.0f + expf(-g))) * u;
             }
             if (M % 8 == 0 && f0 + 32 <= M && (reinterpret_cast<uintptr_t>(a.Y) & 15) == 0) {
 #pragma unroll

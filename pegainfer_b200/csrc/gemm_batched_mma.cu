@@ -107,6 +107,14 @@ int launch_gemm_batched_mma(const bf16* A, const bf16* B, bf16* C, const float* 
   return (int)e;
 }
 
+// the same product with fp32 results, no row factors (gates and decays of recurrences)
+int launch_gemm_batched_mma_f32(const bf16* A, const bf16* B, float* C, int rows, int cols, int K, long lda, long ldb, long ldc, int batch, long bsA,
+                                long bsB, long bsC, cudaStream_t st) {
+  if (K % 8 || lda % 8 || ldb % 8 || bsA % 8 || bsB % 8 || (reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(B) & 15)) return -2;
+  return (int)launch(gemm_batched_mma_kernel<float>, dim3((cols + kBT - 1) / kBT, (rows + kBT - 1) / kBT, batch), dim3(128), 0, st, true, A, B, C,
+                     (const float*)nullptr, rows, cols, K, lda, ldb, ldc, bsA, bsB, bsC, 0, 0);
+}
+
 }  // namespace pk
 
 // out[t][m] (fp32) = W[m] . xa[t] with bf16 operands and fp32 accumulation: the skinny projections (router logits, gates) of a

@@ -85,7 +85,7 @@ gemv_stream_kernel(const GemvArgs a) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int G = gridDim.x;
   const int M = a.M, K = a.K;
-  const bool glu = a.epi == 1 || a.epi == 4;  // interleaved gate / up row groups
+  const bool glu = a.epi == 1 || a.epi >= 4;  // interleaved gate / up row groups
   const int rows_per_group = glu ? kCW / 2 : kCW;
   const int r0 = (int)(((int64_t)blockIdx.x * M) / G);
   const int r1 = (int)(((int64_t)(blockIdx.x + 1) * M) / G);
@@ -317,7 +317,7 @@ gemv_stream_kernel(const GemvArgs a) {
         for (int n = 0; n < NTOK; ++n) {
           const float gt = round_bf16(acc[n]);                   // gate_up_out is bf16 in the reference
           const float up = round_bf16(sw[warp * NTOK + n]);
-          float sl = gt / (1.0f + expf(-gt));
+          float sl = a.epi == 5 ? fmaxf(gt, 0.f) : gt / (1.0f + expf(-gt));
           if (a.epi == 4) sl = round_bf16(sl);                   // Qwen3.5's unfused silu_mul rounds SiLU first (elementwise.cu:36-41)
           a.Y[0][(size_t)n * M + out_row] = f2bf(sl * up);
         }
@@ -462,7 +462,7 @@ bool gemv_stream_supported(const void* W, const void* X, int N, int K) {
 // CTA count of the streaming kernel: every CTA owns >= one row group, at most ctas_per_sm CTAs per SM.
 int gemv_grid(int M, int epi) {
   gemv_tuning();
-  const int rpg = (epi == 1 || epi == 4) ? kCW / 2 : kCW;
+  const int rpg = (epi == 1 || epi >= 4) ? kCW / 2 : kCW;
   int grid = sm_count() * g_gemv_ctas_per_sm;
   const int max_useful = (M + rpg - 1) / rpg;
   if (grid > max_useful) grid = max_useful;
@@ -557,7 +557,7 @@ int pk_b200_gemv_fused(const pk_b200_gemv_args* g, pk_stream stream) {
   if (!g || g->M <= 0 || g->K <= 0) return -1;
   if (!gemv_stream_supported(g->W, g->X, g->N, g->K)) return -1;
   if (g->x_mode >= 1 && (g->hidden_out == nullptr || g->hidden_out == g->X || g->K > 10240)) return -1;
-  if (g->x_mode < 0 || g->x_mode > 3 || g->epi < 0 || g->epi > 4) return -1;
+  if (g->x_mode < 0 || g->x_mode > 3 || g->epi < 0 || g->epi > 5) return -1;
   GemvArgs a{};
   a.W = (const bf16*)g->W;
   a.X = (const bf16*)g->X;

@@ -1,21 +1,26 @@
-// C++ host of the decoder designs whose checkpoint configuration lists the layers one by one (Vamadra, Risolorn, Nagosun, Goguzen), on an
-// fp32 residual stream.  A layer is a mixer plus an optional feed-forward, put together in one of four block forms:
+// C++ host of the decoder designs whose checkpoint configuration lists the layers one by one (Vamadra, Risolorn, Nagosun, Goguzen, Rilonex),
+// on an fp32 residual stream.  A layer is a mixer plus an optional feed-forward, put together in one of five block forms:
 //   block 0  sequential sublayers with the norm on each sublayer's OUTPUT:  x += norm(mixer(x));  x += norm(ff(x))
 //   block 1  parallel sublayers under one Dynamic-Tanh pre-norm:            h = dyt(x);  x += mixer(h) + ff(h)
 //   block 2  "sandwich": a grouped RMS norm before AND after each sublayer, the sublayer's result gated by a logistic
 //            projection of its input, the sum scaled:  h = gn(x); x += m * gn(f(h) * logistic(W_rg h + b))   (mixers 0 and 1)
 //   block 3  pre-norm sequential sublayers with plain-weight RMS norms:      x += mixer(rms(x) w1);  x += ff(rms(x) w2)   (mixers 1 and 4);
 //            a layer may run with another layer's weights (and a cache / state of its own); logits are scaled and soft-capped
+//   block 4  pre-norm sequential sublayers over a residual of parallel streams (hyper-connections): a sublayer reads u = sum_s in[s] x_s,
+//            h = rms(u) w, and its result y goes back as x_t <- sum_s mix[s][t] x_s + out[t] y   (mixers 2, 5 and 6)
 // Mixers: 0 latent attention (compressed paged cache, shared rotated key part, per-head sink, logistic output gate, optional
 // reuse of an earlier layer's cache); 1 grouped-query attention with biases, rotary embedding from a frequency table, a
 // chunk-local causal mask and a sink, over a paged K/V cache (block 2 adds: sliding window, score soft cap, linear distance
 // bias, unit-RMS cached values, a sink of score zero, an element-wise output gate); 2 gated delta rule behind short causal
 // convolutions; 3 xLSTM matrix memory; 4 two branches side by side on the same input -- grouped-query attention and a state-space layer
 // (scalar decay per head, short causal convolution, gated group-normed read-out) -- each branch's result RMS-normed over the width, the
-// mixer's result their mean.  Block 3 gives the attention (mixer 1 and the attention branch of 4) further options: RMS norm of q and k per
+// mixer's result their mean; 5 real-gated linear recurrent unit behind a short convolution, times a GELU branch; 6 two branches side by
+// side -- grouped-query attention with mixed scores, logistic weights and a gate per head, and a gated delta rule -- summed with constants.
+// In block 4 the delta rule may decay per head and key channel and its read-out gate may be logistic, both through low-rank projections.
+// Block 3 gives the attention (mixer 1 and the attention branch of 4) further options: RMS norm of q and k per
 // head or over the whole projection, a query factor that grows with the logarithm of the position, values that are the keys as projected,
-// a window that keeps the first positions visible, rotary frequencies rescaled by wavelength.  Mixers 2, 3 and 4 keep an fp32 state per
-// request in numbered state slots.  Feed-forward: dense SwiGLU or a mixture of experts (softmax or logistic router or plain top logits;
+// a window that keeps the first positions visible, rotary frequencies rescaled by wavelength.  Mixers 2 to 6 keep an fp32 state per
+// request in numbered state slots.  Feed-forward: dense SwiGLU, dense with a ReLU gate, or a mixture of experts (softmax or logistic router or plain top logits;
 // relu^2, gated-SiLU or clamped gated experts; a shared expert with or without a gate).
 //
 // Same structure as the other hosts in this folder: kernels are reached only through the C ABI
@@ -84,6 +89,14 @@ struct LayerCfg {  // mirrored by ctypes in pegainfer_b200/vamadra.py
   float act_limit, act_slope;  // expert_act 2: g = min(gate, limit), u = clamp(up, +-limit), g logistic(slope g) (u + 1)
   float shared_limit;        // the shared expert's limit (router_kind 2: shared expert of the same form, no gate)
   int weights_of;            // >= 0: the layer runs with that layer's weights
+  // options read by block 4.  Mixer 2 and the recurrent branch of mixer 6 take their delta rule from d_*; mixer 6's attention the fields above
+  int d_heads, d_kv_heads, d_dim, d_vdim;
+  int decay_rank;            // 0: one decay per head (projection 'a'); > 0: per head and key channel, through 'a1' [rank, width] and 'a2'
+  int gate_rank;             // 0: read-out gate silu(W_g h); > 0: logistic, through 'g1' [rank, width] and 'g2'
+  float left_scale, right_scale;  // 6: factors of the attention's and the delta rule's result
+  int lru_width, lru_blocks;      // 5
+  float lru_rate;                 // 5: log a = -lru_rate * r * softplus(lam)
+  int mlp_act;               // dense feed-forward: 0 SiLU gate, 1 ReLU gate
 };
 struct ModelCfg {
   int vocab, width, n_layers;
@@ -95,6 +108,7 @@ struct ModelCfg {
   float residual_mult;    // block 2: multiplier of every sublayer's normed result
   int gated_residual;     // block 2: sublayer results times logistic(W_rg h + b) ('rg1' / 'rg2') before their norm
   float logit_softcap;    // block 3: logits <- cap * tanh(logits / cap) after the multiplier (0: none)
+  int streams;            // block 4: parallel rows of the residual; 0: one row, x += y, no stream weights in the checkpoint
 };
 
 struct Lib {
@@ -104,23 +118,29 @@ struct Lib {
   X(cuda_set_device) X(cublas_init) X(cublas_destroy) X(gemm_cuda) X(flashinfer_top1_cuda) X(pk_b200_set_pdl) X(pk_b200_launch_count)      \
   X(pk_res32_skinny_proj) X(pk_convert) X(pk_gemm_strided) X(pk_proj_rows_f32out) X(pk_scale_to_f32) X(pk_top1_rows_f32)
 #define PV_MOE(X) X(pk_moe_down_combine) X(pk_moe_grouped_workspace_bytes) X(pk_moe_up_act_p) X(pk_moe_grouped_act_p)
-#define PV_DENSE(X) X(pk_act) X(pk_b200_gemv_fused) X(pk_b200_gemm_swiglu)
+#define PV_DENSE(X) X(pk_act) X(pk_b200_gemv_fused) X(pk_b200_gemm_gated)
 #define PV_BLOCK0(X)                                                                                                                        \
   X(pk_res32_embed) X(pk_res32_offset_norm_add) X(pk_res32_offset_norm_rows) X(pk_rope_slice) X(pk_latent_kv_append) X(pk_latent_attention) \
   X(pk_router_grouped_topk)
 #define PV_BLOCK1(X)                                                                                                                        \
   X(pk_res32_embed_scaled) X(pk_res32_add_dyt) X(pk_res32_dyt_rows) X(pk_gqa_rope_append) X(pk_gqa_attention) X(pk_causal_conv_silu)       \
-  X(pk_gated_delta_seq) X(pk_mlstm_seq) X(pk_router_topk_ex)
+  X(pk_mlstm_seq) X(pk_router_topk_ex)
 #define PV_BLOCK13(X) X(pk_head_norm_gate)
 #define PV_BLOCK23(X) X(pk_res32_gnorm_rows) X(pk_gqa_attention_ex)
 #define PV_BLOCK3(X)                                                                                                                        \
   X(pk_res32_embed_scaled_norm) X(pk_res32_branches_add_norm) X(pk_logits_scale_cap) X(pk_act_clamped) X(pk_gqa_norm_append)               \
   X(pk_causal_conv_silu_bias) X(pk_ssd_seq) X(pk_router_topk_logits)
 #define PV_BLOCK2(X)                                                                                                                        \
-  X(pk_res32_embed_gnorm) X(pk_res32_gated_gnorm_add) X(pk_gqa_rope_append_ex) X(pk_rope_slice_ex)   \
+  X(pk_res32_embed_gnorm) X(pk_res32_gated_gnorm_add) X(pk_rope_slice_ex)   \
   X(pk_latent_kv_append_ex) X(pk_latent_attention_ex) X(pk_b200_gemm_segments)
+#define PV_BLOCK14(X) X(pk_gated_delta_seq)
+#define PV_BLOCK24(X) X(pk_gqa_rope_append_ex)
+#define PV_BLOCK4(X)                                                                                                                        \
+  X(pk_res32_streams_embed) X(pk_res32_streams_step) X(pk_res32_streams_rows) X(pk_gqa_mixed_attention) X(pk_causal_conv)                  \
+  X(pk_channel_delta_seq) X(pk_lru_seq) X(pk_head_norm_gate_ex) X(pk_gemm_strided_f32out)
 #define PV_FN(name) decltype(&::name) name = nullptr;
-  PV_COMMON(PV_FN) PV_MOE(PV_FN) PV_DENSE(PV_FN) PV_BLOCK0(PV_FN) PV_BLOCK1(PV_FN) PV_BLOCK2(PV_FN) PV_BLOCK13(PV_FN) PV_BLOCK23(PV_FN) PV_BLOCK3(PV_FN)
+  PV_COMMON(PV_FN) PV_MOE(PV_FN) PV_DENSE(PV_FN) PV_BLOCK0(PV_FN) PV_BLOCK1(PV_FN) PV_BLOCK2(PV_FN) PV_BLOCK3(PV_FN) PV_BLOCK4(PV_FN)
+  PV_BLOCK13(PV_FN) PV_BLOCK14(PV_FN) PV_BLOCK23(PV_FN) PV_BLOCK24(PV_FN)
 #undef PV_FN
   // a library built for one design need not hold the other block form's kernels: only what `block_kind` runs is required
   std::string load(const std::string& p, int block_kind) {
@@ -134,9 +154,11 @@ struct Lib {
     if (block_kind == 0) {
       PV_MOE(PV_REQ) PV_DENSE(PV_REQ) PV_BLOCK0(PV_REQ)
     } else if (block_kind == 1) {
-      PV_MOE(PV_REQ) PV_BLOCK1(PV_REQ) PV_BLOCK13(PV_REQ)
+      PV_MOE(PV_REQ) PV_BLOCK1(PV_REQ) PV_BLOCK13(PV_REQ) PV_BLOCK14(PV_REQ)
     } else if (block_kind == 2) {  // the sandwich block form has no mixture of experts
-      PV_DENSE(PV_REQ) PV_BLOCK2(PV_REQ) PV_BLOCK23(PV_REQ)
+      PV_DENSE(PV_REQ) PV_BLOCK2(PV_REQ) PV_BLOCK23(PV_REQ) PV_BLOCK24(PV_REQ)
+    } else if (block_kind == 4) {  // no mixture of experts either
+      PV_DENSE(PV_REQ) PV_BLOCK4(PV_REQ) PV_BLOCK14(PV_REQ) PV_BLOCK24(PV_REQ)
     } else {
       PV_MOE(PV_REQ) PV_BLOCK3(PV_REQ) PV_BLOCK13(PV_REQ) PV_BLOCK23(PV_REQ)
     }
@@ -166,6 +188,8 @@ struct Layer {
   DeviceBuf alpha32, corr32, p0_32, p1_32, p2_32;          // float copies of small parameter vectors (made in finalize)
   Mat alpha, corr, p0, p1, p2;
   Mat qn, kn, conv_b, o2, lout, rout;                      // block 3: q / k norm weights; mixer 4: convolution bias, second output projection, branch norms
+  Mat a2, g2, gates, conv_in_b, r_bias, i_bias, talk, hc[2][3];  // block 4: low-rank second factors; linear unit; score mixing; stream weights in / out / mix
+  DeviceBuf hc32[2][3];
   int wsrc = 0;                                            // the layer whose weights this layer runs with (itself unless the configuration says otherwise)
   int64_t state_off = 0;                                   // float offset of the layer's block inside a state slot
   DeviceBuf freq;                                          // [rot_dims / 2] fp32 angular frequencies
@@ -198,6 +222,7 @@ struct Model {
   int cap_t = 0, cap_r = 0;
   DeviceBuf h32, big, convo, zs, orec, den;  // block 1: unrounded norm output, stacked projections, conv outputs, few-row fp32, read-out
   DeviceBuf ao2, mix2;                       // mixer 4: the state-space branch's gated read-out and its projection
+  DeviceBuf zc, gbuf, one32;                 // block 4: fp32 decay / gate pre-activations, low-rank read-out gate; the constant 1 (weights of a single stream)
   DeviceBuf x, xa, q, dkv, qa, gate, olat, ao, mix, gu, act, z, ids, wts, hid, yf, sgl, sh, xr, logits_e, logits_f, logits_bf, sampled_d, top1_val,
       top1_states, trail, moe_ws;
   DeviceBuf meta_d;
@@ -213,7 +238,7 @@ struct Model {
   std::set<GraphKey> seen;
   bool use_graph = true;
   // widest layer
-  int mx_big = 0, mx_conv = 0, mx_small = 0, mx_inner = 0;
+  int mx_big = 0, mx_conv = 0, mx_small = 0, mx_inner = 0, mx_zc = 0, mx_gbuf = 0, n_streams = 1;
   int mx_q = 0, mx_dkv = 0, mx_qa = 0, mx_h = 0, mx_olat = 0, mx_ao = 0, mx_gu = 0, mx_act = 0, mx_e = 0, mx_top = 0, mx_hid = 0;
 
   bool fail(const std::string& m) {
@@ -252,6 +277,12 @@ struct Model {
   bool run_prenorm_layer(int li, int T, int max_kv, const int* M, int n);
   bool run_parallel_layer(int li, int T, const int* M, int n);
   bool run_sandwich_layer(int li, int T, int max_kv, const int* M);
+  bool run_streams_layer(int li, int T, int max_kv, const int* M, int n);
+  bool delta_branch(const Layer& L, const char* rows, int nbig, const float* small, int nsmall, float* slot0, void* out, int ld_out, float factor, int T,
+                    const int* M, int n);
+  bool gated_ff(const Layer& L, int T);
+  bool load_streams_tensor(Layer& L, const std::string& sub, const std::string& name, const void* data, int rows, int cols, bool* known);
+  bool put_cols(Mat& m, int rows, int cols, int col0, const void* src, int src_cols, const std::string& name, int got_rows, int got_cols);
   bool lin_segments(const Mat& W, const void* X, void* const* Y, const int* seg_rows, int N);
   bool run_layer(int li, int T, int max_kv, const int* d_pos, const int* d_req, const int* d_poff, const int* d_pages);
   bool forward(int T, int n, int n_rows, int max_kv, int want_sample);
@@ -264,13 +295,26 @@ struct Model {
   }
 };
 
+// sizes of a layer's delta rule in block 4 (mixer 2, or the recurrent branch of mixer 6)
+struct DeltaDims {
+  int H, G, D, V, nq, nk, nv, C, ng, rank_a, rank_g;  // C: channels of the short convolutions; ng: rows of an ungated-rank read-out gate
+  explicit DeltaDims(const LayerCfg& a)
+      : H(a.d_heads), G(a.d_kv_heads), D(a.d_dim), V(a.d_vdim), nq(G * D), nk(G * D), nv(H * V), C(nq + nk + nv), ng(a.gate_rank > 0 ? 0 : H * V),
+        rank_a(a.decay_rank), rank_g(a.gate_rank) {}
+  int big() const { return C + ng + rank_a + rank_g; }        // stacked [q | k | v (| g) (| a1) (| g1)]
+  int small() const { return (rank_a > 0 ? 0 : H) + H; }      // few-row fp32 projections [(a) | b]
+  int64_t state(int taps) const { return (int64_t)H * D * V + (int64_t)std::max(taps - 1, 0) * C; }
+};
+
 static std::string lname(int i, const char* s) { return "l" + std::to_string(i) + "." + s; }
 
 bool Model::configure(const ModelCfg& mc, const LayerCfg* lc) {
   c = mc;
   es = c.f32 ? 4 : 2;
   if (c.vocab <= 0 || c.width <= 0 || c.n_layers <= 0) return fail("vocab, width and the number of layers must be positive");
-  if (c.block_kind < 0 || c.block_kind > 3) return fail("unknown block form");
+  if (c.block_kind < 0 || c.block_kind > 4) return fail("unknown block form");
+  if (c.streams < 0 || c.streams > 16) return fail("streams: 1 to 16 parallel rows of the residual");
+  n_streams = c.block_kind == 4 ? std::max(c.streams, 1) : 1;
   if (c.block_kind == 3 && c.logit_softcap < 0.f) return fail("logit_softcap must not be negative");
   if (c.block_kind == 2 && (c.norm_groups <= 0 || c.width % c.norm_groups)) return fail("norm.groups must divide the width");
   if (c.page_size <= 0) c.page_size = 16;
@@ -281,7 +325,58 @@ bool Model::configure(const ModelCfg& mc, const LayerCfg* lc) {
     Layer& L = layers[i];
     L.c = lc[i];
     const LayerCfg& a = L.c;
-    if (a.mixer_kind < 0 || a.mixer_kind > 4) return fail(lname(i, "mixer: unknown kind"));
+    if (a.mixer_kind < 0 || a.mixer_kind > 6) return fail(lname(i, "mixer: unknown kind"));
+    if (c.block_kind == 4) {
+      if (a.mixer_kind != 2 && a.mixer_kind < 5) return fail(lname(i, "mixer: not available in this block form"));
+      L.wsrc = i;
+      L.state_off = soff;
+      int wide = 0;  // input of the output projection
+      if (a.mixer_kind == 5) {
+        if (a.lru_width <= 0 || a.lru_blocks <= 0 || a.lru_width % a.lru_blocks || a.conv <= 0 || !(a.lru_rate > 0.f))
+          return fail(lname(i, "mixer: inconsistent linear recurrent unit (width, blocks, conv)"));
+        soff += (int64_t)a.lru_width * a.conv;  // the state and the convolution's last conv - 1 inputs
+        mx_big = std::max(mx_big, 2 * a.lru_width);
+        mx_conv = std::max(mx_conv, a.lru_width);
+        mx_zc = std::max(mx_zc, 2 * a.lru_width);
+        wide = a.lru_width;
+      } else {
+        if (a.d_heads <= 0 || a.d_kv_heads <= 0 || a.d_heads % a.d_kv_heads || a.d_dim <= 0 || a.d_vdim <= 0 || a.conv <= 0 || a.decay_rank < 0 || a.gate_rank < 0)
+          return fail(lname(i, "mixer: inconsistent delta rule"));
+        if (a.d_dim > 256) return fail(lname(i, "mixer: head sizes above 256 are outside the kernels' range"));
+        const DeltaDims d(a);
+        soff += d.state(a.conv);
+        int nbig = d.big(), nsmall = d.small();
+        if (a.mixer_kind == 6) {
+          if (a.heads <= 0 || a.kv_heads <= 0 || a.heads % a.kv_heads || a.dim <= 0 || a.vdim <= 0) return fail(lname(i, "mixer: inconsistent attention"));
+          if (a.rot_dims < 0 || a.rot_dims > a.dim || (a.rot_dims & 1)) return fail(lname(i, "mixer: rot.dims must be even and at most dim"));
+          L.owner = i;
+          L.cache_off = off;
+          off += (int64_t)c.page_size * a.kv_heads * (a.dim + a.vdim);
+          off = (off + 7) / 8 * 8;  // every layer's block starts 16-byte aligned in both element types
+          nbig += a.heads * a.dim + a.kv_heads * (a.dim + a.vdim);
+          nsmall += a.heads;
+          mx_q = std::max(mx_q, a.heads * a.dim);
+          wide = a.heads * a.vdim;
+        }
+        mx_big = std::max(mx_big, nbig);
+        mx_small = std::max(mx_small, nsmall);
+        mx_conv = std::max(mx_conv, d.C);
+        mx_inner = std::max(mx_inner, d.nv);
+        if (d.rank_a > 0) mx_zc = std::max(mx_zc, d.H * d.D);
+        if (d.rank_g > 0) mx_gbuf = std::max(mx_gbuf, d.nv);
+        wide += d.nv;
+      }
+      mx_ao = std::max(mx_ao, wide);
+      soff = (soff + 3) / 4 * 4;
+      if (a.mlp_kind != 0 && a.mlp_kind != 1) return fail(lname(i, "mlp: this block form has dense feed-forwards only"));
+      if (a.mlp_kind == 1) {
+        if (a.ff <= 0) return fail(lname(i, "mlp: ff must be positive"));
+        mx_gu = std::max(mx_gu, 2 * a.ff);
+        mx_act = std::max(mx_act, a.ff);
+      }
+      continue;
+    }
+    if (a.mixer_kind > 4) return fail(lname(i, "mixer: not available in this block form"));
     if (c.block_kind == 3 ? (a.mixer_kind != 1 && a.mixer_kind != 4)
                           : a.mixer_kind == 4 || (c.block_kind == 2 ? a.mixer_kind > 1 : (a.mixer_kind == 0) != (c.block_kind == 0)))
       return fail(lname(i, "mixer: not available in this block form"));
@@ -418,6 +513,18 @@ bool Model::put_rows(Mat& m, int rows, int cols, int row0, int row_step, const v
             name.c_str());
 }
 
+// the same with destination columns col0 .. col0 + src_cols of a [rows, cols] matrix (two matrices side by side along the contraction axis)
+bool Model::put_cols(Mat& m, int rows, int cols, int col0, const void* src, int src_cols, const std::string& name, int got_rows, int got_cols) {
+  if (got_rows != rows || got_cols != src_cols) return fail(name + ": shape does not match the configuration");
+  if (!m.d.ptr) {
+    m.rows = rows;
+    m.cols = cols;
+    if (!m.d.alloc_zeros((size_t)rows * cols * es)) return fail("allocation failed for " + name);
+  }
+  return cu(cudaMemcpy2D((char*)m.d.ptr + (size_t)col0 * es, (size_t)cols * es, src, (size_t)src_cols * es, (size_t)src_cols * es, rows, cudaMemcpyDefault),
+            name.c_str());
+}
+
 // W_uk [heads * dim, rank] as stored, and a second copy with the contraction axis of the query fold contiguous: [head][rank][dim]
 bool Model::put_uk(Layer& L, const void* data, const std::string& name, int rows, int cols) {
   const LayerCfg& a = L.c;
@@ -440,6 +547,85 @@ bool Model::to_f32(const Mat& m, DeviceBuf* out) {
   return rc(k.pk_convert(m.d.ptr, c.f32, out->ptr, 1, n, st), "parameter conversion");
 }
 
+// a tensor of a block 4 layer; *known = false: not one of this layer's.  The mixer's projections are stacked
+//   mixer 2  [q | k | v (| g) (| a1) (| g1)]        mixer 6  [q | k | v of the attention | the same of the delta rule]        mixer 5  [x | y]
+// and its few-row fp32 projections [head gate of the attention | (a) | b].
+bool Model::load_streams_tensor(Layer& L, const std::string& sub, const std::string& name, const void* data, int rows, int cols, bool* known) {
+  const LayerCfg& a = L.c;
+  const int W = c.width, S = n_streams;
+  *known = true;
+  if (sub == "norm1") return put(L.norm1, 1, W, 0, data, 1, name, rows, cols);
+  if (a.mlp_kind && sub == "norm2") return put(L.norm2, 1, W, 0, data, 1, name, rows, cols);
+  if (c.streams > 0 && sub.size() > 4 && sub.compare(0, 2, "hc") == 0 && (sub[2] == '1' || (sub[2] == '2' && a.mlp_kind)) && sub[3] == '.') {
+    const int q = sub[2] - '1';
+    const std::string part = sub.substr(4);
+    if (part == "in") return put(L.hc[q][0], 1, S, 0, data, 1, name, rows, cols);
+    if (part == "out") return put(L.hc[q][1], 1, S, 0, data, 1, name, rows, cols);
+    if (part == "mix") return put(L.hc[q][2], S, S, 0, data, S, name, rows, cols);
+  }
+  if (a.mlp_kind == 1) {
+    if (sub == "mlp.gate") return put(L.gate_up, 2 * a.ff, W, 0, data, a.ff, name, rows, cols);
+    if (sub == "mlp.up") return put(L.gate_up, 2 * a.ff, W, a.ff, data, a.ff, name, rows, cols);
+    if (sub == "mlp.down") return put(L.down, W, a.ff, 0, data, W, name, rows, cols);
+  }
+  if (a.mixer_kind == 5) {
+    const int C = a.lru_width, nb = a.lru_blocks, n = C / nb;
+    if (sub == "mix.x") return put(L.qkv, 2 * C, W, 0, data, C, name, rows, cols);
+    if (sub == "mix.y") return put(L.qkv, 2 * C, W, C, data, C, name, rows, cols);
+    if (sub == "mix.x.b") return put(L.conv_in_b, 1, C, 0, data, 1, name, rows, cols);
+    if (sub == "mix.y.b") return put(L.qkv_bias, 1, C, 0, data, 1, name, rows, cols);
+    if (sub == "mix.conv") return put(L.conv_w, C, a.conv, 0, data, C, name, rows, cols);
+    if (sub == "mix.conv.b") return put(L.conv_b, 1, C, 0, data, 1, name, rows, cols);
+    if (sub == "mix.ra.b") return put(L.r_bias, nb, n, 0, data, nb, name, rows, cols);
+    if (sub == "mix.ri.b") return put(L.i_bias, nb, n, 0, data, nb, name, rows, cols);
+    if (sub == "mix.lam") return put(L.p0, 1, C, 0, data, 1, name, rows, cols);
+    if (sub == "mix.o") return put(L.o, W, C, 0, data, W, name, rows, cols);
+    if (sub == "mix.ra" || sub == "mix.ri") {  // [nb, n, n] each -> per block the rows [ra ; ri]
+      if (rows != C || cols != n) return fail(name + ": shape does not match the configuration");
+      for (int b = 0; b < nb; ++b)
+        if (!put(L.gates, 2 * C, n, b * 2 * n + (sub == "mix.ri" ? n : 0), (const char*)data + (size_t)b * n * n * es, n, name, n, n)) return false;
+      return true;
+    }
+  } else {
+    const DeltaDims d(a);
+    const bool two = a.mixer_kind == 6;
+    const int H = two ? a.heads : 0, nq = two ? H * a.dim : 0, nk = two ? a.kv_heads * a.dim : 0, nv = two ? a.kv_heads * a.vdim : 0, r0 = nq + nk + nv;
+    const int nbig = r0 + d.big(), nsmall = H + d.small(), wo = two ? H * a.vdim : 0;
+    if (two) {
+      if (sub == "mix.left.q") return put(L.qkv, nbig, W, 0, data, nq, name, rows, cols);
+      if (sub == "mix.left.k") return put(L.qkv, nbig, W, nq, data, nk, name, rows, cols);
+      if (sub == "mix.left.v") return put(L.qkv, nbig, W, nq + nk, data, nv, name, rows, cols);
+      if (sub == "mix.left.g") return put(L.small, nsmall, W, 0, data, H, name, rows, cols);
+      if (sub == "mix.left.talk") return put(L.talk, H, H, 0, data, H, name, rows, cols);
+      if (sub == "mix.left.pb") return put(L.p2, 1, H, 0, data, 1, name, rows, cols);
+      if (sub == "mix.left.o") return put_cols(L.o, W, wo + d.nv, 0, data, wo, name, rows, cols);
+    }
+    const std::string pre = two ? "mix.right." : "mix.";
+    if (sub.compare(0, pre.size(), pre) == 0) {
+      const std::string t = sub.substr(pre.size());
+      if (t == "q") return put(L.qkv, nbig, W, r0, data, d.nq, name, rows, cols);
+      if (t == "k") return put(L.qkv, nbig, W, r0 + d.nq, data, d.nk, name, rows, cols);
+      if (t == "v") return put(L.qkv, nbig, W, r0 + d.nq + d.nk, data, d.nv, name, rows, cols);
+      if (t == "q.conv") return put(L.conv_w, d.C, a.conv, 0, data, d.nq, name, rows, cols);
+      if (t == "k.conv") return put(L.conv_w, d.C, a.conv, d.nq, data, d.nk, name, rows, cols);
+      if (t == "v.conv") return put(L.conv_w, d.C, a.conv, d.nq + d.nk, data, d.nv, name, rows, cols);
+      if (!d.rank_g && t == "g") return put(L.qkv, nbig, W, r0 + d.C, data, d.ng, name, rows, cols);
+      if (d.rank_a && t == "a1") return put(L.qkv, nbig, W, r0 + d.C + d.ng, data, d.rank_a, name, rows, cols);
+      if (d.rank_g && t == "g1") return put(L.qkv, nbig, W, r0 + d.C + d.ng + d.rank_a, data, d.rank_g, name, rows, cols);
+      if (d.rank_a && t == "a2") return put(L.a2, d.H * d.D, d.rank_a, 0, data, d.H * d.D, name, rows, cols);
+      if (d.rank_g && t == "g2") return put(L.g2, d.nv, d.rank_g, 0, data, d.nv, name, rows, cols);
+      if (!d.rank_a && t == "a") return put(L.small, nsmall, W, H, data, d.H, name, rows, cols);
+      if (t == "b") return put(L.small, nsmall, W, nsmall - d.H, data, d.H, name, rows, cols);
+      if (t == "A_log") return put(L.p0, 1, d.H, 0, data, 1, name, rows, cols);
+      if (t == "dt_bias") return put(L.p1, 1, d.rank_a ? d.H * d.D : d.H, 0, data, 1, name, rows, cols);
+      if (t == "norm") return put(L.hnorm, 1, d.V, 0, data, 1, name, rows, cols);
+      if (t == "o") return put_cols(L.o, W, wo + d.nv, wo, data, d.nv, name, rows, cols);
+    }
+  }
+  *known = false;
+  return false;
+}
+
 bool Model::load_tensor(const std::string& name, const void* data, int rows, int cols, int is_f32) {
   if ((is_f32 != 0) != (c.f32 != 0)) return fail(name + ": element type differs from the model's");
   const int W = c.width;
@@ -458,6 +644,13 @@ bool Model::load_tensor(const std::string& name, const void* data, int rows, int
   const LayerCfg& a = L.c;
   const std::string sub = name.substr(dot + 1);
   bool ok;
+  if (c.block_kind == 4) {
+    bool known;
+    ok = load_streams_tensor(L, sub, name, data, rows, cols, &known);
+    if (!known) return fail("unknown tensor " + name + " for the configuration of layer " + std::to_string(li));
+    if (ok) L.got.insert(sub);
+    return ok;
+  }
   if (c.block_kind == 1) {
     // parallel block: one Dynamic-Tanh norm; projections stacked [q | k | v (| gate)], few-row fp32 projections [router | za | zb]
     const int H = a.heads, G = a.kv_heads, mk = a.mixer_kind;
@@ -688,13 +881,34 @@ bool Model::finalize() {
   if (c.block_kind == 2 && !embed_norm.d.ptr) return fail("embed.norm missing");
   if (c.block_kind == 2 && !zero_sink.alloc_zeros((size_t)std::max(mx_h, 1) * es)) return fail("allocation failed");
   if (c.block_kind == 1 && (!final_b.d.ptr || !final_alpha.d.ptr || !to_f32(final_alpha, &final_alpha32))) return fail("final.norm.b / final.norm.alpha missing");
+  if (c.block_kind == 4) {
+    const float one = 1.f;
+    if (!one32.alloc_zeros(4) || !cu(cudaMemcpy(one32.ptr, &one, 4, cudaMemcpyHostToDevice), "constants")) return fail("allocation failed");
+  }
   if (slot_stride > 0 && !state.alloc_zeros((size_t)c.max_requests * slot_stride * 4)) return fail("state slot allocation failed");
   if (page_stride == 0) page_stride = 8;  // no layer keeps a paged cache: the pool only counts tokens
   for (int i = 0; i < c.n_layers; ++i) {
     Layer& L = layers[i];
     const LayerCfg& a = L.c;
     std::vector<std::string> need;
-    if (c.block_kind == 3) {
+    if (c.block_kind == 4) {
+      need = {"norm1"};
+      if (a.mlp_kind) need.push_back("norm2");
+      for (int q = 0; q < (c.streams > 0 ? (a.mlp_kind ? 2 : 1) : 0); ++q)
+        for (const char* n : {".in", ".out", ".mix"}) need.push_back("hc" + std::to_string(q + 1) + n);
+      if (a.mixer_kind == 5)
+        for (const char* n : {"x", "y", "x.b", "y.b", "conv", "conv.b", "ra", "ri", "ra.b", "ri.b", "lam", "o"}) need.push_back(std::string("mix.") + n);
+      if (a.mixer_kind == 6)
+        for (const char* n : {"q", "k", "v", "g", "talk", "pb", "o"}) need.push_back(std::string("mix.left.") + n);
+      if (a.mixer_kind != 5) {
+        const std::string pre = a.mixer_kind == 6 ? "mix.right." : "mix.";
+        for (const char* n : {"q", "k", "v", "q.conv", "k.conv", "v.conv", "b", "A_log", "dt_bias", "norm", "o"}) need.push_back(pre + n);
+        need.push_back(pre + (a.decay_rank ? "a1" : "a"));
+        need.push_back(pre + (a.gate_rank ? "g1" : "g"));
+        if (a.decay_rank) need.push_back(pre + "a2");
+        if (a.gate_rank) need.push_back(pre + "g2");
+      }
+    } else if (c.block_kind == 3) {
       if (L.wsrc == i) {
         const std::string am = a.mixer_kind == 4 ? "mix.left." : "mix.";
         need = {"norm1", am + "q", am + "k", am + "o"};
@@ -749,6 +963,16 @@ bool Model::finalize() {
       if (a.mlp_kind == 2 && !to_f32(L.corr, &L.corr32)) return false;
       if (a.mixer_kind == 4 && (!to_f32(L.p0, &L.p0_32) || !to_f32(L.p1, &L.p1_32) || !to_f32(L.p2, &L.p2_32))) return false;
     }
+    if (c.block_kind == 4) {  // parameters that enter fp32 arithmetic only
+      for (int q = 0; q < (c.streams > 0 ? (a.mlp_kind ? 2 : 1) : 0); ++q)
+        for (int j = 0; j < 3; ++j)
+          if (!to_f32(L.hc[q][j], &L.hc32[q][j])) return false;
+      if (!to_f32(L.p0, &L.p0_32)) return false;
+      if (a.mixer_kind == 5 && (!to_f32(L.r_bias, &L.p1_32) || !to_f32(L.i_bias, &L.p2_32))) return false;
+      if (a.mixer_kind != 5 && !to_f32(L.p1, &L.p1_32)) return false;
+      if (a.mixer_kind == 6 && !to_f32(L.p2, &L.p2_32)) return false;
+      if (a.mixer_kind != 6) continue;  // only the attention rotates
+    }
     if (c.block_kind >= 2 && a.rot_dims == 0) continue;  // nothing rotates
     std::vector<float> f;
     rotary_table(a, &f, &L.mag);
@@ -779,7 +1003,7 @@ bool Model::ensure_scratch(int T, int R) {
     cudaStreamSynchronize(st);
     drop_graphs();
     const size_t n = ((size_t)T + 63) / 64 * 64, W = c.width;
-    ok = x.alloc_uninit(n * W * 4) && xa.alloc_uninit(n * W * es) && q.alloc_uninit(n * mx_q * es) && dkv.alloc_uninit(n * mx_dkv * es) &&
+    ok = x.alloc_uninit(n * W * 4 * n_streams) && xa.alloc_uninit(n * W * es) && q.alloc_uninit(n * mx_q * es) && dkv.alloc_uninit(n * mx_dkv * es) &&
          qa.alloc_uninit(n * mx_qa * es) && gate.alloc_uninit(n * mx_h * 4) && olat.alloc_uninit(n * mx_olat * es) &&
          ao.alloc_uninit(n * mx_ao * es) && mix.alloc_uninit(n * W * es) && gu.alloc_uninit(n * std::max(mx_gu, 1) * es) &&
          act.alloc_uninit(n * std::max(mx_act, 1) * es) && z.alloc_uninit(n * std::max(mx_e, 1) * 4) && ids.alloc_uninit(n * std::max(mx_top, 1) * 4) &&
@@ -788,6 +1012,10 @@ bool Model::ensure_scratch(int T, int R) {
     if (ok && c.block_kind == 1)
       ok = h32.alloc_uninit(n * W * 4) && big.alloc_uninit(n * std::max(mx_big, 1) * es) && convo.alloc_uninit(n * std::max(mx_conv, 1) * es) &&
            zs.alloc_uninit(n * std::max(mx_small, 1) * 4) && orec.alloc_uninit(n * std::max(mx_ao, 1) * 4) && den.alloc_uninit(n * std::max(mx_h, 1) * 4);
+    if (ok && c.block_kind == 4)
+      ok = h32.alloc_uninit(n * W * 4) && big.alloc_uninit(n * std::max(mx_big, 1) * es) && convo.alloc_uninit(n * std::max(mx_conv, 1) * es) &&
+           zs.alloc_uninit(n * std::max(mx_small, 1) * 4) && orec.alloc_uninit(n * std::max(mx_inner, 1) * 4) && zc.alloc_uninit(n * std::max(mx_zc, 1) * 4) &&
+           gbuf.alloc_uninit(n * std::max(mx_gbuf, 1) * es);
     if (ok && c.block_kind == 2) ok = big.alloc_uninit(n * std::max(mx_big, 1) * es) && rgbuf.alloc_uninit(n * W * es);
     if (ok && c.block_kind == 3)
       ok = h32.alloc_uninit(n * W * 4) && big.alloc_uninit(n * std::max(mx_big, 1) * es) && convo.alloc_uninit(n * std::max(mx_conv, 1) * es) &&
@@ -866,27 +1094,7 @@ bool Model::run_layer(int li, int T, int max_kv, const int* d_pos, const int* d_
   if (!rc(k.pk_res32_offset_norm_add(mix.ptr, f32, L.norm1.d.ptr, (float*)x.ptr, xa.ptr, W, T, c.eps, f32, st), "norm1")) return false;
   // ---- feed-forward
   if (a.mlp_kind == 1) {
-    // bf16: gate | up projection with the SwiGLU activation in its epilogue (the library's fused GEMV for <= 4 tokens, its
-    // tensor-core GEMM above; the same rounding points as the two launches they replace, which remain the fallback)
-    bool fused = false;
-    if (!f32 && T <= 4) {
-      pk_b200_gemv_args g{};
-      g.W = (const pk_bf16*)L.gate_up.d.ptr;
-      g.X = (const pk_bf16*)xa.ptr;
-      g.Y[0] = (pk_bf16*)act.ptr;
-      g.seg_rows[0] = a.ff;
-      g.M = a.ff;
-      g.N = T;
-      g.K = W;
-      g.epi = 1;
-      fused = k.pk_b200_gemv_fused(&g, st) == 0;
-    } else if (!f32) {
-      fused = k.pk_b200_gemm_swiglu((const pk_bf16*)L.gate_up.d.ptr, (const pk_bf16*)xa.ptr, (pk_bf16*)act.ptr, a.ff, T, W, st) == 0;
-    }
-    if (!fused) {
-      if (!lin(L.gate_up, xa.ptr, gu.ptr, T)) return false;
-      if (!rc(k.pk_act(gu.ptr, act.ptr, a.ff, T, 0, f32, st), "SwiGLU")) return false;
-    }
+    if (!gated_ff(L, T)) return false;
     if (!lin(L.down, act.ptr, mix.ptr, T)) return false;
     if (!rc(k.pk_res32_offset_norm_add(mix.ptr, f32, L.norm2.d.ptr, (float*)x.ptr, xa.ptr, W, T, c.eps, f32, st), "norm2")) return false;
   } else if (a.mlp_kind == 2) {
@@ -908,6 +1116,30 @@ bool Model::run_layer(int li, int T, int max_kv, const int* d_pos, const int* d_
   if (keep_trail)
     return cu(cudaMemcpyAsync((char*)trail.ptr + (size_t)li * T * W * 4, x.ptr, (size_t)T * W * 4, cudaMemcpyDeviceToDevice, st), "trail copy");
   return true;
+}
+
+// dense gated feed-forward up to its hidden activations: act = f(W_gate xa) * (W_up xa), f SiLU or ReLU.  bf16: gate | up projection with the
+// activation in its epilogue (the library's fused GEMV for <= 4 tokens, its tensor-core GEMM above; the same rounding points as the two
+// launches they replace, which remain the fallback)
+bool Model::gated_ff(const Layer& L, int T) {
+  const LayerCfg& a = L.c;
+  bool fused = false;
+  if (!c.f32 && T <= 4) {
+    pk_b200_gemv_args g{};
+    g.W = (const pk_bf16*)L.gate_up.d.ptr;
+    g.X = (const pk_bf16*)xa.ptr;
+    g.Y[0] = (pk_bf16*)act.ptr;
+    g.seg_rows[0] = a.ff;
+    g.M = a.ff;
+    g.N = T;
+    g.K = c.width;
+    g.epi = a.mlp_act == 1 ? 5 : 1;
+    fused = k.pk_b200_gemv_fused(&g, st) == 0;
+  } else if (!c.f32) {
+    fused = k.pk_b200_gemm_gated((const pk_bf16*)L.gate_up.d.ptr, (const pk_bf16*)xa.ptr, (pk_bf16*)act.ptr, a.ff, T, c.width, a.mlp_act, st) == 0;
+  }
+  if (fused) return true;
+  return lin(L.gate_up, xa.ptr, gu.ptr, T) && rc(k.pk_act(gu.ptr, act.ptr, a.ff, T, a.mlp_act == 1 ? 2 : 0, c.f32, st), "gated activation");
 }
 
 // routed experts of one layer for the tokens in xa: router logits are in zs (block 1) or z (block 0); result in yf (fp32)
@@ -1097,26 +1329,7 @@ bool Model::run_sandwich_layer(int li, int T, int max_kv, const int* M) {
           "mixer result: gate, norm, residual"))
     return false;
   if (a.mlp_kind == 1) {
-    // gate | up projection with the SwiGLU activation in its epilogue where the library has it (as in the sequential block)
-    bool fused = false;
-    if (!f32 && T <= 4) {
-      pk_b200_gemv_args g{};
-      g.W = (const pk_bf16*)L.gate_up.d.ptr;
-      g.X = (const pk_bf16*)xa.ptr;
-      g.Y[0] = (pk_bf16*)act.ptr;
-      g.seg_rows[0] = a.ff;
-      g.M = a.ff;
-      g.N = T;
-      g.K = W;
-      g.epi = 1;
-      fused = k.pk_b200_gemv_fused(&g, st) == 0;
-    } else if (!f32) {
-      fused = k.pk_b200_gemm_swiglu((const pk_bf16*)L.gate_up.d.ptr, (const pk_bf16*)xa.ptr, (pk_bf16*)act.ptr, a.ff, T, W, st) == 0;
-    }
-    if (!fused) {
-      if (!lin(L.gate_up, xa.ptr, gu.ptr, T)) return false;
-      if (!rc(k.pk_act(gu.ptr, act.ptr, a.ff, T, 0, f32, st), "SwiGLU")) return false;
-    }
+    if (!gated_ff(L, T)) return false;
     if (rg && !lin(L.rg2, xa.ptr, rgbuf.ptr, T)) return false;
     if (!lin(L.down, act.ptr, mix.ptr, T)) return false;
     if (!rc(k.pk_res32_gated_gnorm_add(mix.ptr, f32, nullptr, rg ? rgbuf.ptr : nullptr, W, rg ? L.rg2_bias.d.ptr : nullptr, L.norm2b.d.ptr, c.residual_mult,
@@ -1219,6 +1432,116 @@ bool Model::run_prenorm_layer(int li, int T, int max_kv, const int* M, int n) {
   return true;
 }
 
+// One gated delta rule of block 4.  rows: the layer's stacked projection from its q column on (row stride nbig); small: its few-row projections
+// [(a) | b] (row stride nsmall); slot0: S and the convolution's last inputs inside a state slot.  factor * gated normed read-out goes to out.
+bool Model::delta_branch(const Layer& L, const char* rows, int nbig, const float* small, int nsmall, float* slot0, void* out, int ld_out, float factor, int T,
+                         const int* M, int n) {
+  const LayerCfg& a = L.c;
+  const DeltaDims d(a);
+  const int f32 = c.f32;
+  const int *d_slot = M + 3 * T + n, *d_row0 = M + 3 * T + 2 * n, *d_len = M + 3 * T + 3 * n;
+  if (!rc(k.pk_causal_conv(rows, nbig, nullptr, L.conv_w.d.ptr, nullptr, 1, slot0 + (size_t)d.H * d.D * d.V, slot_stride, d_slot, d_row0, d_len, convo.ptr,
+                           d.C, d.C, a.conv, T, n, f32, st),
+          "short convolution"))
+    return false;
+  if (d.rank_a > 0) {
+    if (!rc(k.pk_gemm_strided_f32out(rows + (size_t)(d.C + d.ng) * es, L.a2.d.ptr, (float*)zc.ptr, T, d.H * d.D, d.rank_a, nbig, d.rank_a, (long)d.H * d.D, 1,
+                                     0, 0, 0, f32, st),
+            "decay projection"))
+      return false;
+    if (!rc(k.pk_channel_delta_seq(convo.ptr, d.C, 0, d.nq, d.nq + d.nk, small, nsmall, 0, (const float*)zc.ptr, d.H * d.D, (const float*)L.p0_32.ptr,
+                                   (const float*)L.p1_32.ptr, slot0, slot_stride, d_slot, d_row0, d_len, (float*)orec.ptr, d.H, d.G, d.D, d.V, n, f32, st),
+            "gated delta rule"))
+      return false;
+  } else if (!rc(k.pk_gated_delta_seq(convo.ptr, d.C, 0, d.nq, d.nq + d.nk, small, nsmall, 0, d.H, (const float*)L.p0_32.ptr, (const float*)L.p1_32.ptr, slot0,
+                                      slot_stride, d_slot, d_row0, d_len, (float*)orec.ptr, d.H, d.G, d.D, d.V, n, f32, st),
+                 "gated delta rule")) {
+    return false;
+  }
+  const void* gate = rows;  // silu(W_g h): a slice of the projection
+  int gate_ld = nbig, gate_off = d.C, act_kind = 0;
+  if (d.rank_g > 0) {
+    if (!rc(k.pk_gemm_strided(rows + (size_t)(d.C + d.ng + d.rank_a) * es, L.g2.d.ptr, gbuf.ptr, nullptr, T, d.nv, d.rank_g, nbig, 1, d.rank_g, d.nv, 1, 0, 0, 0,
+                              0, 0, f32, st),
+            "read-out gate projection"))
+      return false;
+    gate = gbuf.ptr;
+    gate_ld = d.nv;
+    gate_off = 0;
+    act_kind = 1;
+  }
+  return rc(k.pk_head_norm_gate_ex((const float*)orec.ptr, nullptr, L.hnorm.d.ptr, 0, gate, gate_ld, gate_off, out, ld_out, factor, T, d.H, d.V, c.eps, act_kind,
+                                   f32, st),
+            "read-out norm");
+}
+
+// Block over parallel residual streams: on entry xa (and h32, unrounded) hold this layer's normed input; on exit x holds the streams after the
+// layer and xa / h32 the next layer's normed input (nothing after the last layer).
+bool Model::run_streams_layer(int li, int T, int max_kv, const int* M, int n) {
+  Layer& L = layers[li];
+  const LayerCfg& a = L.c;
+  const int W = c.width, f32 = c.f32, S = n_streams;
+  const int *d_pos = M + T, *d_req = M + 2 * T, *d_poff = M + 3 * T, *d_slot = M + 3 * T + n, *d_row0 = M + 3 * T + 2 * n, *d_len = M + 3 * T + 3 * n;
+  const int* d_pages = M + pages_at;
+  float* slot0 = (float*)state.ptr + L.state_off;
+  const Layer* next = li + 1 < c.n_layers ? &layers[li + 1] : nullptr;
+  const auto coef = [&](const Layer& l, int q, int j) { return (const float*)(c.streams > 0 ? l.hc32[q][j].ptr : one32.ptr); };
+  // y (in mix) back to the streams, and the read + norm of the sublayer that follows
+  const auto write_streams = [&](int q, const char* what) {
+    const bool ff_next = q == 0 && a.mlp_kind;
+    const float* w_in = ff_next ? coef(L, 1, 0) : next ? coef(*next, 0, 0) : nullptr;
+    const void* w_norm = ff_next ? L.norm2.d.ptr : next ? next->norm1.d.ptr : nullptr;
+    return rc(k.pk_res32_streams_step(mix.ptr, coef(L, q, 2), coef(L, q, 1), w_in, (float*)x.ptr, w_norm, xa.ptr, (float*)h32.ptr, W, S, c.eps, T, f32, st), what);
+  };
+  // ---- mixer
+  if (!lin(L.qkv, xa.ptr, big.ptr, T)) return false;
+  if (a.mixer_kind == 5) {
+    const int C = a.lru_width, nb = a.lru_blocks, b = C / nb;
+    if (!rc(k.pk_causal_conv(big.ptr, 2 * C, L.conv_in_b.d.ptr, L.conv_w.d.ptr, L.conv_b.d.ptr, 0, slot0 + C, slot_stride, d_slot, d_row0, d_len, convo.ptr, C, C,
+                             a.conv, T, n, f32, st),
+            "short convolution"))
+      return false;
+    if (!rc(k.pk_gemm_strided_f32out(convo.ptr, L.gates.d.ptr, (float*)zc.ptr, T, 2 * b, b, C, b, 2 * C, nb, b, (long)2 * b * b, 2 * b, f32, st),
+            "block-diagonal gates"))
+      return false;
+    if (!rc(k.pk_lru_seq(convo.ptr, C, (const float*)zc.ptr, 2 * C, (const float*)L.p1_32.ptr, (const float*)L.p2_32.ptr, (const float*)L.p0_32.ptr, a.lru_rate, nb,
+                         (const char*)big.ptr + (size_t)C * es, 2 * C, L.qkv_bias.d.ptr, slot0, slot_stride, d_slot, d_row0, d_len, ao.ptr, C, C, T, n, f32, st),
+            "linear recurrent unit"))
+      return false;
+  } else {
+    const DeltaDims d(a);
+    const bool two = a.mixer_kind == 6;
+    const int H = two ? a.heads : 0, G = a.kv_heads, r0 = two ? H * a.dim + G * (a.dim + a.vdim) : 0;
+    const int nbig = r0 + d.big(), nsmall = H + d.small(), wo = two ? H * a.vdim : 0, ld = wo + d.nv;
+    if (!skinny(L.small, (float*)zs.ptr, T, "few-row projections", (const float*)h32.ptr)) return false;
+    if (two) {
+      char* pool_base = (char*)cache.ptr + (size_t)L.cache_off * es;
+      if (!rc(k.pk_gqa_rope_append_ex(big.ptr, nbig, nullptr, d_pos, d_req, d_poff, d_pages, q.ptr, pool_base, page_stride, c.page_size, H, G, a.dim, a.vdim,
+                                      a.rot_dims, a.rot_interleaved, (const float*)L.freq.ptr, L.mag, 0.f, T, f32, st),
+              "rotation + cache append"))
+        return false;
+      if (!rc(k.pk_gqa_mixed_attention(q.ptr, pool_base, L.talk.d.ptr, (const float*)L.p2_32.ptr, (const float*)zs.ptr, nsmall, d_pos, d_req, d_poff, d_pages,
+                                       ao.ptr, ld, a.left_scale, page_stride, c.page_size, T, H, G, a.dim, a.vdim, a.scale, max_kv, f32, st),
+              "attention"))
+        return false;
+    }
+    if (!delta_branch(L, (const char*)big.ptr + (size_t)r0 * es, nbig, (const float*)zs.ptr + H, nsmall, slot0, (char*)ao.ptr + (size_t)wo * es, ld,
+                      two ? a.right_scale : 1.f, T, M, n))
+      return false;
+  }
+  // the branches of mixer 6 lie side by side in ao, as their output projections do in o: one product projects and sums them
+  if (!lin(L.o, ao.ptr, mix.ptr, T)) return false;
+  if (!write_streams(0, "mixer result: streams, next norm")) return false;
+  // ---- feed-forward
+  if (a.mlp_kind == 1) {
+    if (!gated_ff(L, T) || !lin(L.down, act.ptr, mix.ptr, T)) return false;
+    if (!write_streams(1, "feed-forward result: streams, next norm")) return false;
+  }
+  if (keep_trail)
+    return rc(k.pk_res32_streams_rows((const float*)x.ptr, nullptr, nullptr, nullptr, (float*)trail.ptr + (size_t)li * T * W, W, S, c.eps, T, f32, st), "trail");
+  return true;
+}
+
 // everything between the metadata upload and the final synchronisation: launches only (no allocation, no synchronisation)
 bool Model::forward(int T, int n, int n_rows, int max_kv, int want_sample) {
   const int* M = meta_d.i32();
@@ -1229,6 +1552,13 @@ bool Model::forward(int T, int n, int n_rows, int max_kv, int want_sample) {
     if (!rc(k.pk_res32_embed(embed.d.ptr, d_tok, (float*)x.ptr, xa.ptr, W, T, c.f32, st), "embedding")) return false;
     for (int li = 0; li < c.n_layers; ++li)
       if (!run_layer(li, T, max_kv, d_pos, d_req, d_poff, d_pages)) return false;
+  } else if (c.block_kind == 4) {
+    if (!rc(k.pk_res32_streams_embed(embed.d.ptr, d_tok, (const float*)(c.streams > 0 ? layers[0].hc32[0][0].ptr : one32.ptr), (float*)x.ptr,
+                                     layers[0].norm1.d.ptr, xa.ptr, (float*)h32.ptr, W, n_streams, c.eps, T, c.f32, st),
+            "embedding"))
+      return false;
+    for (int li = 0; li < c.n_layers; ++li)
+      if (!run_streams_layer(li, T, max_kv, M, n)) return false;
   } else if (c.block_kind == 3) {
     if (!rc(k.pk_res32_embed_scaled_norm(embed.d.ptr, d_tok, c.embed_scale, (float*)x.ptr, layers[layers[0].wsrc].norm1.d.ptr, xa.ptr, (float*)h32.ptr, W, c.eps,
                                          T, c.f32, st),
@@ -1261,6 +1591,9 @@ bool Model::forward(int T, int n, int n_rows, int max_kv, int want_sample) {
   if (n_rows > 0) {
     if (c.block_kind == 0) {
       if (!rc(k.pk_res32_offset_norm_rows((const float*)x.ptr, d_rows, final_norm.d.ptr, xr.ptr, W, n_rows, c.eps, c.f32, st), "final norm")) return false;
+    } else if (c.block_kind == 4) {
+      if (!rc(k.pk_res32_streams_rows((const float*)x.ptr, d_rows, final_norm.d.ptr, xr.ptr, nullptr, W, n_streams, c.eps, n_rows, c.f32, st), "final norm"))
+        return false;
     } else if (c.block_kind >= 2) {  // the pre-norm block form's last norm is the same norm with one group
       if (!rc(k.pk_res32_gnorm_rows((const float*)x.ptr, d_rows, final_norm.d.ptr, xr.ptr, W, c.block_kind == 2 ? c.norm_groups : 1, c.eps, n_rows, c.f32, st),
               "final norm"))

@@ -1,6 +1,9 @@
 // Recurrent mixers with a matrix state per head, for ragged batches whose requests keep their state in numbered slots:
-//   * short causal convolution + SiLU over time per channel, with the last taps - 1 inputs of every request as state;
+//   * short causal convolution (+ SiLU) over time per channel, with the last taps - 1 inputs of every request as state;
 //   * gated delta rule:   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q        (q, k unit vectors per head)
+//     with one decay g per head, or one per head and key channel (g then scales the rows of S);
+//   * real-gated linear recurrent unit, one scalar per channel:  S <- a S + sqrt(1 - a^2) i u,  log a = -rate r softplus(lam),
+//     r and i logistic gates;  the read-out is multiplied by a GELU branch.  Affine maps compose, so a portion is scanned in parallel.
 //   * xLSTM matrix memory: m' = max(f + m, i);  S <- e^(f + m - m') S + e^(i - m') k v^T;  n likewise with k alone;
 //                          o = S^T q / (max(|n . q|, e^(-m')) + 1e-6)        (i, f soft-capped log gates, m starts at 0)
 //     slot layout: S [H][dim][vdim], n [H][dim], m [H][vdim + 1] (every column keeps its own copy of the running maximum)
@@ -16,6 +19,8 @@
 // threads first bring q, k, v and the gate inputs into shared memory and turn them into unit vectors / gates.  The matrix
 // memory's normaliser n is one more column with value 1.  Latency-bound per token (48 FMAs and two shuffle reductions per
 // thread, one warp per scheduler).
+#include <algorithm>
+
 #include "common.cuh"
 #include "typed.cuh"
 
@@ -25,39 +30,60 @@ __device__ __forceinline__ float sigmoidf_(float z) { return 1.f / (1.f + expf(-
 __device__ __forceinline__ float softplusf_(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 __device__ __forceinline__ float logsigmoidf_(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
-// y[t][c] = silu(bias[c] + sum_j w[c][j] * x[t - (taps-1-j)][c]) (bias may be null); inputs before this step's rows come from the slot's state
-// [taps-1][C] (oldest first; zero for a new request).  in / out may have different row strides; out may alias nothing of in.
-template <typename E>
-__global__ void causal_conv_silu_kernel(const E* __restrict__ in, int ld_in, const E* __restrict__ w, const E* __restrict__ bias, const float* __restrict__ state, long slot_stride,
-                                        const int* __restrict__ req, const int* __restrict__ slot, const int* __restrict__ row0, E* __restrict__ out,
-                                        int ld_out, int C, int taps, long total) {
+// y[t][c] = act(bias[c] + sum_j w[c][j] * x[t - (taps-1-j)][c]),  x = in + in_bias (either bias may be null; act 0: none, 1: SiLU).  Inputs
+// before this step's rows come from the slot's state [taps-1][C] (oldest first; zero for a new request), which afterwards holds the last
+// taps - 1 inputs (old ones move up when the portion was shorter).  One thread per (channel, `gs` consecutive tokens of one entry) with
+// gs >= taps - 1: an entry's first group is the only one that reads the old state, so the same thread may replace it when it is done.
+// TAPS > 0: the number of taps at compile time (the window slides through registers); 0: any number.
+template <typename E, int TAPS>
+__global__ void causal_conv_kernel(const E* __restrict__ in, int ld_in, const E* __restrict__ in_bias, const E* __restrict__ w, const E* __restrict__ bias,
+                                   float* __restrict__ state, long slot_stride, const int* __restrict__ slot, const int* __restrict__ row0,
+                                   const int* __restrict__ len, E* __restrict__ out, int ld_out, int C, int taps_any, int act, int entries, int gs) {
   pdl_wait();
   pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
-  for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x) {
-    const int t = (int)(i / C), c = (int)(i % C), e = req[t], off = t - row0[e];
-    const float* st = state + (size_t)slot[e] * slot_stride;
-    float acc = bias ? to_f(bias[c]) : 0.f;
-    for (int j = 0; j < taps; ++j) {
-      const int back = taps - 1 - j;
-      const float x = off - back >= 0 ? to_f(in[(size_t)(t - back) * ld_in + c]) : st[(size_t)(taps - 1 + off - back) * C + c];
-      acc = fmaf(to_f(w[(size_t)c * taps + j]), x, acc);
-    }
-    out[(size_t)t * ld_out + c] = from_f<E>(acc / (1.f + expf(-acc)));
+  const int taps = TAPS > 0 ? TAPS : taps_any;
+  int grp = blockIdx.y, e = 0;
+  for (; e < entries; ++e) {  // the entry this group of tokens belongs to
+    const int ng = (len[e] + gs - 1) / gs;
+    if (grp < ng) break;
+    grp -= ng;
   }
-}
-
-// after the step: the slot keeps the last taps - 1 inputs (old ones move up when the portion was shorter)
-template <typename E>
-__global__ void conv_state_update_kernel(const E* __restrict__ in, int ld_in, float* __restrict__ state, long slot_stride, const int* __restrict__ slot,
-                                         const int* __restrict__ row0, const int* __restrict__ len, int C, int taps) {
-  pdl_wait();
-  pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
-  const int e = blockIdx.y, n = len[e], r0 = row0[e];
-  float* st = state + (size_t)slot[e] * slot_stride;
-  for (int c = blockIdx.x * blockDim.x + threadIdx.x; c < C; c += gridDim.x * blockDim.x)
-    for (int s = 0; s < taps - 1; ++s) {
-      const int o = n - (taps - 1) + s;
-      st[(size_t)s * C + c] = o >= 0 ? to_f(in[(size_t)(r0 + o) * ld_in + c]) : st[(size_t)(s + n) * C + c];
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (e == entries || c >= C) return;
+  const int n = len[e], o0 = grp * gs, o1 = min(n, o0 + gs);
+  const E* x = in + (size_t)row0[e] * ld_in + c;
+  E* y = out + (size_t)row0[e] * ld_out + c;
+  float* st = state + (size_t)slot[e] * slot_stride + c;
+  const float ib = in_bias ? to_f(in_bias[c]) : 0.f, b0 = bias ? to_f(bias[c]) : 0.f;
+  auto input = [&](int o) { return o >= 0 ? to_f(x[(size_t)o * ld_in]) + ib : st[(size_t)(taps - 1 + o) * C]; };
+  auto finish = [&](float v) { return from_f<E>(act ? v / (1.f + expf(-v)) : v); };
+  if constexpr (TAPS > 0) {
+    float wr[TAPS], h[TAPS];  // h[j]: input of taps - 1 - j tokens ago
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) wr[j] = to_f(w[(size_t)c * TAPS + j]);
+#pragma unroll
+    for (int j = 1; j < TAPS; ++j) h[j] = input(o0 - TAPS + j);
+#pragma unroll 4
+    for (int o = o0; o < o1; ++o) {
+#pragma unroll
+      for (int j = 0; j + 1 < TAPS; ++j) h[j] = h[j + 1];
+      h[TAPS - 1] = to_f(x[(size_t)o * ld_in]) + ib;
+      float acc = b0;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) acc = fmaf(wr[j], h[j], acc);
+      y[(size_t)o * ld_out] = finish(acc);
+    }
+  } else {
+    for (int o = o0; o < o1; ++o) {
+      float acc = b0;
+      for (int j = 0; j < taps; ++j) acc = fmaf(to_f(w[(size_t)c * taps + j]), input(o - (taps - 1) + j), acc);
+      y[(size_t)o * ld_out] = finish(acc);
+    }
+  }
+  if (grp == 0)
+    for (int i = 0; i < taps - 1; ++i) {  // ascending: an old entry is read before its place is written
+      const int o = n - (taps - 1) + i;
+      st[(size_t)i * C] = o >= 0 ? to_f(x[(size_t)o * ld_in]) + ib : st[(size_t)(i + n) * C];
     }
 }
 
@@ -78,19 +104,24 @@ struct SeqArgs {
   const void* dt;      // state space: [tokens, ld_dt] element type, step-size projection of head h at dt_off + h
   int ld_dt, dt_off;
   const float* p2;     // state space: skip weight D [H]  (p0 = A_log, p1 = dt_bias)
+  const float* zc;     // delta rule with a decay per key channel: [tokens, ld_zc], pre-activation of (head, channel) at h * dim + d; p1 = dt_bias [H * dim]
+  int ld_zc;
 };
 
 // MODE 0: gated delta rule.  MODE 1: xLSTM matrix memory.  MODE 2: state-space duality (q = C, k = B, v = x; dim = state size).
+// MODE 3: gated delta rule with a decay per key channel (a third vector per token beside k and q).
 // Thread layout: KS = DK / 16 neighbouring lanes share one state column, each holding 16 of its DK entries in registers
 // (entry (m * KS + ks) * 4 + e for m < 4, e < 4, so that the lanes' 16-byte reads of k / q from shared memory fall on
 // consecutive banks); the two dot products per token are finished with log2(KS) shuffles.  128 / KS columns per CTA; the
 // matrix memory's normaliser column rides in one more warp of the head's first CTA.
 template <typename E, int DK, int MODE>
 __global__ void __launch_bounds__(160) recurrent_seq_kernel(SeqArgs a) {
-  constexpr int KS = DK / 16, COLS = 128 / KS, TB = DK <= 128 ? 32 : 16, NS = 16;  // NS state entries per thread
+  constexpr bool DELTA = MODE == 0 || MODE == 3;
+  constexpr int KS = DK / 16, COLS = 128 / KS, TB = (DK <= 128 ? 32 : 16) / (MODE == 3 && DK >= 128 ? 2 : 1), NS = 16;  // NS state entries per thread
   __shared__ __align__(16) float ks[TB][DK];
   __shared__ __align__(16) float qs[TB][DK];
   __shared__ float vs[TB][COLS];
+  __shared__ __align__(16) float gc[MODE == 3 ? TB : 1][MODE == 3 ? DK : 4];  // MODE 3: decay per key channel
   __shared__ float g0[TB], g1[TB];  // delta: decay, write strength;  memory: log forget gate, log input gate
   pdl_wait();
   pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
@@ -171,8 +202,10 @@ __global__ void __launch_bounds__(160) recurrent_seq_kernel(SeqArgs a) {
       }
     } else if (tid < nb) {
       const size_t row = (size_t)(r0 + b0 + tid);
-      const float za = a.z[row * a.ldz + a.za_off + h], zb = a.z[row * a.ldz + a.zb_off + h];
-      if (MODE == 0) {  // za: decay projection, zb: write-strength projection
+      const float za = MODE == 3 ? 0.f : a.z[row * a.ldz + a.za_off + h], zb = a.z[row * a.ldz + a.zb_off + h];
+      if (MODE == 3) {
+        g1[tid] = sigmoidf_(zb);
+      } else if (MODE == 0) {  // za: decay projection, zb: write-strength projection
         g0[tid] = expf(-expf(a.p0[h]) * softplusf_(za + a.p1[h]));
         g1[tid] = sigmoidf_(zb);
       } else {  // za: forget gate, zb: input gate
@@ -180,11 +213,19 @@ __global__ void __launch_bounds__(160) recurrent_seq_kernel(SeqArgs a) {
         g1[tid] = a.cap * tanhf((zb + a.p0[h]) / a.cap);
       }
     }
+    if constexpr (MODE == 3) {
+      const float rate = expf(a.p0[h]);
+#pragma unroll 4
+      for (int i = tid; i < nb * DK; i += blockDim.x) {
+        const int tt = i / DK, d = i % DK;
+        gc[tt][d] = d < dim ? expf(-rate * softplusf_(a.zc[(size_t)(r0 + b0 + tt) * a.ld_zc + h * dim + d] + a.p1[h * dim + d])) : 1.f;
+      }
+    }
     __syncthreads();
     // 2. unit vectors (delta rule) and the query's scale
     for (int tt = warp; MODE != 2 && tt < nb; tt += nw) {
       float qf = qscale, kf = 1.f;
-      if (MODE == 0) {
+      if (DELTA) {
         float qq = 0.f, kk = 0.f;
         for (int i = lane; i < DK; i += 32) {
           qq = fmaf(qs[tt][i], qs[tt][i], qq);
@@ -197,7 +238,7 @@ __global__ void __launch_bounds__(160) recurrent_seq_kernel(SeqArgs a) {
       }
       for (int i = lane; i < DK; i += 32) {
         qs[tt][i] *= qf;
-        if (MODE == 0) ks[tt][i] *= kf;
+        if (DELTA) ks[tt][i] *= kf;
       }
     }
     __syncthreads();
@@ -210,16 +251,18 @@ __global__ void __launch_bounds__(160) recurrent_seq_kernel(SeqArgs a) {
       const float4* k4p = reinterpret_cast<const float4*>(&ks[tt][0]) + ksi;
       const float4* q4p = reinterpret_cast<const float4*>(&qs[tt][0]) + ksi;
       float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
-      if (MODE == 0) {
-        const float g = g0[tt], beta = g1[tt];
+      if (DELTA) {
+        const float g = MODE == 0 ? g0[tt] : 1.f, beta = g1[tt];
+        const float4* g4p = reinterpret_cast<const float4*>(&gc[MODE == 3 ? tt : 0][0]) + ksi;
         float c0 = 0.f, c1 = 0.f, c2 = 0.f, c3 = 0.f;
 #pragma unroll
         for (int mi = 0; mi < NS / 4; ++mi) {
           const float4 k4 = k4p[mi * KS];
-          S[mi * 4] *= g;
-          S[mi * 4 + 1] *= g;
-          S[mi * 4 + 2] *= g;
-          S[mi * 4 + 3] *= g;
+          const float4 g4 = MODE == 3 ? g4p[mi * KS] : make_float4(g, g, g, g);
+          S[mi * 4] *= g4.x;
+          S[mi * 4 + 1] *= g4.y;
+          S[mi * 4 + 2] *= g4.z;
+          S[mi * 4 + 3] *= g4.w;
           c0 = fmaf(S[mi * 4], k4.x, c0);
           c1 = fmaf(S[mi * 4 + 1], k4.y, c1);
           c2 = fmaf(S[mi * 4 + 2], k4.z, c2);
@@ -305,12 +348,12 @@ __global__ void __launch_bounds__(160) recurrent_seq_kernel(SeqArgs a) {
 }
 
 // out[t, h, j] = E( (o[t,h,j] / den[t,h]) / sqrt(mean_j(.^2) + eps) * w[h * w_stride + j] * act(gate[t, gate_off + h*vdim + j]) )
-// act 0: silu, 1: logistic.  act 2: the silu gate comes BEFORE the norm, out = rms_norm(o * silu(gate)) * w.  den may be null.
+// times `factor`, rows of stride ld_out.  act 0: silu, 1: logistic.  act 2: the silu gate comes BEFORE the norm, out = rms_norm(o * silu(gate)) * w.  den may be null.
 // One warp per (token, head); "head" may be any equal part of the row (norm groups).
 template <typename E>
 __global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ den, const E* __restrict__ w, int w_stride,
-                                      const E* __restrict__ gate, int ld_gate, int gate_off, E* __restrict__ out, int H, int vdim, float eps, int act,
-                                      long pairs) {
+                                      const E* __restrict__ gate, int ld_gate, int gate_off, E* __restrict__ out, int ld_out, float factor, int H, int vdim,
+                                      float eps, int act, long pairs) {
   pdl_wait();
   pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
   const int lane = threadIdx.x & 31;
@@ -334,15 +377,16 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* 
     const float v = den ? orow[j] / den[pr] : orow[j];
     const float gz = to_f(gate[(size_t)t * ld_gate + gate_off + h * vdim + j]);
     const float ga = act == 1 ? 1.f / (1.f + expf(-gz)) : gz / (1.f + expf(-gz));
-    out[pr * vdim + j] = from_f<E>(act == 2 ? (v * ga) * inv * to_f(w[(size_t)h * w_stride + j]) : v * inv * to_f(w[(size_t)h * w_stride + j]) * ga);
+    out[(size_t)t * ld_out + h * vdim + j] =
+        from_f<E>(factor * (act == 2 ? (v * ga) * inv * to_f(w[(size_t)h * w_stride + j]) : v * inv * to_f(w[(size_t)h * w_stride + j]) * ga));
   }
 }
 
 // the same for few (token, head) pairs of many entries each (a decode step with wide norm groups): one CTA per pair
 template <typename E>
 __global__ void head_norm_gate_wide_kernel(const float* __restrict__ o, const float* __restrict__ den, const E* __restrict__ w, int w_stride,
-                                           const E* __restrict__ gate, int ld_gate, int gate_off, E* __restrict__ out, int H, int vdim, float eps,
-                                           int act) {
+                                           const E* __restrict__ gate, int ld_gate, int gate_off, E* __restrict__ out, int ld_out, float factor, int H,
+                                           int vdim, float eps, int act) {
   __shared__ float red[33];
   pdl_wait();
   pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
@@ -369,8 +413,122 @@ __global__ void head_norm_gate_wide_kernel(const float* __restrict__ o, const fl
 #pragma unroll
   for (int u = 0; u < 4; ++u) {
     const int j = threadIdx.x + u * blockDim.x;
-    if (j < vdim) out[pr * vdim + j] = from_f<E>(act == 2 ? v[u] * inv * to_f(w[(size_t)h * w_stride + j]) : v[u] * inv * to_f(w[(size_t)h * w_stride + j]) * ga[u]);
+    if (j < vdim)
+      out[(size_t)t * ld_out + h * vdim + j] =
+          from_f<E>(factor * (act == 2 ? v[u] * inv * to_f(w[(size_t)h * w_stride + j]) : v[u] * inv * to_f(w[(size_t)h * w_stride + j]) * ga[u]));
   }
+}
+
+// ---- real-gated linear recurrent unit.  z holds the gates' pre-activations without bias: block b of n channels has r at b * 2n + j and i
+// at b * 2n + n + j.  out = E(S * gelu(y + y_bias)), gelu in its tanh form.
+struct LruArgs {
+  const void *u, *y, *y_bias;  // [tokens, ld_u] convolved input, [tokens, ld_y] raw branch, its bias [C] or null
+  const float *z, *r_bias, *i_bias, *lam;
+  float* state;                // [C] per slot
+  const int *slot, *row0, *len;
+  void* out;
+  long slot_stride;
+  int ld_u, ld_y, ldz, ld_out, C, n;  // n: channels of a gate block
+  float rate;
+};
+__device__ __forceinline__ float gelu_tanh_(float z) {
+  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));  // sqrt(2 / pi)
+}
+// the affine map S -> a S + b of one token
+__device__ __forceinline__ float2 lru_map(float u, float zr, float zi, float neg_rate) {
+  const float la = neg_rate * sigmoidf_(zr);
+  return make_float2(expf(la), sqrtf(fmaxf(-expm1f(2.f * la), 0.f)) * sigmoidf_(zi) * u);  // 1 - a^2 = -(e^(2 log a) - 1)
+}
+
+// few tokens per entry: one thread per channel, token by token
+template <typename E>
+__global__ void lru_step_kernel(LruArgs a) {
+  pdl_wait();
+  pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
+  const int c = blockIdx.x * blockDim.x + threadIdx.x, e = blockIdx.y;
+  if (c >= a.C) return;
+  const int n = a.len[e], r0 = a.row0[e], zo = (c / a.n) * 2 * a.n + c % a.n;
+  float* st = a.state + (size_t)a.slot[e] * a.slot_stride + c;
+  const float rb = a.r_bias[c], ib = a.i_bias[c], neg = -a.rate * softplusf_(a.lam[c]), yb = a.y_bias ? to_f(static_cast<const E*>(a.y_bias)[c]) : 0.f;
+  float S = st[0];
+#pragma unroll 2
+  for (int o = 0; o < n; ++o) {
+    const size_t t = (size_t)(r0 + o);
+    const float2 m = lru_map(to_f(static_cast<const E*>(a.u)[t * a.ld_u + c]), a.z[t * a.ldz + zo] + rb, a.z[t * a.ldz + zo + a.n] + ib, neg);
+    S = fmaf(m.x, S, m.y);
+    static_cast<E*>(a.out)[t * a.ld_out + c] = from_f<E>(S * gelu_tanh_(to_f(static_cast<const E*>(a.y)[t * a.ld_y + c]) + yb));
+  }
+  st[0] = S;
+}
+
+// a prompt portion: CTA = 16 channels of one entry, 32 groups of TPT consecutive tokens at a time.  Every thread composes the maps of its
+// tokens, one warp per channel scans the 32 composed maps with shuffles, and every thread then runs its tokens from its start state.
+template <typename E, int TPT>
+__global__ void __launch_bounds__(512) lru_scan_kernel(LruArgs a) {
+  constexpr int CH = 16, NG = 32;
+  __shared__ float sa[NG][CH + 1], sb[NG][CH + 1], s_in[NG][CH + 1], carry[CH];
+  pdl_wait();
+  pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
+  const int tid = threadIdx.x, ch = tid % CH, tg = tid / CH, c = blockIdx.x * CH + ch, e = blockIdx.y, lane = tid & 31, warp = tid >> 5;
+  const bool on = c < a.C;
+  const int n = a.len[e], r0 = a.row0[e], zo = on ? (c / a.n) * 2 * a.n + c % a.n : 0;
+  float* st = a.state + (size_t)a.slot[e] * a.slot_stride;
+  float rb = 0.f, ib = 0.f, neg = 0.f, yb = 0.f;
+  if (on) {
+    rb = a.r_bias[c];
+    ib = a.i_bias[c];
+    neg = -a.rate * softplusf_(a.lam[c]);
+    yb = a.y_bias ? to_f(static_cast<const E*>(a.y_bias)[c]) : 0.f;
+  }
+  if (tid < CH) carry[tid] = blockIdx.x * CH + tid < a.C ? st[blockIdx.x * CH + tid] : 0.f;
+  for (int b0 = 0; b0 < n; b0 += NG * TPT) {
+    float2 m[TPT];
+    float A = 1.f, B = 0.f;
+#pragma unroll
+    for (int k = 0; k < TPT; ++k) {
+      const int o = b0 + tg * TPT + k;
+      m[k] = make_float2(1.f, 0.f);
+      if (on && o < n) {
+        const size_t t = (size_t)(r0 + o);
+        m[k] = lru_map(to_f(static_cast<const E*>(a.u)[t * a.ld_u + c]), a.z[t * a.ldz + zo] + rb, a.z[t * a.ldz + zo + a.n] + ib, neg);
+      }
+      A *= m[k].x;
+      B = fmaf(m[k].x, B, m[k].y);
+    }
+    sa[tg][ch] = A;
+    sb[tg][ch] = B;
+    __syncthreads();
+    {  // warp w: channel w, lane = token group; inclusive scan of the composed maps
+      float xa = sa[lane][warp], xb = sb[lane][warp];
+#pragma unroll
+      for (int d = 1; d < NG; d <<= 1) {
+        const float pa = __shfl_up_sync(0xffffffffu, xa, d), pb = __shfl_up_sync(0xffffffffu, xb, d);
+        if (lane >= d) {
+          xb = fmaf(xa, pb, xb);
+          xa *= pa;
+        }
+      }
+      const float s0 = carry[warp];
+      float ea = __shfl_up_sync(0xffffffffu, xa, 1), eb = __shfl_up_sync(0xffffffffu, xb, 1);
+      if (lane == 0) ea = 1.f, eb = 0.f;
+      s_in[lane][warp] = fmaf(ea, s0, eb);
+      __syncwarp();  // every lane has read the old carry
+      if (lane == NG - 1) carry[warp] = fmaf(xa, s0, xb);
+    }
+    __syncthreads();
+    float S = s_in[tg][ch];
+#pragma unroll
+    for (int k = 0; k < TPT; ++k) {
+      const int o = b0 + tg * TPT + k;
+      S = fmaf(m[k].x, S, m[k].y);
+      if (on && o < n) {
+        const size_t t = (size_t)(r0 + o);
+        static_cast<E*>(a.out)[t * a.ld_out + c] = from_f<E>(S * gelu_tanh_(to_f(static_cast<const E*>(a.y)[t * a.ld_y + c]) + yb));
+      }
+    }
+  }
+  __syncthreads();
+  if (tid < CH && blockIdx.x * CH + tid < a.C) st[blockIdx.x * CH + tid] = carry[tid];
 }
 
 template <typename E, int MODE>
@@ -386,8 +544,6 @@ static int launch_seq(const SeqArgs& a, int entries, cudaStream_t st) {
   return (int)cudaGetLastError();
 }
 
-static inline int grid_for(long n, int block) { return (int)std::min<long>((n + block - 1) / block, 148L * 16); }
-
 }  // namespace pk
 
 using namespace pk;
@@ -401,19 +557,29 @@ extern "C" int pk_causal_conv_silu(const void* in, int ld_in, const void* w, flo
 extern "C" int pk_causal_conv_silu_bias(const void* in, int ld_in, const void* w, const void* bias, float* state, long slot_stride, const int* req,
                                         const int* slot, const int* row0, const int* len, void* out, int ld_out, int channels, int taps, int tokens,
                                         int entries, int f32, pk_stream st) {
-  if (!in || !w || !state || !req || !slot || !row0 || !len || !out || channels <= 0 || taps <= 0 || tokens <= 0 || entries <= 0) return -1;
-  const long total = (long)tokens * channels;
-  if (f32)
-    launch(causal_conv_silu_kernel<float>, dim3(grid_for(total, 256)), dim3(256), 0, st, true, (const float*)in, ld_in, (const float*)w, (const float*)bias,
-           (const float*)state, slot_stride, req, slot, row0, (float*)out, ld_out, channels, taps, total);
-  else
-    launch(causal_conv_silu_kernel<bf16>, dim3(grid_for(total, 256)), dim3(256), 0, st, true, (const bf16*)in, ld_in, (const bf16*)w, (const bf16*)bias,
-           (const float*)state, slot_stride, req, slot, row0, (bf16*)out, ld_out, channels, taps, total);
-  if (taps > 1) {
-    const dim3 g((channels + 255) / 256, entries);
-    if (f32) launch(conv_state_update_kernel<float>, g, dim3(256), 0, st, true, (const float*)in, ld_in, state, slot_stride, slot, row0, len, channels, taps);
-    else launch(conv_state_update_kernel<bf16>, g, dim3(256), 0, st, true, (const bf16*)in, ld_in, state, slot_stride, slot, row0, len, channels, taps);
+  if (!req) return -1;
+  return pk_causal_conv(in, ld_in, nullptr, w, bias, 1, state, slot_stride, slot, row0, len, out, ld_out, channels, taps, tokens, entries, f32, st);
+}
+
+extern "C" int pk_causal_conv(const void* in, int ld_in, const void* in_bias, const void* w, const void* bias, int act, float* state, long slot_stride,
+                              const int* slot, const int* row0, const int* len, void* out, int ld_out, int channels, int taps, int tokens, int entries,
+                              int f32, pk_stream st) {
+  if (!in || !w || !state || !slot || !row0 || !len || !out || channels <= 0 || taps <= 0 || tokens <= 0 || entries <= 0 || act < 0 || act > 1) return -1;
+  const int gs = std::max(8, taps - 1);  // tokens per group; an entry has at most one ragged group
+  const int threads = channels >= 128 * 148 || tokens > 256 ? 128 : 64;
+  const dim3 g((channels + threads - 1) / threads, tokens / gs + entries);
+  if (g.y > 65535) return -2;
+#define PK_CONV(E, TAPS)                                                                                                                      \
+  launch(causal_conv_kernel<E, TAPS>, g, dim3(threads), 0, st, true, (const E*)in, ld_in, (const E*)in_bias, (const E*)w, (const E*)bias, state, \
+         slot_stride, slot, row0, len, (E*)out, ld_out, channels, taps, act, entries, gs)
+  if (f32) {
+    if (taps == 4) PK_CONV(float, 4);
+    else PK_CONV(float, 0);
+  } else {
+    if (taps == 4) PK_CONV(bf16, 4);
+    else PK_CONV(bf16, 0);
   }
+#undef PK_CONV
   return (int)cudaGetLastError();
 }
 
@@ -431,6 +597,16 @@ extern "C" int pk_gated_delta_seq(const void* qkv, int ld, int q_off, int k_off,
   return f32 ? launch_seq<float, 0>(a, entries, st) : launch_seq<bf16, 0>(a, entries, st);
 }
 
+extern "C" int pk_channel_delta_seq(const void* qkv, int ld, int q_off, int k_off, int v_off, const float* z, int ldz, int beta_off, const float* decay,
+                                    int ld_decay, const float* a_log, const float* dt_bias, float* state, long slot_stride, const int* slot,
+                                    const int* row0, const int* len, float* out, int heads, int kv_heads, int dim, int vdim, int entries, int f32,
+                                    pk_stream st) {
+  if (!seq_args_ok(qkv, z, a_log, dt_bias, state, slot, row0, len, out, heads, kv_heads, dim, vdim, entries) || !decay || ld_decay < heads * dim) return -1;
+  SeqArgs a{qkv, ld, q_off, k_off, v_off, z, ldz, 0, beta_off, a_log, dt_bias, state, slot_stride, slot, row0, len, out, nullptr,
+            heads, kv_heads, dim, vdim, 0.f, nullptr, 0, 0, nullptr, decay, ld_decay};
+  return f32 ? launch_seq<float, 3>(a, entries, st) : launch_seq<bf16, 3>(a, entries, st);
+}
+
 extern "C" int pk_mlstm_seq(const void* qkv, int ld, int q_off, int k_off, int v_off, const float* z, int ldz, int forget_off, int input_off,
                             const float* input_bias, const float* forget_bias, float cap, float* state, long slot_stride, const int* slot,
                             const int* row0, const int* len, float* out, float* den, int heads, int dim, int vdim, int entries, int f32,
@@ -443,25 +619,30 @@ extern "C" int pk_mlstm_seq(const void* qkv, int ld, int q_off, int k_off, int v
 
 extern "C" int pk_head_norm_gate(const float* o, const float* den, const void* w, int w_stride, const void* gate, int ld_gate, int gate_off, void* out,
                                  int tokens, int heads, int vdim, float eps, int act, int f32, pk_stream st) {
-  if (!o || !w || !gate || !out || tokens <= 0 || heads <= 0 || vdim <= 0 || act < 0 || act > 2) return -1;
+  return pk_head_norm_gate_ex(o, den, w, w_stride, gate, ld_gate, gate_off, out, heads * vdim, 1.f, tokens, heads, vdim, eps, act, f32, st);
+}
+
+extern "C" int pk_head_norm_gate_ex(const float* o, const float* den, const void* w, int w_stride, const void* gate, int ld_gate, int gate_off, void* out,
+                                    int ld_out, float factor, int tokens, int heads, int vdim, float eps, int act, int f32, pk_stream st) {
+  if (!o || !w || !gate || !out || tokens <= 0 || heads <= 0 || vdim <= 0 || ld_out < heads * vdim || act < 0 || act > 2) return -1;
   const long pairs = (long)tokens * heads;
   if (vdim >= 256 && vdim <= 4096 && pairs <= 1024) {  // few wide pairs: a CTA each, so that a decode step is not one warp's loop
     const dim3 gw((unsigned)pairs), bw(vdim <= 512 ? 128 : vdim <= 1024 ? 256 : 1024);
     if (f32)
       launch(head_norm_gate_wide_kernel<float>, gw, bw, 0, st, true, o, den, (const float*)w, w_stride, (const float*)gate, ld_gate, gate_off, (float*)out,
-             heads, vdim, eps, act);
+             ld_out, factor, heads, vdim, eps, act);
     else
       launch(head_norm_gate_wide_kernel<bf16>, gw, bw, 0, st, true, o, den, (const bf16*)w, w_stride, (const bf16*)gate, ld_gate, gate_off, (bf16*)out,
-             heads, vdim, eps, act);
+             ld_out, factor, heads, vdim, eps, act);
     return (int)cudaGetLastError();
   }
   const dim3 g((unsigned)((pairs + 3) / 4));
   if (f32)
     launch(head_norm_gate_kernel<float>, g, dim3(128), 0, st, true, o, den, (const float*)w, w_stride, (const float*)gate, ld_gate, gate_off, (float*)out,
-           heads, vdim, eps, act, pairs);
+           ld_out, factor, heads, vdim, eps, act, pairs);
   else
-    launch(head_norm_gate_kernel<bf16>, g, dim3(128), 0, st, true, o, den, (const bf16*)w, w_stride, (const bf16*)gate, ld_gate, gate_off, (bf16*)out, heads,
-           vdim, eps, act, pairs);
+    launch(head_norm_gate_kernel<bf16>, g, dim3(128), 0, st, true, o, den, (const bf16*)w, w_stride, (const bf16*)gate, ld_gate, gate_off, (bf16*)out, ld_out,
+           factor, heads, vdim, eps, act, pairs);
   return (int)cudaGetLastError();
 }
 
@@ -474,4 +655,23 @@ extern "C" int pk_ssd_seq(const void* xbc, int ld, int x_off, int b_off, int c_o
   SeqArgs a{xbc, ld, c_off, b_off, x_off, nullptr, 0, 0, 0, a_log, dt_bias, state, slot_stride, slot, row0, len, out, nullptr,
             heads, groups, state_dim, vdim, 0.f, dt, ld_dt, dt_off, d_skip};
   return f32 ? launch_seq<float, 2>(a, entries, st) : launch_seq<bf16, 2>(a, entries, st);
+}
+
+extern "C" int pk_lru_seq(const void* u, int ld_u, const float* z, int ldz, const float* r_bias, const float* i_bias, const float* lam, float rate,
+                          int blocks, const void* y, int ld_y, const void* y_bias, float* state, long slot_stride, const int* slot, const int* row0,
+                          const int* len, void* out, int ld_out, int channels, int tokens, int entries, int f32, pk_stream st) {
+  if (!u || !z || !r_bias || !i_bias || !lam || !y || !state || !slot || !row0 || !len || !out || channels <= 0 || blocks <= 0 || channels % blocks ||
+      tokens <= 0 || entries <= 0 || !(rate > 0.f))
+    return -1;
+  LruArgs a{u, y, y_bias, z, r_bias, i_bias, lam, state, slot, row0, len, out, slot_stride, ld_u, ld_y, ldz, ld_out, channels, channels / blocks, rate};
+  if (tokens <= 8 * entries) {
+    const dim3 g((channels + 63) / 64, entries);
+    if (f32) launch(lru_step_kernel<float>, g, dim3(64), 0, st, true, a);
+    else launch(lru_step_kernel<bf16>, g, dim3(64), 0, st, true, a);
+  } else {
+    const dim3 g((channels + 15) / 16, entries);
+    if (f32) launch(lru_scan_kernel<float, 8>, g, dim3(512), 0, st, true, a);
+    else launch(lru_scan_kernel<bf16, 8>, g, dim3(512), 0, st, true, a);
+  }
+  return (int)cudaGetLastError();
 }

@@ -80,6 +80,7 @@ __global__ void skinny_proj_kernel(const E* __restrict__ W, const float* __restr
 
 // kind 0: out[t][f] = silu(in[t][f]) * in[t][F + f]   (in is [T, 2F]: gate rows stacked over up rows)
 // kind 1: out[t][f] = relu(in[t][f])^2                (in is [T, F])
+// kind 2: out[t][f] = relu(in[t][f]) * in[t][F + f]   (in is [T, 2F])
 template <typename E>
 __global__ void act_kernel(const E* __restrict__ in, E* __restrict__ out, int F, long total, int kind) {
   pdl_wait();
@@ -87,9 +88,9 @@ __global__ void act_kernel(const E* __restrict__ in, E* __restrict__ out, int F,
   for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x) {
     const long t = i / F, f = i % F;
     float r;
-    if (kind == 0) {
+    if (kind != 1) {
       const float g = to_f(in[t * 2 * F + f]), u = to_f(in[t * 2 * F + F + f]);
-      r = g / (1.f + expf(-g)) * u;
+      r = (kind == 2 ? fmaxf(g, 0.f) : g / (1.f + expf(-g))) * u;
     } else {
       const float u = fmaxf(to_f(in[i]), 0.f);
       r = u * u;
@@ -107,8 +108,8 @@ __global__ void convert_kernel(const A* __restrict__ in, B* __restrict__ out, lo
 
 // C[b][i][j] = (sum_k A[b*bsA + i*lda + k] * B[b*bsB + k*sbk + j*sbn]) * f(row_scale[i*ld_scale + b])
 // f = identity (scale_kind 1) or logistic (scale_kind 2); no scale when row_scale is null.  64 x 64 output tile, 256 threads, 4 x 4 each.
-template <typename E>
-__global__ void gemm_strided_kernel(const E* __restrict__ A, const E* __restrict__ B, E* __restrict__ C, const float* __restrict__ row_scale,
+template <typename E, typename O>
+__global__ void gemm_strided_kernel(const E* __restrict__ A, const E* __restrict__ B, O* __restrict__ C, const float* __restrict__ row_scale,
                                     int rows, int cols, int K, long lda, long sbk, long sbn, long ldc, long bsA, long bsB, long bsC,
                                     int ld_scale, int scale_kind) {
   constexpr int TL = 64, KT = 16;
@@ -166,15 +167,15 @@ __global__ void gemm_strided_kernel(const E* __restrict__ A, const E* __restrict
 #pragma unroll
     for (int v = 0; v < 4; ++v) {
       const int j = j0 + tx * 4 + v;
-      if (j < cols) C[(size_t)i * ldc + j] = from_f<E>(acc[u][v] * s);
+      if (j < cols) C[(size_t)i * ldc + j] = from_f<O>(acc[u][v] * s);
     }
   }
 }
 
 // The same product for a few rows (decode) when B is K-contiguous (sbk == 1): grid (row, batch, slice of columns); the A row
 // is staged as fp32 in shared memory and every warp streams whole B rows.
-template <typename E>
-__global__ void gemm_strided_rows_kernel(const E* __restrict__ A, const E* __restrict__ B, E* __restrict__ C, const float* __restrict__ row_scale,
+template <typename E, typename O>
+__global__ void gemm_strided_rows_kernel(const E* __restrict__ A, const E* __restrict__ B, O* __restrict__ C, const float* __restrict__ row_scale,
                                          int cols, int K, long lda, long sbn, long ldc, long bsA, long bsB, long bsC, int ld_scale, int scale_kind) {
   extern __shared__ __align__(16) float a_s[];
   pdl_wait();
@@ -190,11 +191,13 @@ __global__ void gemm_strided_rows_kernel(const E* __restrict__ A, const E* __res
   }
   for (int j = blockIdx.z * nw + warp; j < cols; j += gridDim.z * nw) {
     const float acc = warp_dot(B + (size_t)b * bsB + (size_t)j * sbn, a_s, K, lane);
-    if (lane == 0) C[(size_t)b * bsC + (size_t)i * ldc + j] = from_f<E>(acc * s);
+    if (lane == 0) C[(size_t)b * bsC + (size_t)i * ldc + j] = from_f<O>(acc * s);
   }
 }
 
 // gemm_batched_mma.cu
+int launch_gemm_batched_mma_f32(const bf16* A, const bf16* B, float* C, int rows, int cols, int K, long lda, long ldb, long ldc, int batch, long bsA,
+                                long bsB, long bsC, cudaStream_t st);
 int launch_gemm_batched_mma(const bf16* A, const bf16* B, bf16* C, const float* row_scale, int rows, int cols, int K, long lda, long ldb, long ldc,
                             int batch, long bsA, long bsB, long bsC, int ld_scale, int scale_kind, cudaStream_t st);
 
@@ -536,6 +539,155 @@ __global__ void branches_add_norm_kernel(const Y* __restrict__ ya, const E* __re
   }
 }
 
+// ---- residual in parallel streams (hyper-connections): x [tokens, S, width] fp32.  A sublayer reads u = sum_s w_in[s] x_s through a plain-weight
+// RMS norm; its result y goes back to all streams at once, x_t <- sum_s mix[s][t] x_s + w_out[t] y.  One launch per sublayer boundary does the
+// write of one sublayer and the read + norm of the next.  One CTA per token; the streams of an entry stay in registers (S <= kMaxStreams).
+constexpr int kMaxStreams = 16;
+template <int V>
+__device__ __forceinline__ void ldv(const float* p, float* o) {
+  if constexpr (V == 4) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    o[0] = v.x, o[1] = v.y, o[2] = v.z, o[3] = v.w;
+  } else {
+    o[0] = *p;
+  }
+}
+template <int V>
+__device__ __forceinline__ void ldv(const bf16* p, float* o) {
+  if constexpr (V == 4) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    o[0] = bf16_lo(v.x), o[1] = bf16_hi(v.x), o[2] = bf16_lo(v.y), o[3] = bf16_hi(v.y);
+  } else {
+    o[0] = bf2f(*p);
+  }
+}
+template <int V>
+__device__ __forceinline__ void stv(float* p, const float* v) {
+  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  else *p = v[0];
+}
+template <int V>
+__device__ __forceinline__ void stv(bf16* p, const float* v) {
+  if constexpr (V == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
+  else *p = f2bf(v[0]);
+}
+
+// h (and h32) = row * inv * w_next over the entries this thread wrote into `row` itself
+template <typename E, int V>
+__device__ __forceinline__ void streams_norm_out(const float* row, float inv, const E* __restrict__ w_next, E* __restrict__ h, float* __restrict__ h32,
+                                                 int width) {
+  for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+    float r[V], w[V];
+    ldv<V>(row + i, r);
+    ldv<V>(w_next + i, w);
+#pragma unroll
+    for (int u = 0; u < V; ++u) r[u] *= inv * w[u];
+    stv<V>(h + i, r);
+    if (h32) stv<V>(h32 + i, r);
+  }
+}
+
+// SC > 0: the number of streams at compile time; 0: S of them.  y null: no write (the embedding of token ids[t] fills every stream instead).
+// w_in null: no read.
+template <typename E, int SC, int V>
+__global__ void __launch_bounds__(512) streams_step_kernel(const E* __restrict__ y, const E* __restrict__ embed, const int* __restrict__ ids, const float* __restrict__ mix,
+                                    const float* __restrict__ w_out, const float* __restrict__ w_in, float* __restrict__ x,
+                                    const E* __restrict__ w_next, E* __restrict__ h, float* __restrict__ h32, int width, int S_any, float eps) {
+  constexpr int MS = SC > 0 ? SC : kMaxStreams;
+  extern __shared__ __align__(16) float gn_sm[];
+  __shared__ float co[kMaxStreams * (kMaxStreams + 2)];
+  float* row = gn_sm;
+  float* red = row + width;  // 64 floats
+  const int S = SC > 0 ? SC : S_any;
+  pdl_wait();
+  pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
+  const int t = blockIdx.x;
+  float* xt = x + (size_t)t * S * width;
+  if (w_next)
+    for (int i = threadIdx.x * 64; i < width; i += blockDim.x * 64) prefetch_l2(w_next + i);
+  for (int i = threadIdx.x; i < S * (S + 2); i += blockDim.x)
+    co[i] = i < S ? (w_in ? w_in[i] : 0.f) : i < 2 * S ? (y ? w_out[i - S] : 0.f) : (y ? mix[i - 2 * S] : 0.f);
+  const E* src = y ? y + (size_t)t * width : embed + (size_t)ids[t] * width;
+  __syncthreads();
+  float cin[MS], cout[MS];
+  float cmix[SC > 0 ? SC * SC : 1];
+#pragma unroll
+  for (int s = 0; s < MS; ++s) {
+    cin[s] = s < S ? co[s] : 0.f;
+    cout[s] = s < S ? co[S + s] : 0.f;
+  }
+  if constexpr (SC > 0) {
+#pragma unroll
+    for (int i = 0; i < SC * SC; ++i) cmix[i] = co[2 * SC + i];
+  }
+  float ss = 0.f;
+  for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+    float yv[V], u[V] = {};
+    ldv<V>(src + i, yv);
+    if (y) {
+      float xo[MS][V];
+#pragma unroll
+      for (int s = 0; s < MS; ++s)
+        if (s < S) ldv<V>(xt + (size_t)s * width + i, xo[s]);
+#pragma unroll
+      for (int d = 0; d < MS; ++d) {
+        if (d >= S) break;
+        float v[V];
+#pragma unroll
+        for (int k = 0; k < V; ++k) v[k] = cout[d] * yv[k];
+#pragma unroll
+        for (int s = 0; s < MS; ++s) {
+          if (s >= S) break;
+          const float m = SC > 0 ? cmix[SC > 0 ? s * SC + d : 0] : co[2 * S + s * S + d];
+#pragma unroll
+          for (int k = 0; k < V; ++k) v[k] = fmaf(m, xo[s][k], v[k]);
+        }
+        stv<V>(xt + (size_t)d * width + i, v);
+#pragma unroll
+        for (int k = 0; k < V; ++k) u[k] = fmaf(cin[d], v[k], u[k]);
+      }
+    } else {
+#pragma unroll
+      for (int d = 0; d < MS; ++d) {
+        if (d >= S) break;
+        stv<V>(xt + (size_t)d * width + i, yv);
+#pragma unroll
+        for (int k = 0; k < V; ++k) u[k] = fmaf(cin[d], yv[k], u[k]);
+      }
+    }
+    stv<V>(row + i, u);
+#pragma unroll
+    for (int k = 0; k < V; ++k) ss = fmaf(u[k], u[k], ss);
+  }
+  if (!w_next) return;
+  const float inv = 1.f / sqrtf(block_sum2(ss, 0.f, red).x / (float)width + eps);
+  streams_norm_out<E, V>(row, inv, w_next, h + (size_t)t * width, h32 ? h32 + (size_t)t * width : nullptr, width);
+}
+
+// out[r] = rms(sum_s x[rows[r]][s]) * w in the element type (rows null: every row);  w null: out32[r] = the sum itself
+template <typename E>
+__global__ void streams_rows_kernel(const float* __restrict__ x, const int* __restrict__ rows, const E* __restrict__ w, E* __restrict__ out,
+                                    float* __restrict__ out32, int width, int S, float eps) {
+  extern __shared__ __align__(16) float gn_sm[];
+  float* row = gn_sm;
+  float* red = row + width;
+  pdl_wait();
+  pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
+  const int r = blockIdx.x;
+  const float* xt = x + (size_t)(rows ? rows[r] : r) * S * width;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < width; i += blockDim.x) {
+    float v = 0.f;
+    for (int s = 0; s < S; ++s) v += xt[(size_t)s * width + i];
+    row[i] = v;
+    ss = fmaf(v, v, ss);
+    if (!w) out32[(size_t)r * width + i] = v;
+  }
+  if (!w) return;
+  const float inv = 1.f / sqrtf(block_sum2(ss, 0.f, red).x / (float)width + eps);
+  for (int i = threadIdx.x; i < width; i += blockDim.x) out[(size_t)r * width + i] = from_f<E>(row[i] * inv * to_f(w[i]));
+}
+
 // out = cap * tanh(float(in) * scale / cap)  (cap 0: float(in) * scale)
 template <typename A>
 __global__ void logits_scale_cap_kernel(const A* __restrict__ in, float* __restrict__ out, long n, float scale, float cap) {
@@ -572,6 +724,28 @@ static bool gnorm_fits(K kernel, size_t smem) {  // rows above 48 KB of shared m
   if (smem <= 48 * 1024) return true;
   if (smem > 200 * 1024) return false;
   return cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) == cudaSuccess;
+}
+
+template <typename E>
+static int launch_streams(const E* y, const E* embed, const int* ids, const float* mix, const float* w_out, const float* w_in, float* x, const E* w_next, E* h,
+                          float* h32, int width, int S, float eps, int tokens, cudaStream_t st) {
+  const size_t sm = (size_t)(width + 64) * sizeof(float);
+  auto al = [](const void* p, int n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)) == 0; };
+  const bool vec = width % 4 == 0 && al(x, 16) && al(y, 4 * sizeof(E)) && al(embed, 4 * sizeof(E)) && al(w_next, 4 * sizeof(E)) && al(h, 4 * sizeof(E)) && al(h32, 16);
+  const int v = vec ? 4 : 1, thr = std::min(tokens > 64 ? 256 : 512, std::max(32, (width / v + 31) / 32 * 32));
+#define PK_ST(SC, V)                                                                                                                              \
+  do {                                                                                                                                            \
+    if (!gnorm_fits(streams_step_kernel<E, SC, V>, sm)) return -2;                                                                                \
+    launch(streams_step_kernel<E, SC, V>, dim3(tokens), dim3(thr), sm, st, true, y, embed, ids, mix, w_out, w_in, x, w_next, h, h32, width, S, eps); \
+  } while (0)
+  if (!vec) PK_ST(0, 1);
+  else if (S == 1) PK_ST(1, 4);
+  else if (S == 2) PK_ST(2, 4);
+  else if (S == 3) PK_ST(3, 4);
+  else if (S == 4) PK_ST(4, 4);
+  else PK_ST(0, 4);
+#undef PK_ST
+  return (int)cudaGetLastError();
 }
 
 }  // namespace pk
@@ -625,7 +799,7 @@ extern "C" int pk_res32_skinny_proj(const void* W, const float* x, float* out, i
 }
 
 extern "C" int pk_act(const void* in, void* out, int F, int tokens, int kind, int f32, pk_stream st) {
-  if (!in || !out || F <= 0 || tokens <= 0 || kind < 0 || kind > 1) return -1;
+  if (!in || !out || F <= 0 || tokens <= 0 || kind < 0 || kind > 2) return -1;
   const long total = (long)F * tokens;
   PK_BY_TYPE(f32, launch(act_kernel<float>, dim3(grid_1d(total, 256)), dim3(256), 0, st, true, (const float*)in, (float*)out, F, total, kind),
              launch(act_kernel<bf16>, dim3(grid_1d(total, 256)), dim3(256), 0, st, true, (const bf16*)in, (bf16*)out, F, total, kind));
@@ -649,9 +823,9 @@ extern "C" int pk_gemm_strided(const void* A, const void* B, void* C, const floa
     const dim3 gr(rows, batch, (cols + 31) / 32), br(256);
     const size_t sm = (size_t)K * sizeof(float);
     PK_BY_TYPE(f32,
-               launch(gemm_strided_rows_kernel<float>, gr, br, sm, st, true, (const float*)A, (const float*)B, (float*)C, row_scale, cols, K, lda, sbn,
+               launch(gemm_strided_rows_kernel<float, float>, gr, br, sm, st, true, (const float*)A, (const float*)B, (float*)C, row_scale, cols, K, lda, sbn,
                       ldc, bsA, bsB, bsC, ld_scale, scale_kind),
-               launch(gemm_strided_rows_kernel<bf16>, gr, br, sm, st, true, (const bf16*)A, (const bf16*)B, (bf16*)C, row_scale, cols, K, lda, sbn, ldc,
+               launch(gemm_strided_rows_kernel<bf16, bf16>, gr, br, sm, st, true, (const bf16*)A, (const bf16*)B, (bf16*)C, row_scale, cols, K, lda, sbn, ldc,
                       bsA, bsB, bsC, ld_scale, scale_kind));
     return (int)cudaGetLastError();
   }
@@ -662,10 +836,36 @@ extern "C" int pk_gemm_strided(const void* A, const void* B, void* C, const floa
   }
   const dim3 g((cols + 63) / 64, (rows + 63) / 64, batch), b(256);
   PK_BY_TYPE(f32,
-             launch(gemm_strided_kernel<float>, g, b, 0, st, true, (const float*)A, (const float*)B, (float*)C, row_scale, rows, cols, K, lda, sbk,
+             launch(gemm_strided_kernel<float, float>, g, b, 0, st, true, (const float*)A, (const float*)B, (float*)C, row_scale, rows, cols, K, lda, sbk,
                     sbn, ldc, bsA, bsB, bsC, ld_scale, scale_kind),
-             launch(gemm_strided_kernel<bf16>, g, b, 0, st, true, (const bf16*)A, (const bf16*)B, (bf16*)C, row_scale, rows, cols, K, lda, sbk, sbn,
+             launch(gemm_strided_kernel<bf16, bf16>, g, b, 0, st, true, (const bf16*)A, (const bf16*)B, (bf16*)C, row_scale, rows, cols, K, lda, sbk, sbn,
                     ldc, bsA, bsB, bsC, ld_scale, scale_kind));
+  return (int)cudaGetLastError();
+}
+
+extern "C" int pk_gemm_strided_f32out(const void* A, const void* B, float* C, int rows, int cols, int K, long lda, long ldb, long ldc, int batch, long bsA,
+                                      long bsB, long bsC, int f32, pk_stream st) {
+  if (!A || !B || !C || rows <= 0 || cols <= 0 || K <= 0 || batch <= 0) return -1;
+  if (rows <= 8 && K <= 8192) {
+    const dim3 gr(rows, batch, (cols + 31) / 32), br(256);
+    const size_t sm = (size_t)K * sizeof(float);
+    PK_BY_TYPE(f32,
+               launch(gemm_strided_rows_kernel<float, float>, gr, br, sm, st, true, (const float*)A, (const float*)B, C, (const float*)nullptr, cols, K, lda,
+                      ldb, ldc, bsA, bsB, bsC, 0, 0),
+               launch(gemm_strided_rows_kernel<bf16, float>, gr, br, sm, st, true, (const bf16*)A, (const bf16*)B, C, (const float*)nullptr, cols, K, lda, ldb,
+                      ldc, bsA, bsB, bsC, 0, 0));
+    return (int)cudaGetLastError();
+  }
+  if (!f32) {
+    const int rc = launch_gemm_batched_mma_f32((const bf16*)A, (const bf16*)B, C, rows, cols, K, lda, ldb, ldc, batch, bsA, bsB, bsC, st);
+    if (rc != -2) return rc;
+  }
+  const dim3 g((cols + 63) / 64, (rows + 63) / 64, batch), b(256);
+  PK_BY_TYPE(f32,
+             launch(gemm_strided_kernel<float, float>, g, b, 0, st, true, (const float*)A, (const float*)B, C, (const float*)nullptr, rows, cols, K, lda, 1L,
+                    ldb, ldc, bsA, bsB, bsC, 0, 0),
+             launch(gemm_strided_kernel<bf16, float>, g, b, 0, st, true, (const bf16*)A, (const bf16*)B, C, (const float*)nullptr, rows, cols, K, lda, 1L, ldb,
+                    ldc, bsA, bsB, bsC, 0, 0));
   return (int)cudaGetLastError();
 }
 
@@ -799,5 +999,34 @@ extern "C" int pk_act_clamped(const void* in, void* out, int F, int tokens, floa
   const long total = (long)F * tokens;
   PK_BY_TYPE(f32, launch(act_clamped_kernel<float>, dim3(grid_1d(total, 256)), dim3(256), 0, st, true, (const float*)in, (float*)out, F, total, limit, slope),
              launch(act_clamped_kernel<bf16>, dim3(grid_1d(total, 256)), dim3(256), 0, st, true, (const bf16*)in, (bf16*)out, F, total, limit, slope));
+  return (int)cudaGetLastError();
+}
+
+extern "C" int pk_res32_streams_embed(const void* embed, const int* token_ids, const float* w_in, float* x, const void* w_next, void* h, float* h32, int width,
+                                      int streams, float eps, int tokens, int f32, pk_stream st) {
+  if (!embed || !token_ids || !x || (w_next && (!h || !w_in)) || width <= 0 || tokens <= 0 || streams <= 0 || streams > kMaxStreams) return -1;
+  if (f32)
+    return launch_streams<float>(nullptr, (const float*)embed, token_ids, nullptr, nullptr, w_in, x, (const float*)w_next, (float*)h, h32, width, streams, eps,
+                                 tokens, st);
+  return launch_streams<bf16>(nullptr, (const bf16*)embed, token_ids, nullptr, nullptr, w_in, x, (const bf16*)w_next, (bf16*)h, h32, width, streams, eps, tokens,
+                              st);
+}
+
+extern "C" int pk_res32_streams_step(const void* y, const float* mix, const float* w_out, const float* w_in, float* x, const void* w_next, void* h, float* h32,
+                                     int width, int streams, float eps, int tokens, int f32, pk_stream st) {
+  if (!y || !mix || !w_out || !x || (w_next && (!h || !w_in)) || width <= 0 || tokens <= 0 || streams <= 0 || streams > kMaxStreams) return -1;
+  if (f32)
+    return launch_streams<float>((const float*)y, nullptr, nullptr, mix, w_out, w_in, x, (const float*)w_next, (float*)h, h32, width, streams, eps, tokens, st);
+  return launch_streams<bf16>((const bf16*)y, nullptr, nullptr, mix, w_out, w_in, x, (const bf16*)w_next, (bf16*)h, h32, width, streams, eps, tokens, st);
+}
+
+extern "C" int pk_res32_streams_rows(const float* x, const int* rows, const void* w, void* out, float* out32, int width, int streams, float eps, int n_rows,
+                                     int f32, pk_stream st) {
+  if (!x || (w ? !out : !out32) || width <= 0 || n_rows <= 0 || streams <= 0) return -1;
+  const size_t sm = (size_t)(width + 64) * sizeof(float);
+  if (!(f32 ? gnorm_fits(streams_rows_kernel<float>, sm) : gnorm_fits(streams_rows_kernel<bf16>, sm))) return -2;
+  const dim3 g(n_rows), b(gnorm_threads(width, n_rows));
+  PK_BY_TYPE(f32, launch(streams_rows_kernel<float>, g, b, sm, st, true, x, rows, (const float*)w, (float*)out, out32, width, streams, eps),
+             launch(streams_rows_kernel<bf16>, g, b, sm, st, true, x, rows, (const bf16*)w, (bf16*)out, out32, width, streams, eps));
   return (int)cudaGetLastError();
 }

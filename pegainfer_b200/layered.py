@@ -28,14 +28,17 @@ class LayerCfg(C.Structure):
                [("q_temp_coef", C.c_float)] + \
                [(n, C.c_int) for n in ("q_temp_every", "values_are_keys", "scaling_kind", "ssm_heads", "ssm_vdim", "ssm_state", "ssm_groups",
                                        "ssm_norm_groups")] + \
-               [(n, C.c_float) for n in ("act_limit", "act_slope", "shared_limit")] + [("weights_of", C.c_int)]
+               [(n, C.c_float) for n in ("act_limit", "act_slope", "shared_limit")] + [("weights_of", C.c_int)] + \
+               [(n, C.c_int) for n in ("d_heads", "d_kv_heads", "d_dim", "d_vdim", "decay_rank", "gate_rank")] + \
+               [("left_scale", C.c_float), ("right_scale", C.c_float), ("lru_width", C.c_int), ("lru_blocks", C.c_int), ("lru_rate", C.c_float),
+                ("mlp_act", C.c_int)]
 
 
 class ModelCfg(C.Structure):
     _fields_ = [("vocab", C.c_int), ("width", C.c_int), ("n_layers", C.c_int), ("eps", C.c_float)] + \
                [(n, C.c_int) for n in ("f32", "page_size", "num_pages", "max_requests", "device", "enable_pdl", "block_kind")] + \
                [("embed_scale", C.c_float), ("logit_scale", C.c_float), ("norm_groups", C.c_int), ("residual_mult", C.c_float),
-                ("gated_residual", C.c_int), ("logit_softcap", C.c_float)]
+                ("gated_residual", C.c_int), ("logit_softcap", C.c_float), ("streams", C.c_int)]
 
 
 def typed_host():
@@ -89,6 +92,11 @@ class LayeredModel:
         raise NotImplementedError
 
     @staticmethod
+    def complete_config(cfg, shapes: dict):
+        """The configuration with the sizes that only the checkpoint's tensors give (``shapes``: name -> shape) filled in."""
+        return cfg
+
+    @staticmethod
     def layer_struct(layer) -> "LayerCfg":
         raise NotImplementedError
 
@@ -104,6 +112,8 @@ class LayeredModel:
             raise RuntimeError("pegainfer_b200 needs a CUDA device (there is no CPU path)")
         if dtype not in (torch.bfloat16, torch.float32):
             raise ValueError("dtype must be torch.bfloat16 or torch.float32")
+        if isinstance(weights, dict):
+            cfg = self.complete_config(cfg, {n: tuple(t.shape) for n, t in weights.items()})
         self.cfg, self.dtype, self._h = cfg, dtype, typed_host()
         f32 = int(dtype == torch.float32)
         lcs = (LayerCfg * len(cfg.layers))()
@@ -112,7 +122,7 @@ class LayeredModel:
         mc = self.model_struct(cfg, ModelCfg(vocab=cfg.vocab, width=cfg.width, n_layers=len(cfg.layers), eps=cfg.eps, f32=f32, page_size=PAGE_SIZE,
                                              num_pages=pages_for(max_tokens) if max_tokens > 0 else 0, max_requests=max_requests, device=device_ordinal,
                                              enable_pdl=int(enable_pdl), block_kind=0, embed_scale=1.0, logit_scale=1.0, norm_groups=1,
-                                             residual_mult=1.0, gated_residual=0, logit_softcap=0.0))
+                                             residual_mult=1.0, gated_residual=0, logit_softcap=0.0, streams=0))
         torch.cuda.set_device(device_ordinal)
         self._m = self._h.pv_create(C.byref(mc), lcs, (kernel_lib or ffi.KERNEL_LIB_PATH).encode())
         if not self._m:
@@ -129,7 +139,7 @@ class LayeredModel:
             if t.is_cuda:
                 torch.cuda.current_stream().synchronize()
             t = t.to(dtype).contiguous()
-            rows, cols = (t.shape[0], t.shape[1]) if t.dim() == 2 else (1, t.numel())
+            rows, cols = (t.numel() // t.shape[-1], t.shape[-1]) if t.dim() >= 2 else (1, t.numel())
             self._ck(self._h.pv_load_tensor(self._m, name.encode(), t.data_ptr(), rows, cols, f32))
             seen.add(name)
         missing = [n for n in shapes if n not in seen]
@@ -145,6 +155,12 @@ class LayeredModel:
         with open(os.path.join(model_path, "config.json")) as f:
             cfg = cls.config_class.from_dict(json.load(f), os.path.basename(os.path.normpath(model_path)) or "custom")
         files, _ = load_shard_info(model_path)
+
+        shapes = {}
+        for p in files:
+            with safe_open(p, framework="pt", device="cpu") as h:
+                shapes.update((name, tuple(h.get_slice(name).get_shape())) for name in h.keys())
+        cfg = cls.complete_config(cfg, shapes)
 
         def tensors():
             for p in files:

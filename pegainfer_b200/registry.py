@@ -33,6 +33,11 @@ def _load_goguzen(path, dtype, max_tokens, max_requests, **kw):
     return GoguzenModel.from_pretrained(path, dtype=dtype, max_tokens=max_tokens, max_requests=max_requests, **kw)
 
 
+def _load_rilonex(path, dtype, max_tokens, max_requests, **kw):
+    from .rilonex import RilonexModel
+    return RilonexModel.from_pretrained(path, dtype=dtype, max_tokens=max_tokens, max_requests=max_requests, **kw)
+
+
 def _load_qwen3(path, dtype, max_tokens, max_requests, **kw):
     from .config import PAGE_SIZE
     from .model import ModelRuntimeConfig, Qwen3Model
@@ -48,11 +53,12 @@ ARCHITECTURES = {
     "Risolorn": _load_risolorn,
     "Nagosun": _load_nagosun,
     "Goguzen": _load_goguzen,
+    "Rilonex": _load_rilonex,
     "Qwen3ForCausalLM": _load_qwen3,
     "qwen3": _load_qwen3,
 }
 # designs whose kernels run with every product in fp32 as well
-FLOAT32_CAPABLE = {"Vamadra", "Risolorn", "Nagosun", "Goguzen"}
+FLOAT32_CAPABLE = {"Vamadra", "Risolorn", "Nagosun", "Goguzen", "Rilonex"}
 
 
 def architecture_of(model_path: str) -> str:
