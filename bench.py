@@ -825,6 +825,22 @@ def _goguzen_sizes():
     return {"w2048": gog(2048, 16, 4, 128, 1024, 64, 6, 1408, 2816, 32768), "w1024": gog(1024, 8, 2, 64, 1024, 16, 2, 768, 1536, 32768)}
 
 
+def _rilonex_sizes():
+    """Rilonex stacks of the same width, head count and vocabulary as the Goguzen stacks of `_goguzen_sizes` (its closest relative: attention
+    beside a recurrent branch on the same host), with the dense feed-forward of the Qwen3 stack of that width: attention beside a delta rule,
+    linear recurrent unit, per-channel delta rule, attention beside a delta rule; four residual streams."""
+    def ril(width, heads, kv, dim, ff, rank, vocab):
+        mlp = {"kind": "dense", "ff": ff}
+        dlt = {"heads": heads, "kv_heads": heads // 2, "dim": dim, "vdim": dim, "conv": 4}
+        par = {"type": "parallel", "mlp": mlp,
+               "mixer": {"left": {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "rot": {"dims": dim, "base": 1000000.0}},
+                         "right": dlt, "left_scale": 0.5, "right_scale": 0.5}}
+        return ({"architecture": "Rilonex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "streams": 4,
+                 "layers": [par, {"type": "rglru", "mlp": mlp, "mixer": {"width": width, "blocks": heads, "conv": 4}},
+                            {"type": "channel_delta", "mlp": mlp, "mixer": dict(dlt, kv_heads=heads)}, par]}, rank)
+    return {"w2048": ril(2048, 16, 4, 128, 6 * 1408 + 2816, 128, 32768), "w1024": ril(1024, 8, 2, 64, 2 * 768 + 1536, 64, 32768)}
+
+
 def _measure_layered(vm, prompts, ctx, med, synthetic_prompt):
     """prefill tok/s per prompt length and decode tok/s at batch 1 and 4 of a model on the layer-list host"""
     res = {}
@@ -853,7 +869,8 @@ def _measure_layered(vm, prompts, ctx, med, synthetic_prompt):
 
 def run_arch_compare(args):
     """`--arch vamadra`: prefill and decode throughput of the Vamadra path beside the Qwen3 path at equal size.  `--arch risolorn` /
-    `--arch nagosun`: that design's path beside both.  `--arch goguzen`: that design's path beside Risolorn's and Qwen3's.  Wall clock around each public-API call (token ids from the host in, logits / token back out,
+    `--arch nagosun`: that design's path beside both.  `--arch goguzen`: that design's path beside Risolorn's and Qwen3's.  `--arch rilonex`:
+    beside Goguzen's, Risolorn's and Qwen3's.  Wall clock around each public-API call (token ids from the host in, logits / token back out,
     stream synchronised), median of the repeats after warm-up; between repeats nothing else runs on the GPU.  One JSON line."""
     import torch
     from pegainfer_b200.model import ModelRuntimeConfig, Qwen3Model
@@ -861,7 +878,7 @@ def run_arch_compare(args):
     from pegainfer_b200.vamadra import VamadraConfig, VamadraModel, iter_random_weights as vam_weights
     reps, warm = max(3, min(args.steps, 20)), max(3, min(args.warmup, 5))
     prompts, ctx, dec_steps = [512, 2048], 2048, 32
-    beside = {"vamadra": "qwen3", "goguzen": "risolorn, qwen3"}.get(args.arch, "vamadra, qwen3")
+    beside = {"vamadra": "qwen3", "goguzen": "risolorn, qwen3", "rilonex": "goguzen, risolorn, qwen3"}.get(args.arch, "vamadra, qwen3")
     out = {"metric": "prefill_and_decode_tok_s", "arch": args.arch, "beside": beside, "dtype": "bf16",
            "data": "synthetic", "n_gpus": 1,
            "timing": "wall clock around the public API call incl. host->device ids and device->host result, stream synchronised", "sizes": {}}
@@ -881,13 +898,22 @@ def run_arch_compare(args):
         if args.arch_size and name not in args.arch_size.split(","):
             continue
         row = {}
-        if args.arch == "goguzen":
+        if args.arch == "rilonex":
+            from pegainfer_b200.rilonex import RilonexConfig, RilonexModel, iter_random_weights as ril_weights, with_ranks
+            lcfg_d, rank = _rilonex_sizes()[name]
+            lcfg = RilonexConfig.from_dict(lcfg_d)
+            ranks = {f"l{i}.mix.{n}": (rank, lcfg.width) for i in range(len(lcfg.layers)) for n in ("a1", "g1")}
+            lcfg = with_ranks(lcfg, ranks)
+            lm = RilonexModel(lcfg, ril_weights(lcfg, 0, "cuda"), max_tokens=pool_tokens, max_requests=5)
+            row["rilonex"] = _measure_layered(lm, prompts, ctx, med, synthetic_prompt)
+            lm.close()
+        if args.arch in ("goguzen", "rilonex"):
             from pegainfer_b200.goguzen import GoguzenConfig, GoguzenModel, iter_random_weights as gog_weights
             gcfg = GoguzenConfig.from_dict(_goguzen_sizes()[name])
             gm = GoguzenModel(gcfg, gog_weights(gcfg, 0, "cuda"), max_tokens=pool_tokens, max_requests=5)
             row["goguzen"] = _measure_layered(gm, prompts, ctx, med, synthetic_prompt)
             gm.close()
-        if args.arch in ("risolorn", "goguzen"):
+        if args.arch in ("risolorn", "goguzen", "rilonex"):
             from pegainfer_b200.risolorn import RisolornConfig, RisolornModel, iter_random_weights as ris_weights
             rcfg = RisolornConfig.from_dict(_risolorn_sizes()[name])
             rm = RisolornModel(rcfg, ris_weights(rcfg, 0, "cuda"), max_tokens=pool_tokens, max_requests=5)
@@ -899,7 +925,7 @@ def run_arch_compare(args):
             nm = NagosunModel(ncfg, nag_weights(ncfg, 0, "cuda"), max_tokens=pool_tokens, max_requests=5)
             row["nagosun"] = _measure_layered(nm, prompts, ctx, med, synthetic_prompt)
             nm.close()
-        if args.arch != "goguzen":
+        if args.arch not in ("goguzen", "rilonex"):
             vcfg = VamadraConfig.from_dict(vcfg_d)
             vm = VamadraModel(vcfg, vam_weights(vcfg, 0, "cuda"), max_tokens=pool_tokens, max_requests=5)
             row["vamadra"] = _measure_layered(vm, prompts, ctx, med, synthetic_prompt)
@@ -946,7 +972,7 @@ def main():
     ap.add_argument("--weights", default="cpu", choices=["cpu", "cuda"],
                     help="cpu (default): the seed-0 CPU checkpoint the oracle fixtures were computed on; cuda: generated on "
                          "each GPU (fast; tuning sweeps only -- the parity key then reports a different checkpoint)")
-    ap.add_argument("--arch", default=None, choices=["vamadra", "risolorn", "nagosun", "goguzen"],
+    ap.add_argument("--arch", default=None, choices=["vamadra", "risolorn", "nagosun", "goguzen", "rilonex"],
                     help="instead of the headline workload: prefill / decode throughput of this design beside the closest existing ones at equal size")
     ap.add_argument("--arch-size", default=None, help="with --arch: comma-separated subset of the sizes (w2048,w1024)")
     args = ap.parse_args()
