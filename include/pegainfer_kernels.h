@@ -630,21 +630,23 @@ int pk_res32_streams_rows(const float* x, const int* rows, const void* w, void* 
  * s_h(j) = scale * q[t,h] . k_j;  z_h = sum_g score_mix[h * heads + g] s_g + head_bias[h] (score_mix element type, NULL: z_h = s_h + bias; head_bias float,
  * may be NULL);  out[t,h] = out_scale * logistic(gate[t * gate_ld + h]) * sum_{j <= positions[t]} logistic(z_h(j)) v_j, not normalised over keys.
  * gate: fp32 pre-activations, may be NULL.  out has rows of stride out_ld.  max_kv_len: longest context of the step (0: unknown), a hint for
- * splitting the key axis. */
+ * splitting the key axis; the shares' partial sums (tokens * heads * vdim floats each) go to the workspace (NULL: no splitting). */
 int pk_gqa_mixed_attention(const void* q, const void* cache, const void* score_mix, const float* head_bias, const float* gate, int gate_ld,
                            const int* positions, const int* req, const int* page_off, const int* pages, void* out, int out_ld, float out_scale,
-                           long page_stride, int page_size, int tokens, int heads, int kv_heads, int dim, int vdim, float scale, int max_kv_len, int f32,
-                           pk_stream st);
+                           long page_stride, int page_size, int tokens, int heads, int kv_heads, int dim, int vdim, float scale, int max_kv_len, void* workspace,
+                           long workspace_bytes, int f32, pk_stream st);
 /* Short causal convolution per channel of in + in_bias, plus bias, act 0: none / 1: SiLU (either bias may be NULL); the slot's state keeps the last
  * taps - 1 biased inputs [taps-1][channels] and is updated by the same launch. */
 int pk_causal_conv(const void* in, int ld_in, const void* in_bias, const void* w, const void* bias, int act, float* state, long slot_stride,
                    const int* slot, const int* row0, const int* len, void* out, int ld_out, int channels, int taps, int tokens, int entries, int f32,
                    pk_stream st);
 /* pk_gated_delta_seq with one decay per head and key channel: decay [tokens, ld_decay] fp32 holds its pre-activation at h * dim + d,
- * g = exp(-exp(a_log[h]) * softplus(decay + dt_bias[h * dim + d])). */
+ * g = exp(-exp(a_log[h]) * softplus(decay + dt_bias[h * dim + d])); with decay_ready it holds the decays g themselves. */
 int pk_channel_delta_seq(const void* qkv, int ld, int q_off, int k_off, int v_off, const float* z, int ldz, int beta_off, const float* decay, int ld_decay,
-                         const float* a_log, const float* dt_bias, float* state, long slot_stride, const int* slot, const int* row0, const int* len,
+                         int decay_ready, const float* a_log, const float* dt_bias, float* state, long slot_stride, const int* slot, const int* row0, const int* len,
                          float* out, int heads, int kv_heads, int dim, int vdim, int entries, int f32, pk_stream st);
+/* z [tokens, heads * dim] <- those decays, in place (many tokens: once, instead of in every CTA that reads them) */
+int pk_channel_decay(float* z, const float* a_log, const float* dt_bias, int tokens, int heads, int dim, pk_stream st);
 /* Real-gated linear recurrent unit, one scalar of state per channel: r = logistic(z_r + r_bias), i = logistic(z_i + i_bias), log a = -rate * r * softplus(lam),
  * S <- a S + sqrt(1 - a^2) i u,  out = S * gelu_tanh(y + y_bias) (y_bias element type, may be NULL).  z [tokens, ldz] fp32: block b of n = channels / blocks
  * channels has z_r at b * 2n + j and z_i at b * 2n + n + j. */

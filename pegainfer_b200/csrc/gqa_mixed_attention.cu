@@ -10,6 +10,7 @@
 //   mixed_attention_mma_kernel   bf16 prompt portions on the tensor cores: 16 query rows of every head per CTA.
 //   mixed_attention_merge_kernel adds the shares' partial sums and applies the gate.
 #include <algorithm>
+#include <type_traits>
 
 #include "common.cuh"
 #include "mma.cuh"
@@ -151,7 +152,13 @@ constexpr int kMxHS = kMxRows * kMxLS + 4;
 constexpr int kMxLP = kMxKeys + 8;                      // bf16 per weight row; head stride 4 mod 32 words
 constexpr int kMxHP = kMxRows * kMxLP + 8;
 
-__device__ __forceinline__ float fast_logistic(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+// logistic of z from z2 = -z * log2(e), on the special-function unit (relative error of a few 2^-22; 2^z2 = inf gives 0)
+__device__ __forceinline__ float fast_logistic2(float z2) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(z2));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(e + 1.f));
+  return r;
+}
 // x = hi + mid + lo, each a bf16: the pair (x0, x1) as three packed registers
 __device__ __forceinline__ void split3(float x0, float x1, uint32_t& hi, uint32_t& mid, uint32_t& lo) {
   hi = pack_bf16(x0, x1);
@@ -219,14 +226,17 @@ __global__ void __launch_bounds__(256, 1) mixed_attention_mma_kernel(MixedArgs a
       ta[kk][3] = pack_bf16(m(h + 8, g + 8), m(h + 8, g + 9));
     }
   }
-  const float bias_a = a.bias && gq < nh ? a.bias[h_base + gq] : 0.f, bias_b = a.bias && gq + 8 < nh ? a.bias[h_base + gq + 8] : 0.f;
+  constexpr float kNegLog2e = -1.4426950408889634f;
+  const float scale2 = a.scale * kNegLog2e;  // mixed raw score -> argument of fast_logistic2
+  const float bias_a = a.bias && gq < nh ? a.bias[h_base + gq] * kNegLog2e : 0.f, bias_b = a.bias && gq + 8 < nh ? a.bias[h_base + gq + 8] * kNegLog2e : 0.f;
   float o[HPW][DV / 8][4] = {};
   int r_first = 0;
   while (r_first < kMxRows && s_req[r_first] >= 0) {
     const int rq = s_req[r_first];
     int r_last = r_first;
     while (r_last + 1 < kMxRows && s_req[r_last + 1] == rq) ++r_last;
-    const int p_max = s_pos[r_last];
+    const int p_max = s_pos[r_last], p_min = s_pos[r_first];
+    const bool whole_tile = r_first == 0 && r_last == kMxRows - 1;
     const int* pg = a.pages + a.page_off[rq];
     const int n_blocks = p_max / kMxKeys + 1, per_split = (n_blocks + a.splits - 1) / a.splits;
     const int b0 = split * per_split, b_end = min(n_blocks, b0 + per_split);
@@ -292,9 +302,9 @@ __global__ void __launch_bounds__(256, 1) mixed_attention_mma_kernel(MixedArgs a
         }
       }
     };
-    auto weights = [&](int b) {  // step 2
+    auto weights = [&](int b, auto masked) {  // step 2; masked: some key of the block is hidden from some row of the tile
       const int k0 = b * kMxKeys;
-#pragma unroll 2
+#pragma unroll 4
       for (int nt = warp; nt < kMxRows * (kMxKeys / 8); nt += nw) {
         const int r = nt / (kMxKeys / 8), ko = (nt % (kMxKeys / 8)) * 8;
         const float* src = S + r * kMxLS + ko + gq;
@@ -303,8 +313,8 @@ __global__ void __launch_bounds__(256, 1) mixed_attention_mma_kernel(MixedArgs a
         for (int kk = 0; kk < NK; ++kk) {
           if (kk * 16 < H) {
             const int g = kk * 16 + 2 * tq;
-            const float x0 = g < H ? src[(size_t)g * kMxHS] : 0.f, x1 = g + 1 < H ? src[(size_t)(g + 1) * kMxHS] : 0.f;
-            const float x2 = g + 8 < H ? src[(size_t)(g + 8) * kMxHS] : 0.f, x3 = g + 9 < H ? src[(size_t)(g + 9) * kMxHS] : 0.f;
+            const float x0 = g < H ? src[g * kMxHS] : 0.f, x1 = g + 1 < H ? src[(g + 1) * kMxHS] : 0.f;
+            const float x2 = g + 8 < H ? src[(g + 8) * kMxHS] : 0.f, x3 = g + 9 < H ? src[(g + 9) * kMxHS] : 0.f;
             uint32_t hi[2], mid[2], lo[2];
             split3(x0, x1, hi[0], mid[0], lo[0]);
             split3(x2, x3, hi[1], mid[1], lo[1]);
@@ -313,11 +323,14 @@ __global__ void __launch_bounds__(256, 1) mixed_attention_mma_kernel(MixedArgs a
             mma_bf16_16816(z, ta[kk], hi[0], hi[1]);
           }
         }
-        const bool on = s_req[r] == rq;
-        const int seen = s_pos[r] - k0 - ko - 2 * tq;  // keys 2 tq + c of this group of eight are visible for c <= seen
-        const float w0 = on && seen >= 0 ? fast_logistic(fmaf(z[0], a.scale, bias_a)) : 0.f, w1 = on && seen >= 1 ? fast_logistic(fmaf(z[1], a.scale, bias_a)) : 0.f;
-        const float w2 = on && seen >= 0 ? fast_logistic(fmaf(z[2], a.scale, bias_b)) : 0.f, w3 = on && seen >= 1 ? fast_logistic(fmaf(z[3], a.scale, bias_b)) : 0.f;
-        bf16* d = P + (size_t)gq * kMxHP + r * kMxLP + ko + 2 * tq;
+        float w0 = fast_logistic2(fmaf(z[0], scale2, bias_a)), w1 = fast_logistic2(fmaf(z[1], scale2, bias_a));
+        float w2 = fast_logistic2(fmaf(z[2], scale2, bias_b)), w3 = fast_logistic2(fmaf(z[3], scale2, bias_b));
+        if (masked) {
+          const int seen = s_req[r] == rq ? s_pos[r] - k0 - ko - 2 * tq : -1;  // keys 2 tq + c of this group of eight are visible for c <= seen
+          if (seen < 0) w0 = w2 = 0.f;
+          if (seen < 1) w1 = w3 = 0.f;
+        }
+        bf16* d = P + gq * kMxHP + r * kMxLP + ko + 2 * tq;
         if (gq < nh) *reinterpret_cast<uint32_t*>(d) = pack_bf16(w0, w1);
         if (gq + 8 < nh) *reinterpret_cast<uint32_t*>(d + 8 * kMxHP) = pack_bf16(w2, w3);
       }
@@ -366,7 +379,8 @@ __global__ void __launch_bounds__(256, 1) mixed_attention_mma_kernel(MixedArgs a
         __syncthreads();  // this block's scores are complete; nobody reads the other stage or the weights any more
         if (more && stages == 2) load(b + 1);
         if (more) find(b + 2);  // the offsets of block b were read before the barrier above
-        weights(b);
+        if (whole_tile && (b + 1) * kMxKeys <= p_min + 1) weights(b, std::false_type{});
+        else weights(b, std::true_type{});
         if (stages == 2) cp_async_wait_all();
         __syncthreads();  // weights complete, block b + 1 has landed (two stages)
         values(b);
@@ -432,12 +446,11 @@ __global__ void mixed_attention_merge_kernel(MixedArgs a) {
   static_cast<E*>(a.out)[(size_t)t * a.out_ld + i] = from_f<E>(s * f);
 }
 
-static inline void fit_splits(MixedArgs& a) {  // partial sums must fit into the thread's scratch buffer
-  ThreadState& ts = tls();
+static inline void fit_splits(MixedArgs& a, float* ws, size_t ws_bytes) {  // partial sums must fit into the workspace
   const size_t one = (size_t)a.T * a.H * a.vdim * sizeof(float);
-  if (!ts.scratch) a.splits = 1;
-  while (a.splits > 1 && one * a.splits > ts.scratch_bytes) --a.splits;
-  a.part = static_cast<float*>(ts.scratch);
+  if (!ws) a.splits = 1;
+  while (a.splits > 1 && one * a.splits > ws_bytes) --a.splits;
+  a.part = ws;
 }
 
 template <typename E>
@@ -446,7 +459,7 @@ static void launch_merge(const MixedArgs& a, cudaStream_t st) {
 }
 
 template <int DQ, int DV, int HPW, int NK>
-static int launch_mixed_mma(MixedArgs a, int max_kv, cudaStream_t st) {
+static int launch_mixed_mma(MixedArgs a, int max_kv, float* ws, size_t ws_bytes, cudaStream_t st) {
   const int tok = a.G * (a.dim + a.vdim);
   const size_t stage = (size_t)kMxKeys * (tok + 8) * 2, rest = (size_t)a.H * kMxHS * 4 + (size_t)16 * kMxHP * 2;
   const size_t limit = 220 * 1024;
@@ -460,19 +473,18 @@ static int launch_mixed_mma(MixedArgs a, int max_kv, cudaStream_t st) {
   }
   const int tiles = (a.T + kMxRows - 1) / kMxRows, slices = (a.H + 15) / 16;
   const int warps = std::min(8, (std::min(16, a.H) + HPW - 1) / HPW);
-  // shares of the key axis: enough CTAs for every SM, and for a long prompt two shares per tile, so that the tiles with the most keys
-  // do not run on alone; a share is at least four blocks
+  // shares of the key axis: about three CTAs per SM, so that the tiles with the most keys do not run on alone; a share is at least four blocks
   const int span = max_kv > 0 ? max_kv : a.T, blocks = (span + kMxKeys - 1) / kMxKeys;
-  const int want = std::max(2, (sm_count() + tiles * slices - 1) / (tiles * slices));
+  const int want = (3 * sm_count() + tiles * slices - 1) / (tiles * slices);
   a.splits = std::max(1, std::min({want, blocks / 4, 32}));
-  fit_splits(a);
+  fit_splits(a, ws, ws_bytes);
   launch(mixed_attention_mma_kernel<DQ, DV, HPW, NK>, dim3(tiles, a.splits, slices), dim3(warps * 32), stages * stage + rest, st, true, a, stages);
   if (a.splits > 1) launch_merge<bf16>(a, st);
   return (int)cudaGetLastError();
 }
 
 template <typename E>
-static int launch_mixed(MixedArgs a, int max_kv, cudaStream_t st) {
+static int launch_mixed(MixedArgs a, int max_kv, float* ws, size_t ws_bytes, cudaStream_t st) {
   int kb = 32;
   while (kb > 4 && mixed_smem(a.H, a.G, a.dim, a.vdim, kb) > 100 * 1024) kb /= 2;
   const size_t smem = mixed_smem(a.H, a.G, a.dim, a.vdim, kb);
@@ -486,7 +498,7 @@ static int launch_mixed(MixedArgs a, int max_kv, cudaStream_t st) {
   }
   const int blocks = max_kv > 0 ? (max_kv + kb - 1) / kb : 1;
   a.splits = std::max(1, std::min({(2 * sm_count() + a.T - 1) / a.T, blocks, 128}));
-  fit_splits(a);
+  fit_splits(a, ws, ws_bytes);
   launch(mixed_attention_kernel<E>, dim3(a.T, a.splits), dim3(256), smem, st, true, a, kb);
   if (a.splits > 1) launch_merge<E>(a, st);
   return (int)cudaGetLastError();
@@ -499,9 +511,9 @@ using namespace pk;
 extern "C" int pk_gqa_mixed_attention(const void* q, const void* cache, const void* score_mix, const float* head_bias, const float* gate, int gate_ld,
                                       const int* positions, const int* req, const int* page_off, const int* pages, void* out, int out_ld,
                                       float out_scale, long page_stride, int page_size, int tokens, int heads, int kv_heads, int dim, int vdim,
-                                      float scale, int max_kv_len, int f32, pk_stream st) {
+                                      float scale, int max_kv_len, void* workspace, long workspace_bytes, int f32, pk_stream st) {
   if (!q || !cache || !positions || !req || !page_off || !pages || !out || tokens <= 0 || heads <= 0 || kv_heads <= 0 || heads % kv_heads || dim <= 0 ||
-      vdim <= 0 || page_size <= 0 || out_ld < heads * vdim || max_kv_len < 0)
+      vdim <= 0 || page_size <= 0 || out_ld < heads * vdim || max_kv_len < 0 || workspace_bytes < 0)
     return -1;
   MixedArgs a{q, cache, score_mix, head_bias, gate, positions, req, page_off, pages, out, nullptr, page_stride, gate_ld, out_ld, page_size, tokens, heads,
               kv_heads, dim, vdim, 1, scale, out_scale};
@@ -510,13 +522,13 @@ extern "C" int pk_gqa_mixed_attention(const void* q, const void* cache, const vo
   if (!f32 && tokens >= 16 && aligned && dim % 16 == 0 && vdim % 16 == 0 && dim <= 128 && vdim <= 128 && heads <= 16 * kMxMaxK) {
     int rc;
 #define PK_MX(DQ, DV)                                                            \
-  (heads > 16  ? launch_mixed_mma<DQ, DV, 2, kMxMaxK>(a, max_kv_len, st) \
-   : heads > 8 ? launch_mixed_mma<DQ, DV, 2, 1>(a, max_kv_len, st)       \
-               : launch_mixed_mma<DQ, DV, 1, 1>(a, max_kv_len, st))
+  (heads > 16  ? launch_mixed_mma<DQ, DV, 2, kMxMaxK>(a, max_kv_len, static_cast<float*>(workspace), (size_t)workspace_bytes, st) \
+   : heads > 8 ? launch_mixed_mma<DQ, DV, 2, 1>(a, max_kv_len, static_cast<float*>(workspace), (size_t)workspace_bytes, st)       \
+               : launch_mixed_mma<DQ, DV, 1, 1>(a, max_kv_len, static_cast<float*>(workspace), (size_t)workspace_bytes, st))
     if (dim <= 64) rc = vdim <= 64 ? PK_MX(64, 64) : PK_MX(64, 128);
     else rc = vdim <= 64 ? PK_MX(128, 64) : PK_MX(128, 128);
 #undef PK_MX
     if (rc != -2) return rc;
   }
-  return f32 ? launch_mixed<float>(a, max_kv_len, st) : launch_mixed<bf16>(a, max_kv_len, st);
+  return f32 ? launch_mixed<float>(a, max_kv_len, static_cast<float*>(workspace), (size_t)workspace_bytes, st) : launch_mixed<bf16>(a, max_kv_len, static_cast<float*>(workspace), (size_t)workspace_bytes, st);
 }

@@ -137,7 +137,7 @@ struct Lib {
 #define PV_BLOCK24(X) X(pk_gqa_rope_append_ex)
 #define PV_BLOCK4(X)                                                                                                                        \
   X(pk_res32_streams_embed) X(pk_res32_streams_step) X(pk_res32_streams_rows) X(pk_gqa_mixed_attention) X(pk_causal_conv)                  \
-  X(pk_channel_delta_seq) X(pk_lru_seq) X(pk_head_norm_gate_ex) X(pk_gemm_strided_f32out)
+  X(pk_channel_decay) X(pk_channel_delta_seq) X(pk_lru_seq) X(pk_head_norm_gate_ex) X(pk_gemm_strided_f32out)
 #define PV_FN(name) decltype(&::name) name = nullptr;
   PV_COMMON(PV_FN) PV_MOE(PV_FN) PV_DENSE(PV_FN) PV_BLOCK0(PV_FN) PV_BLOCK1(PV_FN) PV_BLOCK2(PV_FN) PV_BLOCK3(PV_FN) PV_BLOCK4(PV_FN)
   PV_BLOCK13(PV_FN) PV_BLOCK14(PV_FN) PV_BLOCK23(PV_FN) PV_BLOCK24(PV_FN)
@@ -222,6 +222,8 @@ struct Model {
   int cap_t = 0, cap_r = 0;
   DeviceBuf h32, big, convo, zs, orec, den;  // block 1: unrounded norm output, stacked projections, conv outputs, few-row fp32, read-out
   DeviceBuf ao2, mix2;                       // mixer 4: the state-space branch's gated read-out and its projection
+  DeviceBuf attn_ws;                         // block 4: partial sums of the attention's key shares
+  long attn_ws_bytes = 0;
   DeviceBuf zc, gbuf, one32;                 // block 4: fp32 decay / gate pre-activations, low-rank read-out gate; the constant 1 (weights of a single stream)
   DeviceBuf x, xa, q, dkv, qa, gate, olat, ao, mix, gu, act, z, ids, wts, hid, yf, sgl, sh, xr, logits_e, logits_f, logits_bf, sampled_d, top1_val,
       top1_states, trail, moe_ws;
@@ -238,7 +240,7 @@ struct Model {
   std::set<GraphKey> seen;
   bool use_graph = true;
   // widest layer
-  int mx_big = 0, mx_conv = 0, mx_small = 0, mx_inner = 0, mx_zc = 0, mx_gbuf = 0, n_streams = 1;
+  int mx_big = 0, mx_conv = 0, mx_small = 0, mx_inner = 0, mx_zc = 0, mx_gbuf = 0, mx_attn = 0, n_streams = 1;
   int mx_q = 0, mx_dkv = 0, mx_qa = 0, mx_h = 0, mx_olat = 0, mx_ao = 0, mx_gu = 0, mx_act = 0, mx_e = 0, mx_top = 0, mx_hid = 0;
 
   bool fail(const std::string& m) {
@@ -357,6 +359,7 @@ bool Model::configure(const ModelCfg& mc, const LayerCfg* lc) {
           nsmall += a.heads;
           mx_q = std::max(mx_q, a.heads * a.dim);
           wide = a.heads * a.vdim;
+          mx_attn = std::max(mx_attn, wide);
         }
         mx_big = std::max(mx_big, nbig);
         mx_small = std::max(mx_small, nsmall);
@@ -1016,6 +1019,10 @@ bool Model::ensure_scratch(int T, int R) {
       ok = h32.alloc_uninit(n * W * 4) && big.alloc_uninit(n * std::max(mx_big, 1) * es) && convo.alloc_uninit(n * std::max(mx_conv, 1) * es) &&
            zs.alloc_uninit(n * std::max(mx_small, 1) * 4) && orec.alloc_uninit(n * std::max(mx_inner, 1) * 4) && zc.alloc_uninit(n * std::max(mx_zc, 1) * 4) &&
            gbuf.alloc_uninit(n * std::max(mx_gbuf, 1) * es);
+    if (ok && c.block_kind == 4 && mx_attn > 0) {  // a few tokens: up to 128 shares of the key axis; prompt portions: up to four
+      attn_ws_bytes = (long)(n <= 256 ? std::min<size_t>(128 * n, 4096) : 4 * n) * mx_attn * 4;
+      ok = attn_ws.alloc_uninit((size_t)attn_ws_bytes);
+    }
     if (ok && c.block_kind == 2) ok = big.alloc_uninit(n * std::max(mx_big, 1) * es) && rgbuf.alloc_uninit(n * W * es);
     if (ok && c.block_kind == 3)
       ok = h32.alloc_uninit(n * W * 4) && big.alloc_uninit(n * std::max(mx_big, 1) * es) && convo.alloc_uninit(n * std::max(mx_conv, 1) * es) &&
@@ -1449,7 +1456,9 @@ bool Model::delta_branch(const Layer& L, const char* rows, int nbig, const float
                                      0, 0, 0, f32, st),
             "decay projection"))
       return false;
-    if (!rc(k.pk_channel_delta_seq(convo.ptr, d.C, 0, d.nq, d.nq + d.nk, small, nsmall, 0, (const float*)zc.ptr, d.H * d.D, (const float*)L.p0_32.ptr,
+    const int ready = T >= kGroupedMinTokens;
+    if (ready && !rc(k.pk_channel_decay((float*)zc.ptr, (const float*)L.p0_32.ptr, (const float*)L.p1_32.ptr, T, d.H, d.D, st), "decays")) return false;
+    if (!rc(k.pk_channel_delta_seq(convo.ptr, d.C, 0, d.nq, d.nq + d.nk, small, nsmall, 0, (const float*)zc.ptr, d.H * d.D, ready, (const float*)L.p0_32.ptr,
                                    (const float*)L.p1_32.ptr, slot0, slot_stride, d_slot, d_row0, d_len, (float*)orec.ptr, d.H, d.G, d.D, d.V, n, f32, st),
             "gated delta rule"))
       return false;
@@ -1521,7 +1530,8 @@ bool Model::run_streams_layer(int li, int T, int max_kv, const int* M, int n) {
               "rotation + cache append"))
         return false;
       if (!rc(k.pk_gqa_mixed_attention(q.ptr, pool_base, L.talk.d.ptr, (const float*)L.p2_32.ptr, (const float*)zs.ptr, nsmall, d_pos, d_req, d_poff, d_pages,
-                                       ao.ptr, ld, a.left_scale, page_stride, c.page_size, T, H, G, a.dim, a.vdim, a.scale, max_kv, f32, st),
+                                       ao.ptr, ld, a.left_scale, page_stride, c.page_size, T, H, G, a.dim, a.vdim, a.scale, max_kv,
+                                       attn_ws.ptr, attn_ws_bytes, f32, st),
               "attention"))
         return false;
     }

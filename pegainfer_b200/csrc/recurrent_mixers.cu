@@ -14,7 +14,7 @@
 //
 // Step layout: entry e of the step owns rows [row0[e], row0[e] + len[e]) of every [tokens, features] buffer (a portion
 // of a prompt or one decoded token) and the state slot slot[e]; a slot's state is `state + slot * slot_stride` floats.
-// Sequence kernels: one CTA per (entry, head, slice of value columns); a column of S lives in the registers of DK / 16
+// Sequence kernels: one CTA per (entry, head, slice of value columns); the delta rule has its own (delta_seq_kernel below).  In the other: a column of S lives in the registers of DK / 16
 // neighbouring lanes (key size padded to the template's DK), tokens run one after the other; per block of 32 tokens all
 // threads first bring q, k, v and the gate inputs into shared memory and turn them into unit vectors / gates.  The matrix
 // memory's normaliser n is one more column with value 1.  Latency-bound per token (48 FMAs and two shuffle reductions per
@@ -106,27 +106,25 @@ struct SeqArgs {
   const float* p2;     // state space: skip weight D [H]  (p0 = A_log, p1 = dt_bias)
   const float* zc;     // delta rule with a decay per key channel: [tokens, ld_zc], pre-activation of (head, channel) at h * dim + d; p1 = dt_bias [H * dim]
   int ld_zc;
+  int zc_ready;        // 1: zc holds the decays themselves
 };
 
-// MODE 0: gated delta rule.  MODE 1: xLSTM matrix memory.  MODE 2: state-space duality (q = C, k = B, v = x; dim = state size).
-// MODE 3: gated delta rule with a decay per key channel (a third vector per token beside k and q).
+// MODE 1: xLSTM matrix memory.  MODE 2: state-space duality (q = C, k = B, v = x; dim = state size).
 // Thread layout: KS = DK / 16 neighbouring lanes share one state column, each holding 16 of its DK entries in registers
 // (entry (m * KS + ks) * 4 + e for m < 4, e < 4, so that the lanes' 16-byte reads of k / q from shared memory fall on
 // consecutive banks); the two dot products per token are finished with log2(KS) shuffles.  128 / KS columns per CTA; the
 // matrix memory's normaliser column rides in one more warp of the head's first CTA.
 template <typename E, int DK, int MODE>
 __global__ void __launch_bounds__(160) recurrent_seq_kernel(SeqArgs a) {
-  constexpr bool DELTA = MODE == 0 || MODE == 3;
-  constexpr int KS = DK / 16, COLS = 128 / KS, TB = (DK <= 128 ? 32 : 16) / (MODE == 3 && DK >= 128 ? 2 : 1), NS = 16;  // NS state entries per thread
+  constexpr int KS = DK / 16, COLS = 128 / KS, TB = DK <= 128 ? 32 : 16, NS = 16;  // NS state entries per thread
   __shared__ __align__(16) float ks[TB][DK];
   __shared__ __align__(16) float qs[TB][DK];
   __shared__ float vs[TB][COLS];
-  __shared__ __align__(16) float gc[MODE == 3 ? TB : 1][MODE == 3 ? DK : 4];  // MODE 3: decay per key channel
-  __shared__ float g0[TB], g1[TB];  // delta: decay, write strength;  memory: log forget gate, log input gate
+  __shared__ float g0[TB], g1[TB];  // memory: log forget gate, log input gate;  state space: decay, step size
   pdl_wait();
   pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
   const int e = blockIdx.x, h = blockIdx.y, kvh = h / (a.H / a.G);
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nw = blockDim.x >> 5;
+  const int tid = threadIdx.x, warp = tid >> 5;
   const int n = a.len[e], r0 = a.row0[e], dim = a.dim, vdim = a.vdim;
   const int cl = tid / KS, ksi = tid % KS;  // column inside the CTA, share of the key axis
   const int col0 = blockIdx.z * COLS, col = col0 + cl;
@@ -202,45 +200,14 @@ __global__ void __launch_bounds__(160) recurrent_seq_kernel(SeqArgs a) {
       }
     } else if (tid < nb) {
       const size_t row = (size_t)(r0 + b0 + tid);
-      const float za = MODE == 3 ? 0.f : a.z[row * a.ldz + a.za_off + h], zb = a.z[row * a.ldz + a.zb_off + h];
-      if (MODE == 3) {
-        g1[tid] = sigmoidf_(zb);
-      } else if (MODE == 0) {  // za: decay projection, zb: write-strength projection
-        g0[tid] = expf(-expf(a.p0[h]) * softplusf_(za + a.p1[h]));
-        g1[tid] = sigmoidf_(zb);
-      } else {  // za: forget gate, zb: input gate
-        g0[tid] = logsigmoidf_(a.cap * tanhf((za + a.p1[h]) / a.cap));
-        g1[tid] = a.cap * tanhf((zb + a.p0[h]) / a.cap);
-      }
-    }
-    if constexpr (MODE == 3) {
-      const float rate = expf(a.p0[h]);
-#pragma unroll 4
-      for (int i = tid; i < nb * DK; i += blockDim.x) {
-        const int tt = i / DK, d = i % DK;
-        gc[tt][d] = d < dim ? expf(-rate * softplusf_(a.zc[(size_t)(r0 + b0 + tt) * a.ld_zc + h * dim + d] + a.p1[h * dim + d])) : 1.f;
-      }
+      const float za = a.z[row * a.ldz + a.za_off + h], zb = a.z[row * a.ldz + a.zb_off + h];  // forget gate, input gate
+      g0[tid] = logsigmoidf_(a.cap * tanhf((za + a.p1[h]) / a.cap));
+      g1[tid] = a.cap * tanhf((zb + a.p0[h]) / a.cap);
     }
     __syncthreads();
-    // 2. unit vectors (delta rule) and the query's scale
-    for (int tt = warp; MODE != 2 && tt < nb; tt += nw) {
-      float qf = qscale, kf = 1.f;
-      if (DELTA) {
-        float qq = 0.f, kk = 0.f;
-        for (int i = lane; i < DK; i += 32) {
-          qq = fmaf(qs[tt][i], qs[tt][i], qq);
-          kk = fmaf(ks[tt][i], ks[tt][i], kk);
-        }
-        qq = warp_sum(qq);
-        kk = warp_sum(kk);
-        qf = qscale / sqrtf(qq + 1e-6f);
-        kf = 1.f / sqrtf(kk + 1e-6f);
-      }
-      for (int i = lane; i < DK; i += 32) {
-        qs[tt][i] *= qf;
-        if (DELTA) ks[tt][i] *= kf;
-      }
-    }
+    // 2. the query's scale
+    if (MODE == 1)
+      for (int i = tid; i < nb * DK; i += blockDim.x) qs[i / DK][i % DK] *= qscale;
     __syncthreads();
     if (warp >= 4 && !(MODE == 1 && blockIdx.z == 0)) continue;  // the extra warp only carries the normaliser
     // 3. the recurrence, token by token (whole warps run it: the shuffles below need every lane)
@@ -251,45 +218,7 @@ __global__ void __launch_bounds__(160) recurrent_seq_kernel(SeqArgs a) {
       const float4* k4p = reinterpret_cast<const float4*>(&ks[tt][0]) + ksi;
       const float4* q4p = reinterpret_cast<const float4*>(&qs[tt][0]) + ksi;
       float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
-      if (DELTA) {
-        const float g = MODE == 0 ? g0[tt] : 1.f, beta = g1[tt];
-        const float4* g4p = reinterpret_cast<const float4*>(&gc[MODE == 3 ? tt : 0][0]) + ksi;
-        float c0 = 0.f, c1 = 0.f, c2 = 0.f, c3 = 0.f;
-#pragma unroll
-        for (int mi = 0; mi < NS / 4; ++mi) {
-          const float4 k4 = k4p[mi * KS];
-          const float4 g4 = MODE == 3 ? g4p[mi * KS] : make_float4(g, g, g, g);
-          S[mi * 4] *= g4.x;
-          S[mi * 4 + 1] *= g4.y;
-          S[mi * 4 + 2] *= g4.z;
-          S[mi * 4 + 3] *= g4.w;
-          c0 = fmaf(S[mi * 4], k4.x, c0);
-          c1 = fmaf(S[mi * 4 + 1], k4.y, c1);
-          c2 = fmaf(S[mi * 4 + 2], k4.z, c2);
-          c3 = fmaf(S[mi * 4 + 3], k4.w, c3);
-        }
-        float kv = (c0 + c1) + (c2 + c3);
-#pragma unroll
-        for (int o = 1; o < KS; o <<= 1) kv += __shfl_xor_sync(0xffffffffu, kv, o);
-        const float u = beta * (vt - kv);
-#pragma unroll
-        for (int mi = 0; mi < NS / 4; ++mi) {
-          const float4 k4 = k4p[mi * KS];
-          const float4 q4 = q4p[mi * KS];
-          S[mi * 4] = fmaf(k4.x, u, S[mi * 4]);
-          S[mi * 4 + 1] = fmaf(k4.y, u, S[mi * 4 + 1]);
-          S[mi * 4 + 2] = fmaf(k4.z, u, S[mi * 4 + 2]);
-          S[mi * 4 + 3] = fmaf(k4.w, u, S[mi * 4 + 3]);
-          o0 = fmaf(S[mi * 4], q4.x, o0);
-          o1 = fmaf(S[mi * 4 + 1], q4.y, o1);
-          o2 = fmaf(S[mi * 4 + 2], q4.z, o2);
-          o3 = fmaf(S[mi * 4 + 3], q4.w, o3);
-        }
-        float o = (o0 + o1) + (o2 + o3);
-#pragma unroll
-        for (int s = 1; s < KS; s <<= 1) o += __shfl_xor_sync(0xffffffffu, o, s);
-        if (is_v && ksi == 0) a.out[row * out_ld + h * vdim + col] = o;
-      } else if (MODE == 2) {
+      if (MODE == 2) {
         const float fa = g0[tt], wb = g1[tt] * vt;
 #pragma unroll
         for (int mi = 0; mi < NS / 4; ++mi) {
@@ -344,6 +273,261 @@ __global__ void __launch_bounds__(160) recurrent_seq_kernel(SeqArgs a) {
       }
     }
     if (MODE == 1 && ksi == 0) m_g[0] = m;
+  }
+}
+
+// ---- gated delta rule.  CTA = (entry, head, COLS value columns), warp-specialised: warps 0-3 run the recurrence, warps 4-7 prepare the next
+// TB tokens meanwhile (unit vectors, gates, k . q) in the other of two shared-memory stages; one barrier per TB tokens.
+// Recurrence: KS = DK / 16 neighbouring lanes share one state column, 16 entries each as eight packed pairs (two-wide fp32 arithmetic), entry
+// (m * KS + ks) * 4 + e for m < 4, e < 4, so that the lanes' 16-byte shared-memory reads fall on consecutive banks.  Both products of a
+// token are taken on the decayed state before the write, o = S^T q = (g S)^T q + (k . q) u, so that their reductions over the lanes overlap and
+// only one of them is on the path to the next token.  CH: one decay per key channel (a third vector per token), else one per head.
+struct F2 {  // a packed pair of floats
+  unsigned long long v;
+};
+__device__ __forceinline__ F2 f2_mul(F2 a, F2 b) {
+  F2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r.v) : "l"(a.v), "l"(b.v));
+  return r;
+}
+__device__ __forceinline__ F2 f2_add(F2 a, F2 b) {
+  F2 r;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r.v) : "l"(a.v), "l"(b.v));
+  return r;
+}
+__device__ __forceinline__ F2 f2_fma(F2 a, F2 b, F2 c) {
+  F2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r.v) : "l"(a.v), "l"(b.v), "l"(c.v));
+  return r;
+}
+__device__ __forceinline__ F2 f2_pack(float lo, float hi) {
+  F2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r.v) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ float2 f2_unpack(F2 a) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(a.v));
+  return r;
+}
+
+constexpr int kDeltaTB = 16;  // tokens per stage
+template <int DK, bool CH>
+constexpr int delta_stage_floats() {
+  return kDeltaTB * (2 * DK + 128 / (DK / 16) + (CH ? DK : 0) + 4);
+}
+
+template <typename E, int DK, bool CH>
+__global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
+  constexpr int KS = DK / 16, COLS = 128 / KS, TB = kDeltaTB, NV = DK / 32, TW = TB / 4;  // TW: tokens a preparing warp handles per stage
+  extern __shared__ __align__(16) float ds_sm[];
+  pdl_wait();
+  pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
+  const int e = blockIdx.x, h = blockIdx.y, kvh = h / (a.H / a.G), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int n = a.len[e], r0 = a.row0[e], dim = a.dim, vdim = a.vdim, col0 = blockIdx.z * COLS;
+  const int n_stages = (n + TB - 1) / TB;
+  auto ks_of = [&](int b) { return ds_sm + (b & 1) * delta_stage_floats<DK, CH>(); };  // k [TB][DK] | q [TB][DK] | v [TB][COLS] | scalars [4][TB] | decays [TB][DK]
+  constexpr int QO = TB * DK, VO = 2 * TB * DK, SO = VO + TB * COLS, GO = SO + 4 * TB;
+  if (warp >= 4) {
+    // ---- preparation
+    const E* X = static_cast<const E*>(a.qkv);
+    const int qo = a.q_off + kvh * dim, ko = a.k_off + kvh * dim, vo = a.v_off + h * vdim + col0, pw = warp - 4, d0 = lane * NV;
+    const float qscale = 1.f / sqrtf((float)dim), rate = expf(a.p0[h]);
+    const bool vec = sizeof(E) == 2 && NV > 1 && ((a.ld | qo | ko | dim) & (NV - 1)) == 0 && (reinterpret_cast<uintptr_t>(X) & (2 * NV - 1)) == 0;
+    auto load_row = [&](const E* p, float* o) {  // entries d0 .. d0 + NV - 1 of a head's row (zero from dim on)
+      if constexpr (sizeof(E) == 2 && NV > 1) {
+        if (vec) {
+          uint32_t u[NV / 2] = {};
+          if (d0 < dim) {
+            if constexpr (NV == 2) u[0] = *reinterpret_cast<const uint32_t*>(p + d0);
+            else if constexpr (NV == 4) *reinterpret_cast<uint2*>(u) = *reinterpret_cast<const uint2*>(p + d0);
+            else *reinterpret_cast<uint4*>(u) = *reinterpret_cast<const uint4*>(p + d0);
+          }
+#pragma unroll
+          for (int i = 0; i < NV / 2; ++i) o[2 * i] = bf16_lo(u[i]), o[2 * i + 1] = bf16_hi(u[i]);
+          return;
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < NV; ++i) o[i] = d0 + i < dim ? to_f(p[d0 + i]) : 0.f;
+    };
+    auto fill = [&](int b) {
+      float* sm = ks_of(b);
+      const int t0 = b * TB, nb = min(TB, n - t0);
+      if (pw == 0 && lane < nb) {
+        const float* z = a.z + (size_t)(r0 + t0 + lane) * a.ldz;
+        if (!CH) sm[SO + lane] = expf(-rate * softplusf_(z[a.za_off + h] + a.p1[h]));
+        sm[SO + TB + lane] = sigmoidf_(z[a.zb_off + h]);
+      }
+      float q[TW][NV], k[TW][NV];
+#pragma unroll
+      for (int i = 0; i < TW; ++i) {
+        const int tt = pw + 4 * i;
+        if (tt < nb) {
+          const E* row = X + (size_t)(r0 + t0 + tt) * a.ld;
+          load_row(row + qo, q[i]);
+          load_row(row + ko, k[i]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < NV; ++j) q[i][j] = k[i][j] = 0.f;
+        }
+      }
+      float g[CH ? TW : 1][NV];
+      if constexpr (CH) {
+#pragma unroll
+        for (int i = 0; i < TW; ++i) {
+          const int tt = pw + 4 * i;
+#pragma unroll
+          for (int j = 0; j < NV; ++j) g[i][j] = tt < nb && d0 + j < dim ? a.zc[(size_t)(r0 + t0 + tt) * a.ld_zc + h * dim + d0 + j] : 0.f;
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < TW; ++i) {
+        const int tt = pw + 4 * i;
+        if (tt < nb)
+          for (int c = lane; c < COLS; c += 32) sm[VO + tt * COLS + c] = col0 + c < vdim ? to_f(X[(size_t)(r0 + t0 + tt) * a.ld + vo + c]) : 0.f;
+      }
+      float qq[TW], kk[TW], kq[TW];
+#pragma unroll
+      for (int i = 0; i < TW; ++i) {
+        qq[i] = kk[i] = kq[i] = 0.f;
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+          qq[i] = fmaf(q[i][j], q[i][j], qq[i]);
+          kk[i] = fmaf(k[i][j], k[i][j], kk[i]);
+          kq[i] = fmaf(k[i][j], q[i][j], kq[i]);
+        }
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+        for (int i = 0; i < TW; ++i) {
+          qq[i] += __shfl_xor_sync(0xffffffffu, qq[i], o);
+          kk[i] += __shfl_xor_sync(0xffffffffu, kk[i], o);
+          kq[i] += __shfl_xor_sync(0xffffffffu, kq[i], o);
+        }
+#pragma unroll
+      for (int i = 0; i < TW; ++i) {
+        const int tt = pw + 4 * i;
+        const float qf = qscale / sqrtf(qq[i] + 1e-6f), kf = 1.f / sqrtf(kk[i] + 1e-6f);
+        if (lane == 0) sm[SO + 2 * TB + tt] = kq[i] * qf * kf;
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+          sm[tt * DK + d0 + j] = k[i][j] * kf;
+          sm[QO + tt * DK + d0 + j] = q[i][j] * qf;
+        }
+        if constexpr (CH) {
+#pragma unroll
+          for (int j = 0; j < NV; ++j) {
+            float v = 1.f;
+            if (tt < nb && d0 + j < dim) v = a.zc_ready ? g[i][j] : expf(-rate * softplusf_(g[i][j] + a.p1[h * dim + d0 + j]));
+            sm[GO + tt * DK + d0 + j] = v;
+          }
+        }
+      }
+    };
+    fill(0);
+    for (int b = 0; b < n_stages; ++b) {
+      __syncthreads();  // stage b is complete, and nobody reads the other one any more
+      if (b + 1 < n_stages) fill(b + 1);
+    }
+    return;
+  }
+  // ---- recurrence
+  const int cl = tid / KS, ksi = tid % KS, col = col0 + cl;
+  const bool on = col < vdim;
+  float* S_g = a.state + (size_t)a.slot[e] * a.slot_stride + (size_t)h * dim * vdim;  // [dim][vdim]
+  F2 S[8];
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+    const int i = ((j >> 1) * KS + ksi) * 4 + (j & 1) * 2;
+    S[j] = f2_pack(on && i < dim ? S_g[(size_t)i * vdim + col] : 0.f, on && i + 1 < dim ? S_g[(size_t)(i + 1) * vdim + col] : 0.f);
+  }
+  const size_t out_ld = (size_t)a.H * vdim;
+  float* out = a.out + (size_t)r0 * out_ld + h * vdim + col;
+  for (int b = 0; b < n_stages; ++b) {
+    __syncthreads();
+    const float* sm = ks_of(b);
+    const int nb = min(TB, n - b * TB);
+#pragma unroll 4
+    for (int tt = 0; tt < nb; ++tt) {
+      const ulonglong2* kp = reinterpret_cast<const ulonglong2*>(sm + tt * DK) + ksi;
+      const ulonglong2* qp = reinterpret_cast<const ulonglong2*>(sm + QO + tt * DK) + ksi;
+      const ulonglong2* gp = reinterpret_cast<const ulonglong2*>(sm + GO + tt * DK) + ksi;
+      const float vt = sm[VO + tt * COLS + cl], beta = sm[SO + TB + tt], kq = sm[SO + 2 * TB + tt];
+      const F2 g1 = CH ? F2{0} : f2_pack(sm[SO + tt], sm[SO + tt]);
+      F2 kk[8], c0{0}, c1{0}, o0{0}, o1{0};
+#pragma unroll
+      for (int m = 0; m < 4; ++m) {
+        const ulonglong2 k2 = kp[m * KS], q2 = qp[m * KS];
+        kk[2 * m].v = k2.x;
+        kk[2 * m + 1].v = k2.y;
+        if constexpr (CH) {
+          const ulonglong2 g2 = gp[m * KS];
+          S[2 * m] = f2_mul(S[2 * m], F2{g2.x});
+          S[2 * m + 1] = f2_mul(S[2 * m + 1], F2{g2.y});
+        } else {
+          S[2 * m] = f2_mul(S[2 * m], g1);
+          S[2 * m + 1] = f2_mul(S[2 * m + 1], g1);
+        }
+        c0 = f2_fma(S[2 * m], kk[2 * m], c0);
+        c1 = f2_fma(S[2 * m + 1], kk[2 * m + 1], c1);
+        o0 = f2_fma(S[2 * m], F2{q2.x}, o0);
+        o1 = f2_fma(S[2 * m + 1], F2{q2.y}, o1);
+      }
+      const float2 c2 = f2_unpack(f2_add(c0, c1)), o2 = f2_unpack(f2_add(o0, o1));
+      float kv = c2.x + c2.y, o = o2.x + o2.y;
+#pragma unroll
+      for (int s = 1; s < KS; s <<= 1) {
+        kv += __shfl_xor_sync(0xffffffffu, kv, s);
+        o += __shfl_xor_sync(0xffffffffu, o, s);
+      }
+      const float u = beta * (vt - kv);
+      const F2 u2 = f2_pack(u, u);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) S[j] = f2_fma(kk[j], u2, S[j]);
+      if (on && ksi == 0) out[(size_t)(b * TB + tt) * out_ld] = fmaf(kq, u, o);
+    }
+  }
+  if (on) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int i = ((j >> 1) * KS + ksi) * 4 + (j & 1) * 2;
+      const float2 v = f2_unpack(S[j]);
+      if (i < dim) S_g[(size_t)i * vdim + col] = v.x;
+      if (i + 1 < dim) S_g[(size_t)(i + 1) * vdim + col] = v.y;
+    }
+  }
+}
+
+template <typename E, int DK, bool CH>
+static void launch_delta_t(const SeqArgs& a, int entries, cudaStream_t st) {
+  constexpr int COLS = 128 / (DK / 16);
+  constexpr size_t smem = 2 * delta_stage_floats<DK, CH>() * sizeof(float);
+  static bool attr_set = false;  // per template instance
+  if (smem > 48 * 1024 && !attr_set) {
+    cudaFuncSetAttribute(delta_seq_kernel<E, DK, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    attr_set = true;
+  }
+  launch(delta_seq_kernel<E, DK, CH>, dim3(entries, a.H, (a.vdim + COLS - 1) / COLS), dim3(256), smem, st, true, a);
+}
+template <typename E, bool CH>
+static int launch_delta(const SeqArgs& a, int entries, cudaStream_t st) {
+  if (a.dim > 256) return -2;
+  if (a.dim <= 32) launch_delta_t<E, 32, CH>(a, entries, st);
+  else if (a.dim <= 64) launch_delta_t<E, 64, CH>(a, entries, st);
+  else if (a.dim <= 128) launch_delta_t<E, 128, CH>(a, entries, st);
+  else launch_delta_t<E, 256, CH>(a, entries, st);
+  return (int)cudaGetLastError();
+}
+
+// z <- exp(-exp(a_log[head]) * softplus(z + dt_bias)) in place, C = heads * dim entries per token
+__global__ void channel_decay_kernel(float* __restrict__ z, const float* __restrict__ a_log, const float* __restrict__ dt_bias, long total, int C, int dim) {
+  pdl_wait();
+  pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
+  for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x) {
+    const int c = (int)(i % C);
+    z[i] = expf(-expf(a_log[c / dim]) * softplusf_(z[i] + dt_bias[c]));
   }
 }
 
@@ -594,17 +778,17 @@ extern "C" int pk_gated_delta_seq(const void* qkv, int ld, int q_off, int k_off,
   if (!seq_args_ok(qkv, z, a_log, dt_bias, state, slot, row0, len, out, heads, kv_heads, dim, vdim, entries)) return -1;
   SeqArgs a{qkv, ld, q_off, k_off, v_off, z, ldz, decay_off, beta_off, a_log, dt_bias, state, slot_stride, slot, row0, len, out, nullptr,
             heads, kv_heads, dim, vdim, 0.f};
-  return f32 ? launch_seq<float, 0>(a, entries, st) : launch_seq<bf16, 0>(a, entries, st);
+  return f32 ? launch_delta<float, false>(a, entries, st) : launch_delta<bf16, false>(a, entries, st);
 }
 
 extern "C" int pk_channel_delta_seq(const void* qkv, int ld, int q_off, int k_off, int v_off, const float* z, int ldz, int beta_off, const float* decay,
-                                    int ld_decay, const float* a_log, const float* dt_bias, float* state, long slot_stride, const int* slot,
+                                    int ld_decay, int decay_ready, const float* a_log, const float* dt_bias, float* state, long slot_stride, const int* slot,
                                     const int* row0, const int* len, float* out, int heads, int kv_heads, int dim, int vdim, int entries, int f32,
                                     pk_stream st) {
   if (!seq_args_ok(qkv, z, a_log, dt_bias, state, slot, row0, len, out, heads, kv_heads, dim, vdim, entries) || !decay || ld_decay < heads * dim) return -1;
   SeqArgs a{qkv, ld, q_off, k_off, v_off, z, ldz, 0, beta_off, a_log, dt_bias, state, slot_stride, slot, row0, len, out, nullptr,
-            heads, kv_heads, dim, vdim, 0.f, nullptr, 0, 0, nullptr, decay, ld_decay};
-  return f32 ? launch_seq<float, 3>(a, entries, st) : launch_seq<bf16, 3>(a, entries, st);
+            heads, kv_heads, dim, vdim, 0.f, nullptr, 0, 0, nullptr, decay, ld_decay, decay_ready};
+  return f32 ? launch_delta<float, true>(a, entries, st) : launch_delta<bf16, true>(a, entries, st);
 }
 
 extern "C" int pk_mlstm_seq(const void* qkv, int ld, int q_off, int k_off, int v_off, const float* z, int ldz, int forget_off, int input_off,
@@ -673,5 +857,12 @@ extern "C" int pk_lru_seq(const void* u, int ld_u, const float* z, int ldz, cons
     if (f32) launch(lru_scan_kernel<float, 8>, g, dim3(512), 0, st, true, a);
     else launch(lru_scan_kernel<bf16, 8>, g, dim3(512), 0, st, true, a);
   }
+  return (int)cudaGetLastError();
+}
+
+extern "C" int pk_channel_decay(float* z, const float* a_log, const float* dt_bias, int tokens, int heads, int dim, pk_stream st) {
+  if (!z || !a_log || !dt_bias || tokens <= 0 || heads <= 0 || dim <= 0) return -1;
+  const long total = (long)tokens * heads * dim;
+  launch(channel_decay_kernel, dim3((unsigned)std::min<long>((total + 255) / 256, 148L * 8)), dim3(256), 0, st, true, z, a_log, dt_bias, total, heads * dim, dim);
   return (int)cudaGetLastError();
 }

@@ -180,9 +180,10 @@ RES32_SIGNATURES = {
     "pk_res32_streams_embed": (i32, [vp] * 7 + [i32, i32, f32, i32, i32, vp]),
     "pk_res32_streams_step": (i32, [vp] * 8 + [i32, i32, f32, i32, i32, vp]),
     "pk_res32_streams_rows": (i32, [vp] * 5 + [i32, i32, f32, i32, i32, vp]),
-    "pk_gqa_mixed_attention": (i32, [vp] * 5 + [i32] + [vp] * 5 + [i32, f32, i64l] + [i32] * 6 + [f32, i32, i32, vp]),
+    "pk_gqa_mixed_attention": (i32, [vp] * 5 + [i32] + [vp] * 5 + [i32, f32, i64l] + [i32] * 6 + [f32, i32, vp, i64l, i32, vp]),
     "pk_causal_conv": (i32, [vp, i32, vp, vp, vp, i32, vp, i64l, vp, vp, vp, vp] + [i32] * 6 + [vp]),
-    "pk_channel_delta_seq": (i32, [vp, i32, i32, i32, i32, vp, i32, i32, vp, i32, vp, vp, vp, i64l, vp, vp, vp, vp] + [i32] * 6 + [vp]),
+    "pk_channel_decay": (i32, [vp, vp, vp, i32, i32, i32, vp]),
+    "pk_channel_delta_seq": (i32, [vp, i32, i32, i32, i32, vp, i32, i32, vp, i32, i32, vp, vp, vp, i64l, vp, vp, vp, vp] + [i32] * 6 + [vp]),
     "pk_lru_seq": (i32, [vp, i32, vp, i32, vp, vp, vp, f32, i32, vp, i32, vp, vp, i64l, vp, vp, vp, vp] + [i32] * 5 + [vp]),
     "pk_head_norm_gate_ex": (i32, [vp, vp, vp, i32, vp, i32, i32, vp, i32, f32, i32, i32, i32, f32, i32, i32, vp]),
     "pk_gemm_strided_f32out": (i32, [vp, vp, vp] + [i32] * 3 + [i64l] * 3 + [i32] + [i64l] * 3 + [i32, vp]),

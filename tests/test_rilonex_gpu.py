@@ -246,9 +246,9 @@ def paged(req_lens, page_size, shuffle_seed=0):
     return pages, off, sum(need) + 3
 
 
-def run_attention(lib, dtype, mx, qkv, talk, pb, gate, starts, lens, ps=16, max_kv=0, factor=1.0):
+def run_attention(lib, dtype, mx, qkv, talk, pb, gate, starts, lens, ps=16, max_kv=0, factor=1.0, shares=8):
     """rotation + cache append + attention for a step whose request r brings positions starts[r] .. lens[r] - 1 (earlier positions
-    were appended by a first call); rows [q | k | v]; talk / pb / gate may be None.  Returns [T, H * vdim]."""
+    were appended by a first call); rows [q | k | v]; talk / pb / gate may be None; the workspace holds `shares` shares of the key axis.  Returns [T, H * vdim]."""
     P = Hold()
     H, G, D, Dv = mx["heads"], mx["kv_heads"], mx["dim"], mx["vdim"]
     n_all = H * D + G * D + G * Dv
@@ -273,9 +273,11 @@ def run_attention(lib, dtype, mx, qkv, talk, pb, gate, starts, lens, ps=16, max_
         gt = torch.cat([gate[r][s:e] for r, (s, e) in enumerate(rows_of)]) if gate is not None else None
         assert lib.pk_gqa_rope_append_ex(P(dev(x, dtype)), n_all, None, *a, qo.data_ptr(), cache.data_ptr(), stride, ps, H, G, D, Dv, dims, 0,
                                          freq.data_ptr() if rot else None, 1.0, 0.0, T, f32, None) == 0
+        ws = torch.zeros(shares * T * H * Dv, device="cuda")
         assert lib.pk_gqa_mixed_attention(qo.data_ptr(), cache.data_ptr(), P(dev(talk, dtype)) if talk is not None else None,
                                           P(pb.cuda()) if pb is not None else None, P(gt.cuda()) if gt is not None else None, H + 2, *a, out.data_ptr(), ld,
-                                          factor, stride, ps, T, H, G, D, Dv, float(mx["scale"]), max_kv, f32, None) == 0
+                                          factor, stride, ps, T, H, G, D, Dv, float(mx["scale"]), max_kv, P(ws) if shares else None,
+                                          4 * ws.numel(), f32, None) == 0
         torch.cuda.synchronize()
         assert (out[:, H * Dv:] == 5.0).all()  # nothing past the heads' columns is written
         return out[:, :H * Dv].float().cpu()
@@ -315,8 +317,8 @@ def test_attention_ragged_batch(lib, dtype, H, G, D, Dv, dims):
     qkv = [rounded(torch.randn(n, (H + G) * D + G * Dv, generator=g), dtype) for n in lens]
     talk = rounded(torch.eye(H) + 0.5 * torch.randn(H, H, generator=g), dtype)
     pb, gate = torch.randn(H, generator=g) - 2.0, [torch.randn(n, H + 2, generator=g) for n in lens]
-    for (t, b, gt, max_kv) in ((talk, pb, gate, 0), (talk, pb, gate, 200), (None, None, None, 200)):
-        got = run_attention(lib, dtype, mx, qkv, t, b, gt, starts, lens, max_kv=max_kv, factor=-1.4)
+    for (t, b, gt, max_kv, shares) in ((talk, pb, gate, 0, 8), (talk, pb, gate, 200, 8), (talk, pb, gate, 200, 0), (None, None, None, 200, 2)):
+        got = run_attention(lib, dtype, mx, qkv, t, b, gt, starts, lens, max_kv=max_kv, factor=-1.4, shares=shares)
         want = torch.cat([oracle_attention(mx, qkv[r], t, b, gt[r] if gt else None, starts[r], lens[r], -1.4) for r in range(3)])
         tol = 4e-5 if dtype == F32 else 2e-2
         assert (got - want).abs().max() < tol * max(1.0, want.abs().max().item()), max_kv
@@ -333,8 +335,8 @@ def test_decoded_tokens_of_unequal_contexts_in_one_launch(lib, dtype, H, G, D):
     qkv = [rounded(torch.randn(n, (H + 2 * G) * D, generator=g), dtype) for n in lens]
     talk, pb = rounded(torch.eye(H) + 0.3 * torch.randn(H, H, generator=g), dtype), torch.full((H,), -5.0)
     want = torch.cat([oracle_attention(mx, qkv[r], talk, pb, None, starts[r], lens[r]) for r in range(3)])
-    for max_kv in (0, 1500, 2048):
-        got = run_attention(lib, dtype, mx, qkv, talk, pb, None, starts, lens, max_kv=max_kv)
+    for max_kv, shares in ((0, 0), (1500, 100), (2048, 7)):
+        got = run_attention(lib, dtype, mx, qkv, talk, pb, None, starts, lens, max_kv=max_kv, shares=shares)
         assert (got - want).abs().max() < (3e-5 if dtype == F32 else 1e-2) * max(1.0, want.abs().max().item()), max_kv
 
 
@@ -520,7 +522,11 @@ def test_delta_rule_in_portions_over_reused_slots(lib, dtype, H, G, D, Dv, per_c
         where = (state.data_ptr(), stride, P(i32([slots[r] for r in live])), P(i32(row0)), P(i32(ns)), out.data_ptr(), H, G, D, Dv, len(ns), int(dtype == F32), None)
         head = (P(dev(rows, dtype)), ld, 8, 8 + nq, 8 + 2 * nq, P(cut(zs).cuda()), ldz)
         if per_channel:
-            assert lib.pk_channel_delta_seq(*head, 1 + H, P(cut(zc).cuda()), ldc, P(a_log.cuda()), P(dt.cuda()), *where) == 0
+            c_d, ready = cut(zc).cuda(), k % 2  # every other step: the decays made by a launch of their own
+            if ready:
+                c_d = c_d[:, :H * D].contiguous()
+                assert lib.pk_channel_decay(P(c_d), P(a_log.cuda()), P(dt.cuda()), T, H, D, None) == 0
+            assert lib.pk_channel_delta_seq(*head, 1 + H, P(c_d), c_d.shape[1], ready, P(a_log.cuda()), P(dt.cuda()), *where) == 0
         else:
             assert lib.pk_gated_delta_seq(*head, 1, 1 + H, P(a_log.cuda()), P(dt.cuda()), *where) == 0
         torch.cuda.synchronize()
