@@ -27,7 +27,7 @@ struct MixedArgs {
   void* out;                                   // E, rows of stride out_ld
   float* part;                                 // [splits][T][H * vdim] when the key axis is split
   long page_stride;
-  int gate_ld, out_ld, page_size, T, H, G, dim, vdim, splits;
+  int gate_ld, out_ld, page_size, T, H, G, dim, vdim, splits, tile_rows;  // tile_rows: rows of a tensor-core CTA that are in use (16, or 1 for decode steps)
   float scale, out_scale;
 };
 
@@ -159,38 +159,51 @@ __device__ __forceinline__ float fast_logistic2(float z2) {
   asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(e + 1.f));
   return r;
 }
-// x = hi + mid + lo, each a bf16: the pair (x0, x1) as three packed registers
+// x = hi + mid + lo exactly, each a bf16 (eight significant bits cut off at a time): the pair (x0, x1) as three packed registers
+__device__ __forceinline__ uint32_t upper_halves(float x0, float x1) { return __byte_perm(__float_as_uint(x0), __float_as_uint(x1), 0x7632); }
 __device__ __forceinline__ void split3(float x0, float x1, uint32_t& hi, uint32_t& mid, uint32_t& lo) {
-  hi = pack_bf16(x0, x1);
-  const float r0 = x0 - bf16_lo(hi), r1 = x1 - bf16_hi(hi);
-  mid = pack_bf16(r0, r1);
-  lo = pack_bf16(r0 - bf16_lo(mid), r1 - bf16_hi(mid));
+  hi = upper_halves(x0, x1);
+  const float r0 = x0 - __uint_as_float(__float_as_uint(x0) & 0xffff0000u), r1 = x1 - __uint_as_float(__float_as_uint(x1) & 0xffff0000u);
+  mid = upper_halves(r0, r1);
+  lo = upper_halves(r0 - __uint_as_float(__float_as_uint(r0) & 0xffff0000u), r1 - __uint_as_float(__float_as_uint(r1) & 0xffff0000u));
 }
 
-template <int DQ, int DV, int HPW, int NK>  // upper bounds of dim and vdim, heads a warp holds, ceil(H / 16) at most
+// DQ, DV: dim and vdim (EXACT: no size tests inside the unrolled products, which the compiler then schedules as one block) or their upper bounds;
+// HPW: heads a warp holds; NK: at least ceil(H / 16)
+// mma_bf16_16816 that the compiler may move among independent work
+__device__ __forceinline__ void mma_free(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+template <int DQ, int DV, int HPW, int NK, bool EXACT>
 __global__ void __launch_bounds__(256, 1) mixed_attention_mma_kernel(MixedArgs a, int stages) {
   extern __shared__ __align__(16) unsigned char mm_smem[];
   __shared__ int s_req[kMxRows], s_pos[kMxRows];
   __shared__ long long s_off[2][kMxKeys];
-  const int H = a.H, G = a.G, dim = a.dim, vdim = a.vdim, per = H / G, tok = G * (dim + vdim), ldt = tok + 8;
+  const int H = a.H, G = a.G, dim = EXACT ? DQ : a.dim, vdim = EXACT ? DV : a.vdim, per = H / G, tok = G * (dim + vdim), ldt = tok + 8;
   bf16* const kv0 = reinterpret_cast<bf16*>(mm_smem);                                      // [stages][keys][ldt]: K of G heads | V of G heads
-  float* const S = reinterpret_cast<float*>(mm_smem + (size_t)stages * kMxKeys * ldt * 2);  // [H][kMxHS]
-  bf16* const P = reinterpret_cast<bf16*>(S + (size_t)H * kMxHS);                          // [16][kMxHP]
+  const int H16 = (H + 15) / 16 * 16;                                                         // scores of the heads H .. H16 - 1 stay zero
+  float* const S = reinterpret_cast<float*>(mm_smem + (size_t)stages * kMxKeys * ldt * 2);  // [H16][kMxHS]
+  bf16* const P = reinterpret_cast<bf16*>(S + (size_t)H16 * kMxHS);                          // [16][kMxHP]
   pdl_wait();
   pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
-  // tiles from the end of the step first: they see the most keys
-  const int t0 = (gridDim.x - 1 - blockIdx.x) * kMxRows, split = blockIdx.y, h_base = blockIdx.z * 16, nh = min(16, H - h_base);
+  // grid (share, tile, head slice); tiles from the end of the step first: they see the most keys
+  const int t0 = (gridDim.y - 1 - blockIdx.y) * a.tile_rows, split = blockIdx.x, h_base = blockIdx.z * 16, nh = min(16, H - h_base);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nw = blockDim.x >> 5, gq = lane >> 2, tq = lane & 3;
   if (tid < kMxRows) {
     const int t = t0 + tid;
-    s_req[tid] = t < a.T ? a.req[t] : -1;
-    s_pos[tid] = t < a.T ? a.pos[t] : -1;
+    const bool on = tid < a.tile_rows && t < a.T;
+    s_req[tid] = on ? a.req[t] : -1;
+    s_pos[tid] = on ? a.pos[t] : -1;
   }
   __syncthreads();
+  for (int i = H * kMxHS + tid; i < H16 * kMxHS; i += blockDim.x) S[i] = 0.f;
   const bf16* q = static_cast<const bf16*>(a.q);
   const bf16* cache = static_cast<const bf16*>(a.cache);
   const int row_a = t0 + gq, row_b = t0 + gq + 8;
-  const bool in_a = row_a < a.T, in_b = row_b < a.T;
+  const bool in_a = gq < a.tile_rows && row_a < a.T, in_b = gq + 8 < a.tile_rows && row_b < a.T;
   uint32_t qa[HPW][DQ / 16][4];
   auto load_q = [&](int i, int h) {
 #pragma unroll
@@ -230,6 +243,11 @@ __global__ void __launch_bounds__(256, 1) mixed_attention_mma_kernel(MixedArgs a
   const float scale2 = a.scale * kNegLog2e;  // mixed raw score -> argument of fast_logistic2
   const float bias_a = a.bias && gq < nh ? a.bias[h_base + gq] * kNegLog2e : 0.f, bias_b = a.bias && gq + 8 < nh ? a.bias[h_base + gq + 8] * kNegLog2e : 0.f;
   float o[HPW][DV / 8][4] = {};
+  // shared-memory addresses of this lane's ldmatrix rows: K fragments, V fragments (transposed), weights
+  const uint32_t kv_at = smem_u32(kv0), stage_bytes = (uint32_t)(kMxKeys * ldt * 2), row16 = (uint32_t)(16 * ldt * 2);
+  const uint32_t k_lane = (uint32_t)((((lane & 7) + ((lane >> 4) & 1) * 8) * ldt + ((lane >> 3) & 1) * 8) * 2);
+  const uint32_t v_lane = (uint32_t)((((lane & 7) + ((lane >> 3) & 1) * 8) * ldt + ((lane >> 4) & 1) * 8 + G * dim) * 2);
+  const uint32_t p_at = smem_u32(P) + (uint32_t)((((lane & 7) + ((lane >> 3) & 1) * 8) * kMxLP + ((lane >> 4) & 1) * 8) * 2);
   int r_first = 0;
   while (r_first < kMxRows && s_req[r_first] >= 0) {
     const int rq = s_req[r_first];
@@ -240,27 +258,64 @@ __global__ void __launch_bounds__(256, 1) mixed_attention_mma_kernel(MixedArgs a
     const int* pg = a.pages + a.page_off[rq];
     const int n_blocks = p_max / kMxKeys + 1, per_split = (n_blocks + a.splits - 1) / a.splits;
     const int b0 = split * per_split, b_end = min(n_blocks, b0 + per_split);
-    auto find = [&](int b) {  // cache offsets of block b's keys (-1: past the last visible key)
-      if (tid < kMxKeys) {
-        const int j = b * kMxKeys + tid;
-        s_off[b & 1][tid] = j <= p_max ? (long long)pg[j / a.page_size] * a.page_stride + (long long)(j % a.page_size) * tok : -1;
-      }
+    auto page_of = [&](int b) {  // page of this thread's key of block b (-1: past the last visible key)
+      const int j = b * kMxKeys + tid;
+      return tid < kMxKeys && j <= p_max ? pg[j / a.page_size] : -1;
+    };
+    auto note = [&](int b, int page) {  // cache offsets of block b's keys
+      if (tid < kMxKeys) s_off[b & 1][tid] = page >= 0 ? (long long)page * a.page_stride + (long long)((b * kMxKeys + tid) % a.page_size) * tok : -1;
     };
     auto load = [&](int b) {  // K | V rows of block b into its stage
-      bf16* dst = kv0 + (size_t)(stages == 2 ? (b & 1) : 0) * kMxKeys * ldt;
-      const int pr = tok / 8;
+      bf16* dst = kv0 + (stages == 2 ? (b & 1) : 0) * kMxKeys * ldt;
       for (int r = warp; r < kMxKeys; r += nw) {
         const long long at = s_off[b & 1][r];
+        bf16* d = dst + r * ldt;
         if (at >= 0) {
-          for (int c = lane; c < pr; c += 32) cp_async16(dst + (size_t)r * ldt + c * 8, cache + at + c * 8);
+          const bf16* src = cache + at;
+#pragma unroll 4
+          for (int c = lane * 8; c < tok; c += 256) cp_async16(d + c, src + c);
         } else {
-          for (int c = lane; c < pr; c += 32) *reinterpret_cast<uint4*>(dst + (size_t)r * ldt + c * 8) = make_uint4(0, 0, 0, 0);
+          for (int c = lane * 8; c < tok; c += 256) *reinterpret_cast<uint4*>(d + c) = make_uint4(0, 0, 0, 0);
         }
       }
       cp_async_commit();
     };
-    auto scores = [&](int b) {  // step 1
-      const bf16* kv = kv0 + (size_t)(stages == 2 ? (b & 1) : 0) * kMxKeys * ldt;
+    // step 1 for the heads from h0 on; one_group: they read the same keys
+    auto scores_of = [&](uint32_t kv, int h0, auto one_group) {
+      const uint32_t k_at = kv + k_lane + (uint32_t)(h0 / per * dim * 2);
+      uint32_t k_of[HPW];
+#pragma unroll
+      for (int i = 0; i < HPW; ++i) k_of[i] = kv + k_lane + (uint32_t)(min((h0 + i) / per, G - 1) * dim * 2);
+      float* const d = S + h0 * kMxHS + gq * kMxLS + 2 * tq;
+#pragma unroll
+      for (int np = 0; np < kMxKeys / 16; ++np) {
+        float s[HPW][2][4] = {};
+#pragma unroll
+        for (int kk = 0; kk < DQ / 16; ++kk) {
+          if (EXACT || kk * 16 < dim) {
+            uint32_t f[4];
+            ldsm_x4_at(f, k_at + np * row16 + kk * 32);
+#pragma unroll
+            for (int i = 0; i < HPW; ++i) {
+              if (i > 0 && !one_group) ldsm_x4_at(f, k_of[i] + np * row16 + kk * 32);
+              mma_bf16_16816(s[i][0], qa[i][kk], f[0], f[1]);
+              mma_bf16_16816(s[i][1], qa[i][kk], f[2], f[3]);
+            }
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < HPW; ++i) {
+          if (h0 + i >= H) continue;
+#pragma unroll
+          for (int ni = 0; ni < 2; ++ni) {
+            *reinterpret_cast<float2*>(d + i * kMxHS + (np * 2 + ni) * 8) = make_float2(s[i][ni][0], s[i][ni][1]);
+            *reinterpret_cast<float2*>(d + i * kMxHS + 8 * kMxLS + (np * 2 + ni) * 8) = make_float2(s[i][ni][2], s[i][ni][3]);
+          }
+        }
+      }
+    };
+    auto scores = [&](int b) {
+      const uint32_t kv = kv_at + (stages == 2 ? (b & 1) : 0) * stage_bytes;
       for (int hb = 0; hb < H; hb += hpb) {
         const int h0 = hb + warp * HPW;
         if (h0 >= H) break;
@@ -268,96 +323,61 @@ __global__ void __launch_bounds__(256, 1) mixed_attention_mma_kernel(MixedArgs a
 #pragma unroll
           for (int i = 0; i < HPW; ++i) load_q(i, h0 + i);
         }
-        float s[HPW][kMxKeys / 8][4] = {};
-        const int g0 = h0 / per;
-        const bool shared_k = HPW == 1 || (h0 + HPW - 1 < H ? (h0 + HPW - 1) / per == g0 : true);
-#pragma unroll
-        for (int kk = 0; kk < DQ / 16; ++kk) {
-          if (kk * 16 < dim) {
-#pragma unroll
-            for (int np = 0; np < kMxKeys / 16; ++np) {
-              uint32_t f[4];
-              const bf16* base = kv + (size_t)(np * 16 + (lane & 7) + ((lane >> 4) & 1) * 8) * ldt + kk * 16 + ((lane >> 3) & 1) * 8;
-              ldsm_x4(f, base + g0 * dim);
-              mma_bf16_16816(s[0][np * 2], qa[0][kk], f[0], f[1]);
-              mma_bf16_16816(s[0][np * 2 + 1], qa[0][kk], f[2], f[3]);
-#pragma unroll
-              for (int i = 1; i < HPW; ++i) {
-                if (!shared_k) ldsm_x4(f, base + min((h0 + i) / per, G - 1) * dim);
-                mma_bf16_16816(s[i][np * 2], qa[i][kk], f[0], f[1]);
-                mma_bf16_16816(s[i][np * 2 + 1], qa[i][kk], f[2], f[3]);
-              }
-            }
-          }
-        }
-#pragma unroll
-        for (int i = 0; i < HPW; ++i) {
-          if (h0 + i >= H) continue;
-          float* d = S + (size_t)(h0 + i) * kMxHS + gq * kMxLS + 2 * tq;
-#pragma unroll
-          for (int ni = 0; ni < kMxKeys / 8; ++ni) {
-            *reinterpret_cast<float2*>(d + ni * 8) = make_float2(s[i][ni][0], s[i][ni][1]);
-            *reinterpret_cast<float2*>(d + 8 * kMxLS + ni * 8) = make_float2(s[i][ni][2], s[i][ni][3]);
-          }
-        }
+        if (HPW == 1 || (h0 + HPW - 1) / per == h0 / per) scores_of(kv, h0, std::true_type{});
+        else scores_of(kv, h0, std::false_type{});
       }
     };
     auto weights = [&](int b, auto masked) {  // step 2; masked: some key of the block is hidden from some row of the tile
       const int k0 = b * kMxKeys;
-#pragma unroll 4
-      for (int nt = warp; nt < kMxRows * (kMxKeys / 8); nt += nw) {
+      for (int nt = warp; nt < a.tile_rows * (kMxKeys / 8); nt += nw) {  // rows not in use: whatever their weights are, their sums are dropped
         const int r = nt / (kMxKeys / 8), ko = (nt % (kMxKeys / 8)) * 8;
-        const float* src = S + r * kMxLS + ko + gq;
-        float z[4] = {0.f, 0.f, 0.f, 0.f};
+        const float* src = S + r * kMxLS + ko + gq + 2 * tq * kMxHS;
+        float z0[4] = {}, z1[4] = {}, z2[4] = {};  // the three terms in accumulators of their own: independent products in flight
 #pragma unroll
         for (int kk = 0; kk < NK; ++kk) {
-          if (kk * 16 < H) {
-            const int g = kk * 16 + 2 * tq;
-            const float x0 = g < H ? src[g * kMxHS] : 0.f, x1 = g + 1 < H ? src[(g + 1) * kMxHS] : 0.f;
-            const float x2 = g + 8 < H ? src[(g + 8) * kMxHS] : 0.f, x3 = g + 9 < H ? src[(g + 9) * kMxHS] : 0.f;
+          if (NK == 1 || kk * 16 < H) {
             uint32_t hi[2], mid[2], lo[2];
-            split3(x0, x1, hi[0], mid[0], lo[0]);
-            split3(x2, x3, hi[1], mid[1], lo[1]);
-            mma_bf16_16816(z, ta[kk], lo[0], lo[1]);
-            mma_bf16_16816(z, ta[kk], mid[0], mid[1]);
-            mma_bf16_16816(z, ta[kk], hi[0], hi[1]);
+            split3(src[kk * 16 * kMxHS], src[(kk * 16 + 1) * kMxHS], hi[0], mid[0], lo[0]);
+            split3(src[(kk * 16 + 8) * kMxHS], src[(kk * 16 + 9) * kMxHS], hi[1], mid[1], lo[1]);
+            mma_free(z0, ta[kk], hi[0], hi[1]);
+            mma_free(z1, ta[kk], mid[0], mid[1]);
+            mma_free(z2, ta[kk], lo[0], lo[1]);
           }
         }
-        float w0 = fast_logistic2(fmaf(z[0], scale2, bias_a)), w1 = fast_logistic2(fmaf(z[1], scale2, bias_a));
-        float w2 = fast_logistic2(fmaf(z[2], scale2, bias_b)), w3 = fast_logistic2(fmaf(z[3], scale2, bias_b));
+        float w[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) w[e] = fast_logistic2(fmaf(z0[e] + (z1[e] + z2[e]), scale2, e < 2 ? bias_a : bias_b));
         if (masked) {
-          const int seen = s_req[r] == rq ? s_pos[r] - k0 - ko - 2 * tq : -1;  // keys 2 tq + c of this group of eight are visible for c <= seen
-          if (seen < 0) w0 = w2 = 0.f;
-          if (seen < 1) w1 = w3 = 0.f;
+          const int seen = s_req[r] == rq ? s_pos[r] - k0 - ko - 2 * tq : -1;  // keys 2 tq + c of this group are visible for c <= seen
+          if (seen < 0) w[0] = w[2] = 0.f;
+          if (seen < 1) w[1] = w[3] = 0.f;
         }
-        bf16* d = P + gq * kMxHP + r * kMxLP + ko + 2 * tq;
-        if (gq < nh) *reinterpret_cast<uint32_t*>(d) = pack_bf16(w0, w1);
-        if (gq + 8 < nh) *reinterpret_cast<uint32_t*>(d + 8 * kMxHP) = pack_bf16(w2, w3);
+        bf16* d = P + gq * kMxHP + r * kMxLP + ko + 2 * tq;  // (heads past the last one: weights that nobody reads)
+        *reinterpret_cast<uint32_t*>(d) = pack_bf16(w[0], w[1]);
+        *reinterpret_cast<uint32_t*>(d + 8 * kMxHP) = pack_bf16(w[2], w[3]);
       }
     };
-    auto values = [&](int b) {  // step 3
-      const bf16* kv = kv0 + (size_t)(stages == 2 ? (b & 1) : 0) * kMxKeys * ldt + G * dim;
-      const int l0 = warp * HPW;
-      if (l0 >= nh) return;
-      const int g0 = (h_base + l0) / per;
-      const bool shared_v = HPW == 1 || (l0 + HPW - 1 < nh ? (h_base + l0 + HPW - 1) / per == g0 : true);
+    auto values_of = [&](uint32_t kv, int l0, auto one_group) {  // step 3 for the heads h_base + l0 and on
+      const uint32_t v_at = kv + v_lane + (uint32_t)((h_base + l0) / per * vdim * 2);
+      uint32_t v_of[HPW], p_of[HPW];
+#pragma unroll
+      for (int i = 0; i < HPW; ++i) {
+        v_of[i] = kv + v_lane + (uint32_t)(min((h_base + l0 + i) / per, G - 1) * vdim * 2);
+        p_of[i] = p_at + (uint32_t)(min(l0 + i, nh - 1) * kMxHP * 2);
+      }
 #pragma unroll
       for (int kk = 0; kk < kMxKeys / 16; ++kk) {
         uint32_t pa[HPW][4];
 #pragma unroll
-        for (int i = 0; i < HPW; ++i)
-          ldsm_x4(pa[i], P + (size_t)min(l0 + i, nh - 1) * kMxHP + ((lane & 7) + ((lane >> 3) & 1) * 8) * kMxLP + kk * 16 + ((lane >> 4) & 1) * 8);
+        for (int i = 0; i < HPW; ++i) ldsm_x4_at(pa[i], p_of[i] + kk * 32);
 #pragma unroll
         for (int np = 0; np < DV / 16; ++np) {
-          if (np * 16 < vdim) {
+          if (EXACT || np * 16 < vdim) {
             uint32_t f[4];
-            const bf16* base = kv + (size_t)(kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * ldt + np * 16 + ((lane >> 4) & 1) * 8;
-            ldsm_x4_trans(f, base + g0 * vdim);
-            mma_bf16_16816(o[0][np * 2], pa[0], f[0], f[1]);
-            mma_bf16_16816(o[0][np * 2 + 1], pa[0], f[2], f[3]);
+            ldsm_x4_trans_at(f, v_at + kk * row16 + np * 32);
 #pragma unroll
-            for (int i = 1; i < HPW; ++i) {
-              if (!shared_v) ldsm_x4_trans(f, base + min((h_base + l0 + i) / per, G - 1) * vdim);
+            for (int i = 0; i < HPW; ++i) {
+              if (i > 0 && !one_group) ldsm_x4_trans_at(f, v_of[i] + kk * row16 + np * 32);
               mma_bf16_16816(o[i][np * 2], pa[i], f[0], f[1]);
               mma_bf16_16816(o[i][np * 2 + 1], pa[i], f[2], f[3]);
             }
@@ -365,10 +385,17 @@ __global__ void __launch_bounds__(256, 1) mixed_attention_mma_kernel(MixedArgs a
         }
       }
     };
+    auto values = [&](int b) {
+      const uint32_t kv = kv_at + (stages == 2 ? (b & 1) : 0) * stage_bytes;
+      const int l0 = warp * HPW;
+      if (l0 >= nh) return;
+      if (HPW == 1 || (h_base + l0 + HPW - 1) / per == (h_base + l0) / per) values_of(kv, l0, std::true_type{});
+      else values_of(kv, l0, std::false_type{});
+    };
     if (b0 < b_end) {
       __syncthreads();  // the previous request's readers are done with every buffer
-      find(b0);
-      find(b0 + 1);
+      note(b0, page_of(b0));
+      note(b0 + 1, page_of(b0 + 1));
       __syncthreads();
       load(b0);
       cp_async_wait_all();
@@ -378,9 +405,10 @@ __global__ void __launch_bounds__(256, 1) mixed_attention_mma_kernel(MixedArgs a
         const bool more = b + 1 < b_end;
         __syncthreads();  // this block's scores are complete; nobody reads the other stage or the weights any more
         if (more && stages == 2) load(b + 1);
-        if (more) find(b + 2);  // the offsets of block b were read before the barrier above
+        const int page = page_of(b + 2);  // the lookup travels while the weights are made
         if (whole_tile && (b + 1) * kMxKeys <= p_min + 1) weights(b, std::false_type{});
         else weights(b, std::true_type{});
+        note(b + 2, page);  // the offsets of block b were read before the barrier above
         if (stages == 2) cp_async_wait_all();
         __syncthreads();  // weights complete, block b + 1 has landed (two stages)
         values(b);
@@ -423,27 +451,59 @@ __global__ void __launch_bounds__(256, 1) mixed_attention_mma_kernel(MixedArgs a
   }
 }
 
-// out = out_scale * logistic(gate) * sum of the shares' partial sums (in share order)
-template <typename E>
-__global__ void mixed_attention_merge_kernel(MixedArgs a) {
+// out = out_scale * logistic(gate) * sum of the shares' partial sums.  CTA = 64 entries of one row x PG groups of shares; a group adds its shares
+// in order and the groups are added in order, so the result does not depend on timing.
+template <typename E, int PG>
+__global__ void __launch_bounds__(64 * PG) mixed_attention_merge_kernel(MixedArgs a) {
+  __shared__ float part[PG][64];
   pdl_wait();
   pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
-  const int t = blockIdx.x, i = blockIdx.y * blockDim.x + threadIdx.x, n = a.H * a.vdim;
+  const int t = blockIdx.x, c = threadIdx.x & 63, grp = threadIdx.x >> 6, i = blockIdx.y * 64 + c, n = a.H * a.vdim;
+  float s = 0.f;
+  if (i < n) {
+    const float* p = a.part + (size_t)t * n + i;
+    const size_t step = (size_t)a.T * n;
+    int sp = grp;
+    for (; sp + 7 * PG < a.splits; sp += 8 * PG) {  // eight independent loads in flight
+      float v[8];
+#pragma unroll
+      for (int u = 0; u < 8; ++u) v[u] = p[(size_t)(sp + u * PG) * step];
+#pragma unroll
+      for (int u = 0; u < 8; ++u) s += v[u];
+    }
+    for (; sp < a.splits; sp += PG) s += p[(size_t)sp * step];
+  }
+  if (PG > 1) {
+    part[grp][c] = s;
+    __syncthreads();
+    if (grp) return;
+#pragma unroll
+    for (int g = 1; g < PG; ++g) s += part[g][c];
+  }
+  if (i >= n) return;
+  const float f = a.gate ? a.out_scale * logistic_exact(a.gate[(size_t)t * a.gate_ld + i / a.vdim]) : a.out_scale;
+  static_cast<E*>(a.out)[(size_t)t * a.out_ld + i] = from_f<E>(s * f);
+}
+
+// the same for a few shares of many rows: four entries per thread, 16-byte loads
+template <typename E>
+__global__ void __launch_bounds__(256) mixed_attention_merge4_kernel(MixedArgs a) {
+  pdl_wait();
+  pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
+  const int t = blockIdx.x, i = (blockIdx.y * 256 + threadIdx.x) * 4, n = a.H * a.vdim;
   if (i >= n) return;
   const float* p = a.part + (size_t)t * n + i;
   const size_t step = (size_t)a.T * n;
-  float s = 0.f;
-  int sp = 0;
-  for (; sp + 8 <= a.splits; sp += 8) {  // eight independent loads in flight
-    float v[8];
-#pragma unroll
-    for (int u = 0; u < 8; ++u) v[u] = p[(size_t)(sp + u) * step];
-#pragma unroll
-    for (int u = 0; u < 8; ++u) s += v[u];
+  float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+  for (int sp = 0; sp < a.splits; ++sp) {
+    const float4 v = *reinterpret_cast<const float4*>(p + (size_t)sp * step);
+    s.x += v.x, s.y += v.y, s.z += v.z, s.w += v.w;
   }
-  for (; sp < a.splits; ++sp) s += p[(size_t)sp * step];
-  const float f = a.gate ? a.out_scale * logistic_exact(a.gate[(size_t)t * a.gate_ld + i / a.vdim]) : a.out_scale;
-  static_cast<E*>(a.out)[(size_t)t * a.out_ld + i] = from_f<E>(s * f);
+  const float f = a.gate ? a.out_scale * logistic_exact(a.gate[(size_t)t * a.gate_ld + i / a.vdim]) : a.out_scale;  // vdim is a multiple of 4
+  E* o = static_cast<E*>(a.out) + (size_t)t * a.out_ld + i;
+  if constexpr (sizeof(E) == 2) *reinterpret_cast<uint2*>(o) = make_uint2(pack_bf16(s.x * f, s.y * f), pack_bf16(s.z * f, s.w * f));
+  else *reinterpret_cast<float4*>(o) = make_float4(s.x * f, s.y * f, s.z * f, s.w * f);
 }
 
 static inline void fit_splits(MixedArgs& a, float* ws, size_t ws_bytes) {  // partial sums must fit into the workspace
@@ -455,30 +515,37 @@ static inline void fit_splits(MixedArgs& a, float* ws, size_t ws_bytes) {  // pa
 
 template <typename E>
 static void launch_merge(const MixedArgs& a, cudaStream_t st) {
-  launch(mixed_attention_merge_kernel<E>, dim3(a.T, (a.H * a.vdim + 127) / 128), dim3(128), 0, st, true, a);
+  const dim3 g(a.T, (a.H * a.vdim + 63) / 64);
+  const bool four = a.vdim % 4 == 0 && a.out_ld % 4 == 0 && (reinterpret_cast<uintptr_t>(a.out) & (4 * sizeof(E) - 1)) == 0 &&
+                    (reinterpret_cast<uintptr_t>(a.part) & 15) == 0;
+  if (a.splits <= 8 && four) launch(mixed_attention_merge4_kernel<E>, dim3(a.T, (a.H * a.vdim + 1023) / 1024), dim3(256), 0, st, true, a);
+  else if (a.splits > 8) launch(mixed_attention_merge_kernel<E, 8>, g, dim3(512), 0, st, true, a);
+  else launch(mixed_attention_merge_kernel<E, 1>, g, dim3(64), 0, st, true, a);
 }
 
-template <int DQ, int DV, int HPW, int NK>
+template <int DQ, int DV, int HPW, int NK, bool EXACT>
 static int launch_mixed_mma(MixedArgs a, int max_kv, float* ws, size_t ws_bytes, cudaStream_t st) {
   const int tok = a.G * (a.dim + a.vdim);
-  const size_t stage = (size_t)kMxKeys * (tok + 8) * 2, rest = (size_t)a.H * kMxHS * 4 + (size_t)16 * kMxHP * 2;
+  const size_t stage = (size_t)kMxKeys * (tok + 8) * 2, rest = (size_t)((a.H + 15) / 16 * 16) * kMxHS * 4 + (size_t)16 * kMxHP * 2;
   const size_t limit = 220 * 1024;
   const int stages = 2 * stage + rest <= limit ? 2 : 1;
   if (stages * stage + rest > limit) return -2;
   static bool attr_set = false;  // per template instance
   if (!attr_set) {
-    if (cudaFuncSetAttribute(mixed_attention_mma_kernel<DQ, DV, HPW, NK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)limit) != cudaSuccess)
+    if (cudaFuncSetAttribute(mixed_attention_mma_kernel<DQ, DV, HPW, NK, EXACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)limit) != cudaSuccess)
       return (int)cudaGetLastError();
     attr_set = true;
   }
-  const int tiles = (a.T + kMxRows - 1) / kMxRows, slices = (a.H + 15) / 16;
+  a.tile_rows = a.T < kMxRows ? 1 : kMxRows;  // decode steps: a CTA per row, or rows of several requests would be walked one after the other
+  const int tiles = (a.T + a.tile_rows - 1) / a.tile_rows, slices = (a.H + 15) / 16;
   const int warps = std::min(8, (std::min(16, a.H) + HPW - 1) / HPW);
-  // shares of the key axis: about three CTAs per SM, so that the tiles with the most keys do not run on alone; a share is at least four blocks
+  // shares of the key axis: a long prompt's tiles in two, so that the ones with the most keys do not run on alone; few tiles: a CTA for every SM; in
+  // a prompt portion a share is at least four blocks
   const int span = max_kv > 0 ? max_kv : a.T, blocks = (span + kMxKeys - 1) / kMxKeys;
-  const int want = (3 * sm_count() + tiles * slices - 1) / (tiles * slices);
-  a.splits = std::max(1, std::min({want, blocks / 4, 32}));
+  const int want = a.tile_rows == 1 ? sm_count() / (tiles * slices) : std::max(2, 2 * sm_count() / (tiles * slices));
+  a.splits = std::max(1, std::min({want, a.tile_rows == 1 ? blocks : blocks / 4, 64}));
   fit_splits(a, ws, ws_bytes);
-  launch(mixed_attention_mma_kernel<DQ, DV, HPW, NK>, dim3(tiles, a.splits, slices), dim3(warps * 32), stages * stage + rest, st, true, a, stages);
+  launch(mixed_attention_mma_kernel<DQ, DV, HPW, NK, EXACT>, dim3(a.splits, tiles, slices), dim3(warps * 32), stages * stage + rest, st, true, a, stages);
   if (a.splits > 1) launch_merge<bf16>(a, st);
   return (int)cudaGetLastError();
 }
@@ -516,17 +583,18 @@ extern "C" int pk_gqa_mixed_attention(const void* q, const void* cache, const vo
       vdim <= 0 || page_size <= 0 || out_ld < heads * vdim || max_kv_len < 0 || workspace_bytes < 0)
     return -1;
   MixedArgs a{q, cache, score_mix, head_bias, gate, positions, req, page_off, pages, out, nullptr, page_stride, gate_ld, out_ld, page_size, tokens, heads,
-              kv_heads, dim, vdim, 1, scale, out_scale};
+              kv_heads, dim, vdim, 1, kMxRows, scale, out_scale};
   const bool aligned = ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache)) & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 3) == 0 &&
                        page_stride % 8 == 0 && out_ld % 2 == 0;
-  if (!f32 && tokens >= 16 && aligned && dim % 16 == 0 && vdim % 16 == 0 && dim <= 128 && vdim <= 128 && heads <= 16 * kMxMaxK) {
+  if (!f32 && aligned && dim % 16 == 0 && vdim % 16 == 0 && dim <= 128 && vdim <= 128 && heads <= 16 * kMxMaxK) {
     int rc;
-#define PK_MX(DQ, DV)                                                            \
-  (heads > 16  ? launch_mixed_mma<DQ, DV, 2, kMxMaxK>(a, max_kv_len, static_cast<float*>(workspace), (size_t)workspace_bytes, st) \
-   : heads > 8 ? launch_mixed_mma<DQ, DV, 2, 1>(a, max_kv_len, static_cast<float*>(workspace), (size_t)workspace_bytes, st)       \
-               : launch_mixed_mma<DQ, DV, 1, 1>(a, max_kv_len, static_cast<float*>(workspace), (size_t)workspace_bytes, st))
-    if (dim <= 64) rc = vdim <= 64 ? PK_MX(64, 64) : PK_MX(64, 128);
-    else rc = vdim <= 64 ? PK_MX(128, 64) : PK_MX(128, 128);
+#define PK_MX(DQ, DV, EX)                                                                                                                  \
+  (heads > 16  ? launch_mixed_mma<DQ, DV, 2, kMxMaxK, EX>(a, max_kv_len, static_cast<float*>(workspace), (size_t)workspace_bytes, st) \
+   : heads > 8 ? launch_mixed_mma<DQ, DV, 2, 1, EX>(a, max_kv_len, static_cast<float*>(workspace), (size_t)workspace_bytes, st)       \
+               : launch_mixed_mma<DQ, DV, 1, 1, EX>(a, max_kv_len, static_cast<float*>(workspace), (size_t)workspace_bytes, st))
+    if (dim == 64 && vdim == 64) rc = PK_MX(64, 64, true);
+    else if (dim == 128 && vdim == 128) rc = PK_MX(128, 128, true);
+    else rc = PK_MX(128, 128, false);
 #undef PK_MX
     if (rc != -2) return rc;
   }

@@ -333,69 +333,75 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
     const E* X = static_cast<const E*>(a.qkv);
     const int qo = a.q_off + kvh * dim, ko = a.k_off + kvh * dim, vo = a.v_off + h * vdim + col0, pw = warp - 4, d0 = lane * NV;
     const float qscale = 1.f / sqrtf((float)dim), rate = expf(a.p0[h]);
-    const bool vec = sizeof(E) == 2 && NV > 1 && ((a.ld | qo | ko | dim) & (NV - 1)) == 0 && (reinterpret_cast<uintptr_t>(X) & (2 * NV - 1)) == 0;
-    auto load_row = [&](const E* p, float* o) {  // entries d0 .. d0 + NV - 1 of a head's row (zero from dim on)
-      if constexpr (sizeof(E) == 2 && NV > 1) {
-        if (vec) {
-          uint32_t u[NV / 2] = {};
-          if (d0 < dim) {
-            if constexpr (NV == 2) u[0] = *reinterpret_cast<const uint32_t*>(p + d0);
-            else if constexpr (NV == 4) *reinterpret_cast<uint2*>(u) = *reinterpret_cast<const uint2*>(p + d0);
-            else *reinterpret_cast<uint4*>(u) = *reinterpret_cast<const uint4*>(p + d0);
-          }
+    // Raw inputs of a stage wait in registers from one barrier to the next, so that their loads' latency is hidden: fetch() issues the loads
+    // of a stage, finish() turns them into what the recurrence reads.
+    constexpr int NW = sizeof(E) == 2 ? (NV + 1) / 2 : NV, VPT = TB * COLS / 128;  // 32-bit words per head row and lane; values per thread
+    const bool vec = ((a.ld | qo | ko | dim) & (NV - 1)) == 0 && (reinterpret_cast<uintptr_t>(X) & (sizeof(E) * NV - 1)) == 0;
+    uint32_t qr[TW][NW], kr[TW][NW];
+    float gr[CH ? TW : 1][NV];
+    E vr[VPT];
+    float za = 0.f, zb = 0.f;
+    const int pt = tid - 128;
+    auto load_row = [&](const E* p, uint32_t* w) {  // entries d0 .. d0 + NV - 1 of a head's row (zero from dim on)
 #pragma unroll
-          for (int i = 0; i < NV / 2; ++i) o[2 * i] = bf16_lo(u[i]), o[2 * i + 1] = bf16_hi(u[i]);
-          return;
+      for (int i = 0; i < NW; ++i) w[i] = 0u;
+      if (vec && NV > 1) {
+        if (d0 >= dim) return;
+        if constexpr (NW == 1) w[0] = *reinterpret_cast<const uint32_t*>(p + d0);
+        else if constexpr (NW == 2) *reinterpret_cast<uint2*>(w) = *reinterpret_cast<const uint2*>(p + d0);
+        else {
+#pragma unroll
+          for (int i = 0; i < NW / 4; ++i) *reinterpret_cast<uint4*>(w + 4 * i) = *reinterpret_cast<const uint4*>(reinterpret_cast<const uint32_t*>(p + d0) + 4 * i);
+        }
+      } else {
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+          if (d0 + j >= dim) continue;
+          if constexpr (sizeof(E) == 2) w[j / 2] |= (uint32_t)*reinterpret_cast<const uint16_t*>(p + d0 + j) << (16 * (j & 1));
+          else w[j] = *reinterpret_cast<const uint32_t*>(p + d0 + j);
+        }
+      }
+    };
+    auto word = [&](const uint32_t* w, int j) {
+      if constexpr (sizeof(E) == 2) return j & 1 ? bf16_hi(w[j / 2]) : bf16_lo(w[j / 2]);
+      else return __uint_as_float(w[j]);
+    };
+    auto fetch = [&](int b) {
+      const int t0 = b * TB, nb = min(TB, n - t0);
+#pragma unroll
+      for (int i = 0; i < TW; ++i) {
+        const int tt = min(pw + 4 * i, nb - 1);  // past the end: the last token once more (never read)
+        const E* row = X + (size_t)(r0 + t0 + tt) * a.ld;
+        load_row(row + qo, qr[i]);
+        load_row(row + ko, kr[i]);
+        if constexpr (CH) {
+#pragma unroll
+          for (int j = 0; j < NV; ++j) gr[i][j] = d0 + j < dim ? a.zc[(size_t)(r0 + t0 + tt) * a.ld_zc + h * dim + d0 + j] : 0.f;
         }
       }
 #pragma unroll
-      for (int i = 0; i < NV; ++i) o[i] = d0 + i < dim ? to_f(p[d0 + i]) : 0.f;
-    };
-    auto fill = [&](int b) {
-      float* sm = ks_of(b);
-      const int t0 = b * TB, nb = min(TB, n - t0);
+      for (int i = 0; i < VPT; ++i) {
+        const int at = pt + 128 * i, tt = min(at / COLS, nb - 1), c = at % COLS;
+        vr[i] = col0 + c < vdim ? X[(size_t)(r0 + t0 + tt) * a.ld + vo + c] : from_f<E>(0.f);
+      }
       if (pw == 0 && lane < nb) {
         const float* z = a.z + (size_t)(r0 + t0 + lane) * a.ldz;
-        if (!CH) sm[SO + lane] = expf(-rate * softplusf_(z[a.za_off + h] + a.p1[h]));
-        sm[SO + TB + lane] = sigmoidf_(z[a.zb_off + h]);
+        if (!CH) za = z[a.za_off + h];
+        zb = z[a.zb_off + h];
       }
-      float q[TW][NV], k[TW][NV];
-#pragma unroll
-      for (int i = 0; i < TW; ++i) {
-        const int tt = pw + 4 * i;
-        if (tt < nb) {
-          const E* row = X + (size_t)(r0 + t0 + tt) * a.ld;
-          load_row(row + qo, q[i]);
-          load_row(row + ko, k[i]);
-        } else {
-#pragma unroll
-          for (int j = 0; j < NV; ++j) q[i][j] = k[i][j] = 0.f;
-        }
-      }
-      float g[CH ? TW : 1][NV];
-      if constexpr (CH) {
-#pragma unroll
-        for (int i = 0; i < TW; ++i) {
-          const int tt = pw + 4 * i;
-#pragma unroll
-          for (int j = 0; j < NV; ++j) g[i][j] = tt < nb && d0 + j < dim ? a.zc[(size_t)(r0 + t0 + tt) * a.ld_zc + h * dim + d0 + j] : 0.f;
-        }
-      }
-#pragma unroll
-      for (int i = 0; i < TW; ++i) {
-        const int tt = pw + 4 * i;
-        if (tt < nb)
-          for (int c = lane; c < COLS; c += 32) sm[VO + tt * COLS + c] = col0 + c < vdim ? to_f(X[(size_t)(r0 + t0 + tt) * a.ld + vo + c]) : 0.f;
-      }
+    };
+    auto finish = [&](int b) {
+      float* sm = ks_of(b);
       float qq[TW], kk[TW], kq[TW];
 #pragma unroll
       for (int i = 0; i < TW; ++i) {
         qq[i] = kk[i] = kq[i] = 0.f;
 #pragma unroll
         for (int j = 0; j < NV; ++j) {
-          qq[i] = fmaf(q[i][j], q[i][j], qq[i]);
-          kk[i] = fmaf(k[i][j], k[i][j], kk[i]);
-          kq[i] = fmaf(k[i][j], q[i][j], kq[i]);
+          const float q = word(qr[i], j), k = word(kr[i], j);
+          qq[i] = fmaf(q, q, qq[i]);
+          kk[i] = fmaf(k, k, kk[i]);
+          kq[i] = fmaf(k, q, kq[i]);
         }
       }
 #pragma unroll
@@ -411,25 +417,53 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
         const int tt = pw + 4 * i;
         const float qf = qscale / sqrtf(qq[i] + 1e-6f), kf = 1.f / sqrtf(kk[i] + 1e-6f);
         if (lane == 0) sm[SO + 2 * TB + tt] = kq[i] * qf * kf;
+        float kd[NV], qd[NV];
 #pragma unroll
         for (int j = 0; j < NV; ++j) {
-          sm[tt * DK + d0 + j] = k[i][j] * kf;
-          sm[QO + tt * DK + d0 + j] = q[i][j] * qf;
+          kd[j] = word(kr[i], j) * kf;
+          qd[j] = word(qr[i], j) * qf;
         }
+        float gd[NV];
         if constexpr (CH) {
 #pragma unroll
           for (int j = 0; j < NV; ++j) {
-            float v = 1.f;
-            if (tt < nb && d0 + j < dim) v = a.zc_ready ? g[i][j] : expf(-rate * softplusf_(g[i][j] + a.p1[h * dim + d0 + j]));
-            sm[GO + tt * DK + d0 + j] = v;
+            gd[j] = gr[i][j];
+            if (d0 + j >= dim) gd[j] = 1.f;
+            else if (!a.zc_ready) gd[j] = expf(-rate * softplusf_(gd[j] + a.p1[h * dim + d0 + j]));
+          }
+        }
+        if constexpr (NV >= 4) {
+#pragma unroll
+          for (int j = 0; j < NV; j += 4) {
+            *reinterpret_cast<float4*>(sm + tt * DK + d0 + j) = make_float4(kd[j], kd[j + 1], kd[j + 2], kd[j + 3]);
+            *reinterpret_cast<float4*>(sm + QO + tt * DK + d0 + j) = make_float4(qd[j], qd[j + 1], qd[j + 2], qd[j + 3]);
+            if constexpr (CH) *reinterpret_cast<float4*>(sm + GO + tt * DK + d0 + j) = make_float4(gd[j], gd[j + 1], gd[j + 2], gd[j + 3]);
+          }
+        } else {
+#pragma unroll
+          for (int j = 0; j < NV; ++j) {
+            sm[tt * DK + d0 + j] = kd[j];
+            sm[QO + tt * DK + d0 + j] = qd[j];
+            if constexpr (CH) sm[GO + tt * DK + d0 + j] = gd[j];
           }
         }
       }
+#pragma unroll
+      for (int i = 0; i < VPT; ++i) sm[VO + pt + 128 * i] = to_f(vr[i]);
+      if (pw == 0 && lane < TB) {
+        if (!CH) sm[SO + lane] = expf(-rate * softplusf_(za + a.p1[h]));
+        sm[SO + TB + lane] = sigmoidf_(zb);
+      }
     };
-    fill(0);
+    fetch(0);
+    finish(0);
+    if (n_stages > 1) fetch(1);
     for (int b = 0; b < n_stages; ++b) {
       __syncthreads();  // stage b is complete, and nobody reads the other one any more
-      if (b + 1 < n_stages) fill(b + 1);
+      if (b + 1 < n_stages) {
+        finish(b + 1);
+        if (b + 2 < n_stages) fetch(b + 2);
+      }
     }
     return;
   }
