@@ -6,9 +6,9 @@
 // any split of the key axis simply add up.  Scores, mixing, weights and sums are fp32; the element type E (bf16 or float) is that of the
 // activations and of the cache.  The mixing couples all heads, so a CTA always works on every head of its rows.
 //   mixed_attention_kernel       one CTA per (query row, share of the keys), any sizes, both element types: keys in blocks through shared
-//                                memory, one thread per (head, key) score.  Decode steps, the fp32 path, odd sizes.
-//   mixed_attention_mma_kernel   bf16 prompt portions on the tensor cores: 16 query rows of every head per CTA.
-//   mixed_attention_merge_kernel adds the shares' partial sums and applies the gate.
+//                                memory, one thread per (head, key) score.  The fp32 path and odd sizes.
+//   mixed_attention_mma_kernel   bf16 on the tensor cores: 16 query rows of every head per CTA (decode steps: one row), and a share of the keys.
+//   mixed_attention_merge_kernel, mixed_attention_merge4_kernel   add the shares' partial sums and apply the gate.
 #include <algorithm>
 #include <type_traits>
 

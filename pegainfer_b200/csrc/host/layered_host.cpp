@@ -50,7 +50,7 @@ namespace pv {
 
 using pq::DeviceBuf;
 
-struct LayerCfg {  // mirrored by ctypes in pegainfer_b200/vamadra.py
+struct LayerCfg {  // mirrored by ctypes in pegainfer_b200/layered.py
   int heads, dim, rot_dim, vdim, kv_rank, kv_from;  // kv_from < 0: the layer owns its cache
   int rot_dims;                                      // rotated entries of the rot_dim slice
   float rot_base, scale;

@@ -14,11 +14,11 @@
 //
 // Step layout: entry e of the step owns rows [row0[e], row0[e] + len[e]) of every [tokens, features] buffer (a portion
 // of a prompt or one decoded token) and the state slot slot[e]; a slot's state is `state + slot * slot_stride` floats.
-// Sequence kernels: one CTA per (entry, head, slice of value columns); the delta rule has its own (delta_seq_kernel below).  In the other: a column of S lives in the registers of DK / 16
-// neighbouring lanes (key size padded to the template's DK), tokens run one after the other; per block of 32 tokens all
-// threads first bring q, k, v and the gate inputs into shared memory and turn them into unit vectors / gates.  The matrix
-// memory's normaliser n is one more column with value 1.  Latency-bound per token (48 FMAs and two shuffle reductions per
-// thread, one warp per scheduler).
+// Sequence kernels: one CTA per (entry, head, slice of value columns); a column of S lives in the registers of DK / 16
+// neighbouring lanes (key size padded to the template's DK), tokens run one after the other.  The delta rule has a kernel of its
+// own, delta_seq_kernel; in recurrent_seq_kernel (matrix memory, state space) all threads first bring q, k, v and the gate inputs of a
+// block of 32 tokens into shared memory.  The matrix memory's normaliser n is one more column with value 1.  Latency-bound per token
+// (48 FMAs and two shuffle reductions per thread, one warp per scheduler).
 #include <algorithm>
 
 #include "common.cuh"
