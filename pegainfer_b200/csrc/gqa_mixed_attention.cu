@@ -178,7 +178,7 @@ __device__ __forceinline__ void mma_free(float (&d)[4], const uint32_t (&a)[4], 
 }
 
 template <int DQ, int DV, int HPW, int NK, bool EXACT>
-__global__ void __launch_bounds__(256, 1) mixed_attention_mma_kernel(MixedArgs a, int stages) {
+__global__ void __launch_bounds__(256, DQ <= 64 && HPW == 1 ? 2 : 1) mixed_attention_mma_kernel(MixedArgs a, int stages) {
   extern __shared__ __align__(16) unsigned char mm_smem[];
   __shared__ int s_req[kMxRows], s_pos[kMxRows];
   __shared__ long long s_off[2][kMxKeys];
@@ -539,10 +539,11 @@ static int launch_mixed_mma(MixedArgs a, int max_kv, float* ws, size_t ws_bytes,
   a.tile_rows = a.T < kMxRows ? 1 : kMxRows;  // decode steps: a CTA per row, or rows of several requests would be walked one after the other
   const int tiles = (a.T + a.tile_rows - 1) / a.tile_rows, slices = (a.H + 15) / 16;
   const int warps = std::min(8, (std::min(16, a.H) + HPW - 1) / HPW);
-  // shares of the key axis: a long prompt's tiles in two, so that the ones with the most keys do not run on alone; few tiles: a CTA for every SM; in
+  constexpr int per_sm = DQ <= 64 && HPW == 1 ? 2 : 1;  // CTAs that share an SM (the kernel's launch bounds)
+  // shares of the key axis: a long prompt's tiles in two (or four), so that the ones with the most keys do not run on alone; few tiles: a CTA for every SM; in
   // a prompt portion a share is at least four blocks
   const int span = max_kv > 0 ? max_kv : a.T, blocks = (span + kMxKeys - 1) / kMxKeys;
-  const int want = a.tile_rows == 1 ? sm_count() / (tiles * slices) : std::max(2, 2 * sm_count() / (tiles * slices));
+  const int want = a.tile_rows == 1 ? sm_count() / (tiles * slices) : std::max(2 * per_sm, 2 * per_sm * sm_count() / (tiles * slices));
   a.splits = std::max(1, std::min({want, a.tile_rows == 1 ? blocks : blocks / 4, 64}));
   fit_splits(a, ws, ws_bytes);
   launch(mixed_attention_mma_kernel<DQ, DV, HPW, NK, EXACT>, dim3(a.splits, tiles, slices), dim3(warps * 32), stages * stage + rest, st, true, a, stages);
