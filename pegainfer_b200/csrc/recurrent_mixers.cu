@@ -537,13 +537,17 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
 template <typename E, int DK, bool CH>
 static void launch_delta_t(const SeqArgs& a, int entries, cudaStream_t st) {
   constexpr int COLS = 128 / (DK / 16);
-  constexpr size_t smem = 2 * delta_stage_floats<DK, CH>() * sizeof(float);
+  constexpr size_t need = 2 * delta_stage_floats<DK, CH>() * sizeof(float), apart = 116 * 1024;
+  const dim3 g(entries, a.H, (a.vdim + COLS - 1) / COLS);
+  // the chain of tokens sets the time, so two CTAs never share an SM while there is one for each: a programmatic launch would otherwise place
+  // them wherever the previous kernel's CTAs have just left
+  const size_t smem = (long)g.x * g.y * g.z <= sm_count() ? (need > apart ? need : apart) : need;
   static bool attr_set = false;  // per template instance
-  if (smem > 48 * 1024 && !attr_set) {
-    cudaFuncSetAttribute(delta_seq_kernel<E, DK, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  if (!attr_set) {
+    cudaFuncSetAttribute(delta_seq_kernel<E, DK, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(need > apart ? need : apart));
     attr_set = true;
   }
-  launch(delta_seq_kernel<E, DK, CH>, dim3(entries, a.H, (a.vdim + COLS - 1) / COLS), dim3(256), smem, st, true, a);
+  launch(delta_seq_kernel<E, DK, CH>, g, dim3(256), smem, st, true, a);
 }
 template <typename E, bool CH>
 static int launch_delta(const SeqArgs& a, int entries, cudaStream_t st) {
