@@ -841,6 +841,26 @@ def _rilonex_sizes():
     return {"w2048": ril(2048, 16, 4, 128, 6 * 1408 + 2816, 128, 32768), "w1024": ril(1024, 8, 2, 64, 2 * 768 + 1536, 64, 32768)}
 
 
+def _vegodra_sizes():
+    """Vegodra stacks of the same width, head count, head size, feed-forward width and vocabulary as the Nagosun stacks of `_nagosun_sizes` (its
+    closest relative: grouped-query and latent attention with dense feed-forwards on the same host): chunked attention, latent attention, gated
+    linear attention (heads shaped like the Rilonex stack's per-channel delta rule), chunked attention on the first layer's keys and values."""
+    def veg(width, heads, kv, dim, ff, lat, rec, vocab, chunk=1024):
+        mlp = {"kind": "dense", "ff": ff}
+        att = {"type": "attention", "mlp": mlp,
+               "mixer": {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "mask": {"size": chunk}, "scale": dim ** -0.5,
+                         "rot": {"dims": dim // 2, "base": 500000.0}}}
+        ldim, lrot, lv, rank, q_rank = lat
+        la = {"type": "latent_attention", "mlp": mlp,
+              "mixer": {"heads": heads, "dim": ldim, "rot_dim": lrot, "vdim": lv, "kv_rank": rank, "q_rank": q_rank, "scale": (ldim + lrot) ** -0.5,
+                        "rot": {"dims": lrot, "base": 10000.0}}}
+        gla = {"type": "gla", "mlp": mlp, "mixer": {"heads": heads, "dim": rec, "vdim": rec, "tau": 12.0}}
+        return {"architecture": "Vegodra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+                "layers": [att, la, gla, dict(att, mixer=dict(att["mixer"], kv_from=0))]}
+    return {"w2048": veg(2048, 16, 8, 128, 6 * 1408 + 2816, (128, 64, 128, 512, 768), 128, 32768),
+            "w1024": veg(1024, 8, 4, 128, 2 * 768 + 1536, (64, 32, 64, 256, 384), 64, 32768)}
+
+
 def _measure_layered(vm, prompts, ctx, med, synthetic_prompt):
     """prefill tok/s per prompt length and decode tok/s at batch 1 and 4 of a model on the layer-list host"""
     res = {}
@@ -870,7 +890,7 @@ def _measure_layered(vm, prompts, ctx, med, synthetic_prompt):
 def run_arch_compare(args):
     """`--arch vamadra`: prefill and decode throughput of the Vamadra path beside the Qwen3 path at equal size.  `--arch risolorn` /
     `--arch nagosun`: that design's path beside both.  `--arch goguzen`: that design's path beside Risolorn's and Qwen3's.  `--arch rilonex`:
-    beside Goguzen's, Risolorn's and Qwen3's.  Wall clock around each public-API call (token ids from the host in, logits / token back out,
+    beside Goguzen's, Risolorn's and Qwen3's.  `--arch vegodra`: beside Nagosun's, Rilonex' and Qwen3's.  Wall clock around each public-API call (token ids from the host in, logits / token back out,
     stream synchronised), median of the repeats after warm-up; between repeats nothing else runs on the GPU.  One JSON line."""
     import torch
     from pegainfer_b200.model import ModelRuntimeConfig, Qwen3Model
@@ -878,7 +898,7 @@ def run_arch_compare(args):
     from pegainfer_b200.vamadra import VamadraConfig, VamadraModel, iter_random_weights as vam_weights
     reps, warm = max(3, min(args.steps, 20)), max(3, min(args.warmup, 5))
     prompts, ctx, dec_steps = [512, 2048], 2048, 32
-    beside = {"vamadra": "qwen3", "goguzen": "risolorn, qwen3", "rilonex": "goguzen, risolorn, qwen3"}.get(args.arch, "vamadra, qwen3")
+    beside = {"vamadra": "qwen3", "goguzen": "risolorn, qwen3", "rilonex": "goguzen, risolorn, qwen3", "vegodra": "nagosun, rilonex, qwen3"}.get(args.arch, "vamadra, qwen3")
     out = {"metric": "prefill_and_decode_tok_s", "arch": args.arch, "beside": beside, "dtype": "bf16",
            "data": "synthetic", "n_gpus": 1,
            "timing": "wall clock around the public API call incl. host->device ids and device->host result, stream synchronised", "sizes": {}}
@@ -898,7 +918,14 @@ def run_arch_compare(args):
         if args.arch_size and name not in args.arch_size.split(","):
             continue
         row = {}
-        if args.arch == "rilonex":
+        if args.arch == "vegodra":
+            from pegainfer_b200.vegodra import VegodraConfig, VegodraModel, iter_random_weights as veg_weights, with_ranks as veg_ranks
+            gcfg_v = VegodraConfig.from_dict(_vegodra_sizes()[name])
+            gcfg_v = veg_ranks(gcfg_v, {f"l{i}.mix.a1": (16, gcfg_v.width) for i in range(len(gcfg_v.layers))})
+            gv = VegodraModel(gcfg_v, veg_weights(gcfg_v, 0, "cuda"), max_tokens=pool_tokens, max_requests=5)
+            row["vegodra"] = _measure_layered(gv, prompts, ctx, med, synthetic_prompt)
+            gv.close()
+        if args.arch in ("rilonex", "vegodra"):
             from pegainfer_b200.rilonex import RilonexConfig, RilonexModel, iter_random_weights as ril_weights, with_ranks
             lcfg_d, rank = _rilonex_sizes()[name]
             lcfg = RilonexConfig.from_dict(lcfg_d)
@@ -919,13 +946,13 @@ def run_arch_compare(args):
             rm = RisolornModel(rcfg, ris_weights(rcfg, 0, "cuda"), max_tokens=pool_tokens, max_requests=5)
             row["risolorn"] = _measure_layered(rm, prompts, ctx, med, synthetic_prompt)
             rm.close()
-        if args.arch == "nagosun":
+        if args.arch in ("nagosun", "vegodra"):
             from pegainfer_b200.nagosun import NagosunConfig, NagosunModel, iter_random_weights as nag_weights
             ncfg = NagosunConfig.from_dict(_nagosun_sizes()[name])
             nm = NagosunModel(ncfg, nag_weights(ncfg, 0, "cuda"), max_tokens=pool_tokens, max_requests=5)
             row["nagosun"] = _measure_layered(nm, prompts, ctx, med, synthetic_prompt)
             nm.close()
-        if args.arch not in ("goguzen", "rilonex"):
+        if args.arch not in ("goguzen", "rilonex", "vegodra"):
             vcfg = VamadraConfig.from_dict(vcfg_d)
             vm = VamadraModel(vcfg, vam_weights(vcfg, 0, "cuda"), max_tokens=pool_tokens, max_requests=5)
             row["vamadra"] = _measure_layered(vm, prompts, ctx, med, synthetic_prompt)
@@ -972,7 +999,7 @@ def main():
     ap.add_argument("--weights", default="cpu", choices=["cpu", "cuda"],
                     help="cpu (default): the seed-0 CPU checkpoint the oracle fixtures were computed on; cuda: generated on "
                          "each GPU (fast; tuning sweeps only -- the parity key then reports a different checkpoint)")
-    ap.add_argument("--arch", default=None, choices=["vamadra", "risolorn", "nagosun", "goguzen", "rilonex"],
+    ap.add_argument("--arch", default=None, choices=["vamadra", "risolorn", "nagosun", "goguzen", "rilonex", "vegodra"],
                     help="instead of the headline workload: prefill / decode throughput of this design beside the closest existing ones at equal size")
     ap.add_argument("--arch-size", default=None, help="with --arch: comma-separated subset of the sizes (w2048,w1024)")
     args = ap.parse_args()

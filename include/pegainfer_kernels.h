@@ -243,6 +243,7 @@ typedef struct {
   void* tp_comm; /* pk_tp_comm*, required for x_mode 2 / epi 2 / epi 3 (tensor parallel) */
   const uint32_t* tp_step; /* epi 3: device word, the decode step counter (same value on every rank) */
   int tp_op;               /* epi 3: index of this collective inside the step (0..254) */
+  int y_ld;                /* gated epilogues: elements from one token's output row to the next (0: M) */
 } pk_b200_gemv_args;
 int pk_b200_gemv_fused(const pk_b200_gemv_args* args, pk_stream stream);
 /* Ring depth (2..12 stages of 8 row segments), CTAs per SM and K elements per row segment (multiple of
@@ -541,10 +542,12 @@ typedef struct pk_attn_extra {
   int window;        /* query at position p sees keys p - window + 1 .. p (combined with `chunk`: the later of the two starts) */
   float softcap;     /* scaled score <- softcap * tanh(score / softcap) */
   float slope_log2;  /* head h subtracts 2^(-slope_log2 (h + 1) / heads) * (p - j) from the (capped) score of key j */
-  const void* gate;  /* element type, rows of stride gate_ld: out[t, h, d] *= logistic(gate[t * gate_ld + h * vdim + d]) */
+  const void* gate;  /* element type, rows of stride gate_ld: out[t, h, d] *= logistic(gate[t * gate_ld + h * vdim + d]) (gate_per_head: [t * gate_ld + h]) */
   long gate_ld;
   int max_kv_len;    /* longest context in the step (0 = unknown): lets a step of few rows split the key axis over CTAs */
   int keep_first;    /* with a window: the first keep_first positions of the sequence stay visible to every later query */
+  int gate_per_head; /* 1: one gate per head instead of one per output entry */
+  long out_ld;       /* elements from one row of out to the next (0: heads * vdim) */
 } pk_attn_extra;
 /* pk_gqa_attention with those options (extra == NULL: none).  A sink of score zero ("one added to the denominator") is a sink vector of zeros. */
 int pk_gqa_attention_ex(const void* q, const void* cache, const void* sink, const int* positions, const int* req, const int* page_off,
@@ -578,13 +581,14 @@ int pk_logits_scale_cap(const void* in, int in_f32, float* out, long n, float sc
 int pk_act_clamped(const void* in, void* out, int F, int tokens, float limit, float slope, int f32, pk_stream st);
 /* What pk_gqa_norm_append does to q and k before they are cached / handed to the attention. */
 typedef struct pk_qk_prep {
-  int norm_kind;         /* 0 none; 1 RMS norm per head, weights [dim] shared by the heads; 2 one RMS norm over the whole projection, weights [heads*dim] / [kv_heads*dim] */
+  int norm_kind;         /* 0 none; 1 RMS norm per head, weights [dim] shared by the heads (both NULL: no weights); 2 one RMS norm over the whole projection, weights [heads*dim] / [kv_heads*dim] */
   const void* q_weight;  /* element type */
   const void* k_weight;
   float eps;
   float temp_coef;       /* q *= 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1) at position p; temp_every 0: no factor */
   int temp_every;
   int values_are_keys;   /* 1: qkv has no v part; the cached values are the keys as projected, before their norm (vdim == dim) */
+  int q_only;            /* 1: qkv is [q] alone (a layer that reads another layer's cache): nothing is cached, the cache arguments may be NULL */
 } pk_qk_prep;
 /* pk_gqa_rope_append without biases and with those steps: norm, then rotation of the first `dims` entries, then the query's factor. */
 int pk_gqa_norm_append(const void* qkv, int ld, const int* positions, const int* req, const int* page_off, const int* pages, void* q_out, void* cache,
@@ -659,8 +663,44 @@ int pk_head_norm_gate_ex(const float* o, const float* den, const void* w, int w_
 /* Strided batched product with fp32 results, both operands contraction-major: C[b*bsC + i*ldc + j] = sum_k A[b*bsA + i*lda + k] * B[b*bsB + j*ldb + k] */
 int pk_gemm_strided_f32out(const void* A, const void* B, float* C, int rows, int cols, int K, long lda, long ldb, long ldc, int batch, long bsA, long bsB,
                            long bsC, int f32, pk_stream st);
-/* pk_b200_gemm_swiglu with a choice of the gate's activation: act 0 SiLU, 1 ReLU (pk_b200_gemv_args.epi 5 is the same for a few tokens) */
+/* pk_b200_gemm_swiglu with a choice of the gate's activation: act 0 SiLU, 1 ReLU, 2 GELU in its tanh form (pk_b200_gemv_args.epi 5 and 6 are the
+ * last two for a few tokens); _ex: output rows of stride ldy */
 int pk_b200_gemm_gated(const pk_bf16* W, const pk_bf16* X, pk_bf16* Y, int M, int N, int K, int act, pk_stream stream);
+int pk_b200_gemm_gated_ex(const pk_bf16* W, const pk_bf16* X, pk_bf16* Y, int M, int N, int K, int ldy, int act, pk_stream stream);
+
+/* =============== parallel blocks under a layer norm, latent queries, gated linear attention ===============
+ * ln(v) = (v - mean) / sqrt(mean((v - mean)^2) + eps) * w + b.  A parallel block feeds h = ln(x) to both sublayers and adds their sum to x. */
+/* x[t] = ln_0(embed[ids[t]]) (weight w0, bias b0);  h[t] = ln(x[t]) with w_next, b_next in the element type (w_next NULL: no h) */
+int pk_res32_embed_lnorm(const void* embed, const int* token_ids, const void* w0, const void* b0, float* x, const void* w_next, const void* b_next, void* h,
+                         int width, float eps, int tokens, int f32, pk_stream st);
+/* x[t] += y[t] (element type);  h[t] = ln(x[t]) as above */
+int pk_res32_add_lnorm(const void* y, float* x, const void* w_next, const void* b_next, void* h, int width, float eps, int tokens, int f32, pk_stream st);
+/* out[r] = ln(x[rows[r]]) in the element type (rows NULL: every row) */
+int pk_res32_lnorm_rows(const float* x, const int* rows, const void* w, const void* b, void* out, int width, float eps, int n_rows, int f32, pk_stream st);
+/* pk_act with output rows of stride ld_out and kind 3: out[t][f] = gelu_tanh(in[t][f]) * in[t][F + f] */
+int pk_act_ex(const void* in, void* out, int ld_out, int F, int tokens, int kind, int f32, pk_stream st);
+/* Latent attention whose queries pass a latent too.  rows [tokens, ld]: q latent (q_rank entries) at q_off, kv latent (rank) and shared rotated key
+ * part (rot) at kv_off.  cq[t] = rms(q latent) * q_norm_w ([tokens, q_rank], element type);  cache append as for pk_latent_kv_append_ex. */
+int pk_latent_prep(const void* rows, int ld, int q_off, int q_rank, const void* q_norm_w, void* cq, int kv_off, const void* kv_norm_w, const int* positions,
+                   const int* req, const int* page_off, const int* pages, void* cache, long page_stride, int page_size, int rank, int rot, int dims,
+                   int interleaved, const float* freq, float mag, float eps, int tokens, int f32, pk_stream st);
+/* Queries folded onto the latent and rotated in one launch: for every head h, qa[t,h,:rank] = q[t,h,:dim] W_uk[h] (uk_t [heads][rank][dim]) and
+ * qa[t,h,rank:] = rotated q[t,h,dim:dim+rot] */
+int pk_latent_query(const void* q, const void* uk_t, void* qa, const int* positions, int tokens, int heads, int dim, int rank, int rot, int dims,
+                    int interleaved, const float* freq, float mag, int f32, pk_stream st);
+/* pk_gemm_strided with an element-wise logistic gate on the result: C[b][i][j] = logistic(gate[b * bs_gate + i * ld_gate + j]) * sum_k A[..] B[..],
+ * both operands contraction-major (B[b * bsB + j * ldb + k]) */
+int pk_gemm_strided_gated(const void* A, const void* B, void* C, const void* gate, int rows, int cols, int K, long lda, long ldb, long ldc, int batch,
+                          long bsA, long bsB, long bsC, long ld_gate, long bs_gate, int f32, pk_stream st);
+/* Gated linear attention over each entry's rows: per head S <- diag(a_t) S + k_t v_t^T, out = S^T (q_t / sqrt(dim)), with a decay per key channel
+ * a = logistic(decay + bias)^(1 / tau).  qkv [tokens, ld] holds q, k (heads x dim) and v (heads x vdim) at the given offsets; decay [tokens, ld_decay]
+ * fp32 the pre-activation of (head, channel) at h * dim + d, or with decay_ready the decays themselves; bias [heads * dim] float.  State S
+ * [heads][dim][vdim] fp32 per slot; out fp32 [tokens, heads * vdim]. */
+int pk_gla_seq(const void* qkv, int ld, int q_off, int k_off, int v_off, const float* decay, int ld_decay, int decay_ready, const float* bias, float tau,
+               float* state, long slot_stride, const int* slot, const int* row0, const int* len, float* out, int heads, int dim, int vdim, int entries,
+               int f32, pk_stream st);
+/* z [tokens, channels] <- logistic(z + bias)^(1 / tau) in place */
+int pk_logistic_decay(float* z, const float* bias, float tau, int tokens, int channels, pk_stream st);
 
 #ifdef __cplusplus
 }

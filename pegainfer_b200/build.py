@@ -52,6 +52,8 @@ PARTS_OF = {
 }
 PARTS_OF["Rilonex"] = (("runtime.cu", "gemm.cu", "gemm2.cu", "gemv.cu", "sampling.cu", "residual32_ops.cu", "gemm_batched_mma.cu", "gqa_attention.cu", "gqa_mixed_attention.cu", "recurrent_mixers.cu"),
                        ("qwen3_host.cpp", "layered_host.cpp"))
+PARTS_OF["Vegodra"] = (("runtime.cu", "gemm.cu", "gemm2.cu", "gemv.cu", "sampling.cu", "residual32_ops.cu", "gemm_batched_mma.cu", "gqa_attention.cu", "latent_attention.cu", "latent_attention_mma.cu", "recurrent_mixers.cu"),
+                       ("qwen3_host.cpp", "layered_host.cpp"))
 PARTS_OF["Goguzen"] = PARTS_OF["Risolorn"]  # the same files: attention, recurrent mixers, experts on the fp32 residual stream
 MANIFEST = os.path.join(OBJ, "linked.txt")
 

@@ -78,6 +78,11 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 // round-trip through bf16 (a reference rounding point kept in a fused kernel)
 __device__ __forceinline__ float round_bf16(float v) { return __bfloat162float(__float2bfloat16(v)); }
 
+// tanh form of GELU, 0.5 z (1 + tanh(u)) with u = sqrt(2 / pi) (z + 0.044715 z^3), as z times the logistic function of 2 u
+__device__ __forceinline__ float gelu_tanh_gate(float z) {
+  return z / (1.f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

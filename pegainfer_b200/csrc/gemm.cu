@@ -355,7 +355,7 @@ static int gemm_impl_mode() {  // 0 tcgen05 (default), 1 simt
 void launch_gemm_seg(const bf16* W, const bf16* X, bf16* Y, bf16* Y1, bf16* Y2, int e0, int e1, int M, int N, int K,
                      cudaStream_t stream);
 // gemm2.cu: the CTA-pair kernel (tcgen05.mma.cta_group::2); -2 = not for this shape
-int launch_gemm_pair(const bf16* W, const bf16* X, bf16* Y, bf16* Y1, bf16* Y2, int e0, int e1, int M, int N, int K, int swiglu,
+int launch_gemm_pair(const bf16* W, const bf16* X, bf16* Y, bf16* Y1, bf16* Y2, int e0, int e1, int M, int N, int K, int swiglu, int ldy,
                      cudaStream_t stream);
 static bool gemm_pair_enabled() {  // PK_GEMM_PAIR=0 keeps the round-1 single-CTA kernel for A/B runs
   static int v = -1;
@@ -376,7 +376,7 @@ void launch_gemm_seg(const bf16* W, const bf16* X, bf16* Y, bf16* Y1, bf16* Y2, 
   const bool tma_ok = K % 8 == 0 && (reinterpret_cast<uintptr_t>(W) & 15) == 0 &&
                       (reinterpret_cast<uintptr_t>(X) & 15) == 0;
   if (tma_ok && gemm_impl_mode() == 0 && gemm_pair_enabled() &&
-      launch_gemm_pair(W, X, Y, Y1, Y2, e0, e1, M, N, K, 0, stream) == 0)
+      launch_gemm_pair(W, X, Y, Y1, Y2, e0, e1, M, N, K, 0, M, stream) == 0)
     return;
   if (tma_ok && gemm_impl_mode() == 0) {
     // Tile width by wave count: tiles = ceil(N/128) * ceil(M/BN) on `sms` persistent CTAs; cost ~ waves * (BN + c).
@@ -442,11 +442,14 @@ extern "C" int pk_b200_gemm_segments(const pk_bf16* W, const pk_bf16* X, pk_bf16
 extern "C" int pk_b200_gemm_swiglu(const pk_bf16* W, const pk_bf16* X, pk_bf16* Y, int M, int N, int K, pk_stream stream) {
   return pk_b200_gemm_gated(W, X, Y, M, N, K, 0, stream);
 }
-// the same with a choice of the gate's activation: 0 SiLU, 1 ReLU
+// the same with a choice of the gate's activation: 0 SiLU, 1 ReLU, 2 GELU (tanh form)
 extern "C" int pk_b200_gemm_gated(const pk_bf16* W, const pk_bf16* X, pk_bf16* Y, int M, int N, int K, int act, pk_stream stream) {
-  if (!W || !X || !Y || M <= 0 || N <= 0 || K <= 0 || act < 0 || act > 1) return -1;
+  return pk_b200_gemm_gated_ex(W, X, Y, M, N, K, M, act, stream);
+}
+extern "C" int pk_b200_gemm_gated_ex(const pk_bf16* W, const pk_bf16* X, pk_bf16* Y, int M, int N, int K, int ldy, int act, pk_stream stream) {
+  if (!W || !X || !Y || M <= 0 || N <= 0 || K <= 0 || ldy < M || act < 0 || act > 2) return -1;
   if (!pk::gemm_pair_enabled() || pk::gemm_impl_mode() != 0) return -2;
-  return pk::launch_gemm_pair((const pk::bf16*)W, (const pk::bf16*)X, (pk::bf16*)Y, (pk::bf16*)Y, (pk::bf16*)Y, M, M, M, N, K, 1 + act, stream);
+  return pk::launch_gemm_pair((const pk::bf16*)W, (const pk::bf16*)X, (pk::bf16*)Y, (pk::bf16*)Y, (pk::bf16*)Y, M, M, M, N, K, 1 + act, ldy, stream);
 }
 
 // Same dispatch as gemm_graphsafe_cuda (gemv.cu): N <= 4 streams the weights (HBM-bound GEMV), larger N runs on the

@@ -91,7 +91,8 @@ struct G2Args {
   bf16 *Y, *Y1, *Y2;
   int e0, e1;     // output segments (the fused q|k|v projection): features [0,e0) -> Y, [e0,e1) -> Y1, rest -> Y2
   int M, N, K;    // features, tokens, reduction
-  int swiglu;     // 1: W = [gate (M rows); up (M rows)], Y[tok][M] = silu(gate) * up; 2: relu(gate) * up
+  int swiglu;     // 1: W = [gate (M rows); up (M rows)], Y[tok][M] = silu(gate) * up; 2: relu(gate) * up; 3: gelu (tanh form) of gate * up
+  int ldy;        // gated output: elements from one token's row to the next
 };
 
 // A pair tile is 256 tokens x (NSUB * BN) features: NSUB accumulators of BN columns side by side in TMEM, one
@@ -218,15 +219,15 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant
           tmem_ld32(t_row + (uint32_t)(HB + c), uv);
           const int f0 = nb * HB + c;
           if (tok < N && f0 < M) {
-            bf16* dst = a.Y + (size_t)tok * M + f0;
+            bf16* dst = a.Y + (size_t)tok * a.ldy + f0;
             float r[32];
 #pragma unroll
             for (int j = 0; j < 32; ++j) {
               const float g = round_bf16(__uint_as_float(gv[j]));  // gate_up_out is bf16 in the reference
               const float u = round_bf16(__uint_as_float(uv[j]));
-              r[j] = (a.swiglu == 2 ? fmaxf(g, 0.f) : g / (1.0f + expf(-g))) * u;
+              r[j] = (a.swiglu == 2 ? fmaxf(g, 0.f) : a.swiglu == 3 ? gelu_tanh_gate(g) : g / (1.0f + expf(-g))) * u;
             }
-            if (M % 8 == 0 && f0 + 32 <= M && (reinterpret_cast<uintptr_t>(a.Y) & 15) == 0) {
+            if (M % 8 == 0 && a.ldy % 8 == 0 && f0 + 32 <= M && (reinterpret_cast<uintptr_t>(a.Y) & 15) == 0) {
 #pragma unroll
               for (int j = 0; j < 4; ++j) {
                 uint4 o;
@@ -358,12 +359,12 @@ static int g2_plan(int M, int N, int K, int swiglu, int sms) {
 }
 
 // Returns 0 when launched, -2 when the shape / alignment is not for this kernel (caller uses the 1-CTA kernel).
-int launch_gemm_pair(const bf16* W, const bf16* X, bf16* Y, bf16* Y1, bf16* Y2, int e0, int e1, int M, int N, int K, int swiglu,
+int launch_gemm_pair(const bf16* W, const bf16* X, bf16* Y, bf16* Y1, bf16* Y2, int e0, int e1, int M, int N, int K, int swiglu, int ldy,
                      cudaStream_t stream) {
   if (K % 8 != 0 || (reinterpret_cast<uintptr_t>(W) & 15) != 0 || (reinterpret_cast<uintptr_t>(X) & 15) != 0) return -2;
   const int best = g2_plan(M, N, K, swiglu, sm_count());
   if (best < 0) return -2;
-  G2Args a{Y, Y1, Y2, e0, e1, M, N, K, swiglu};
+  G2Args a{Y, Y1, Y2, e0, e1, M, N, K, swiglu, ldy};
   CUtensorMap mx, mw;
   if (!g2_make_map(&mx, X, N, K, G2_BM)) return -2;
   const int bn[3] = {256, 160, 128};

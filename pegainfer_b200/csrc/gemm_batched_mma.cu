@@ -1,5 +1,6 @@
 // Strided batched product on the tensor cores (bf16, fp32 accumulation) for the per-head factor products of the latent
-// attention over many tokens: C[b][i][j] = f(row_scale[i*ld_scale + b]) * sum_k A[b*bsA + i*lda + k] * B[b*bsB + j*ldb + k].
+// attention over many tokens: C[b][i][j] = f(row_scale[i*ld_scale + b]) * sum_k A[b*bsA + i*lda + k] * B[b*bsB + j*ldb + k],
+// optionally times logistic(gate[b*bs_gate + i*ld_gate + j]).
 // Both operands are contraction-major, so there are no transposes; 64 x 64 x 32 tiles, 4 warps of 32 x 32, mma.sync
 // m16n8k16, operands through a two-stage cp.async ring (the tile loop of moe_grouped.cu without the row gather).
 // Tensor-bound: 2 * batch * rows * cols * K flop.
@@ -13,7 +14,8 @@ constexpr int kBT = 64, kBK = 32, kBLd = kBK + 8;
 template <typename OUT>  // bf16, or float for products whose result must stay fp32 (router logits, gates)
 __global__ void __launch_bounds__(128) gemm_batched_mma_kernel(const bf16* __restrict__ A, const bf16* __restrict__ B, OUT* __restrict__ C,
                                                               const float* __restrict__ row_scale, int rows, int cols, int K, long lda, long ldb,
-                                                              long ldc, long bsA, long bsB, long bsC, int ld_scale, int scale_kind) {
+                                                              long ldc, long bsA, long bsB, long bsC, int ld_scale, int scale_kind,
+                                                              const bf16* __restrict__ gate, long ld_gate, long bs_gate) {
   __shared__ __align__(16) bf16 As[2][kBT * kBLd];
   __shared__ __align__(16) bf16 Bs[2][kBT * kBLd];
   pdl_wait();
@@ -83,7 +85,12 @@ __global__ void __launch_bounds__(128) gemm_batched_mma_kernel(const bf16* __res
       for (int ni = 0; ni < 4; ++ni) {
         const int j = n0 + wn * 32 + ni * 8 + 2 * tq;
         OUT* o = C + (size_t)i * ldc + j;
-        const float v0 = acc[mi][ni][hf * 2] * s, v1 = acc[mi][ni][hf * 2 + 1] * s;
+        float v0 = acc[mi][ni][hf * 2] * s, v1 = acc[mi][ni][hf * 2 + 1] * s;
+        if (gate) {
+          const bf16* gp = gate + (size_t)bz * bs_gate + (size_t)i * ld_gate + j;
+          if (j < cols) v0 *= __fdividef(1.f, 1.f + __expf(-bf2f(gp[0])));
+          if (j + 1 < cols) v1 *= __fdividef(1.f, 1.f + __expf(-bf2f(gp[1])));
+        }
         if constexpr (sizeof(OUT) == 4) {
           if (j < cols) o[0] = v0;
           if (j + 1 < cols) o[1] = v1;
@@ -100,10 +107,11 @@ __global__ void __launch_bounds__(128) gemm_batched_mma_kernel(const bf16* __res
 
 // 0 = launched, -2 = operands not laid out for this kernel (the caller runs the plain FMA kernel)
 int launch_gemm_batched_mma(const bf16* A, const bf16* B, bf16* C, const float* row_scale, int rows, int cols, int K, long lda, long ldb, long ldc,
-                            int batch, long bsA, long bsB, long bsC, int ld_scale, int scale_kind, cudaStream_t st) {
+                            int batch, long bsA, long bsB, long bsC, int ld_scale, int scale_kind, const bf16* gate, long ld_gate, long bs_gate,
+                            cudaStream_t st) {
   if (K % 8 || lda % 8 || ldb % 8 || bsA % 8 || bsB % 8 || (reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(B) & 15)) return -2;
   const cudaError_t e = launch(gemm_batched_mma_kernel<bf16>, dim3((cols + kBT - 1) / kBT, (rows + kBT - 1) / kBT, batch), dim3(128), 0, st, true, A, B,
-                               C, row_scale, rows, cols, K, lda, ldb, ldc, bsA, bsB, bsC, ld_scale, scale_kind);
+                               C, row_scale, rows, cols, K, lda, ldb, ldc, bsA, bsB, bsC, ld_scale, scale_kind, gate, ld_gate, bs_gate);
   return (int)e;
 }
 
@@ -112,7 +120,7 @@ int launch_gemm_batched_mma_f32(const bf16* A, const bf16* B, float* C, int rows
                                 long bsB, long bsC, cudaStream_t st) {
   if (K % 8 || lda % 8 || ldb % 8 || bsA % 8 || bsB % 8 || (reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(B) & 15)) return -2;
   return (int)launch(gemm_batched_mma_kernel<float>, dim3((cols + kBT - 1) / kBT, (rows + kBT - 1) / kBT, batch), dim3(128), 0, st, true, A, B, C,
-                     (const float*)nullptr, rows, cols, K, lda, ldb, ldc, bsA, bsB, bsC, 0, 0);
+                     (const float*)nullptr, rows, cols, K, lda, ldb, ldc, bsA, bsB, bsC, 0, 0, (const bf16*)nullptr, 0L, 0L);
 }
 
 }  // namespace pk
@@ -124,5 +132,6 @@ extern "C" int pk_proj_rows_f32out(const void* W, const void* xa, float* out, in
   if (!W || !xa || !out || M <= 0 || K <= 0 || tokens <= 0) return -1;
   if (K % 8 || (reinterpret_cast<uintptr_t>(W) & 15) || (reinterpret_cast<uintptr_t>(xa) & 15)) return -2;
   return (int)launch(gemm_batched_mma_kernel<float>, dim3((M + kBT - 1) / kBT, (tokens + kBT - 1) / kBT, 1), dim3(128), 0, st, true, (const bf16*)xa,
-                     (const bf16*)W, out, (const float*)nullptr, tokens, M, K, (long)K, (long)K, (long)M, 0L, 0L, 0L, 0, 0);
+                     (const bf16*)W, out, (const float*)nullptr, tokens, M, K, (long)K, (long)K, (long)M, 0L, 0L, 0L, 0, 0,
+                     (const bf16*)nullptr, 0L, 0L);
 }

@@ -45,6 +45,7 @@ struct GemvArgs {
   int tp_op;                // epi 3: collective index inside the step
   int stages;
   int kc;       // K elements per row segment per stage (multiple of 256); stage = 8 segments
+  int y_ld;     // gated epilogues (1, 4, 5, 6): elements from one token's output row to the next
 };
 
 // 8 bf16 x bf16 products onto `acc`, as two interleaved 4-long FMA chains (ILP: the consumer loop is
@@ -317,9 +318,9 @@ gemv_stream_kernel(const GemvArgs a) {
         for (int n = 0; n < NTOK; ++n) {
           const float gt = round_bf16(acc[n]);                   // gate_up_out is bf16 in the reference
           const float up = round_bf16(sw[warp * NTOK + n]);
-          float sl = a.epi == 5 ? fmaxf(gt, 0.f) : gt / (1.0f + expf(-gt));
+          float sl = a.epi == 5 ? fmaxf(gt, 0.f) : a.epi == 6 ? gelu_tanh_gate(gt) : gt / (1.0f + expf(-gt));
           if (a.epi == 4) sl = round_bf16(sl);                   // Qwen3.5's unfused silu_mul rounds SiLU first (elementwise.cu:36-41)
-          a.Y[0][(size_t)n * M + out_row] = f2bf(sl * up);
+          a.Y[0][(size_t)n * a.y_ld + out_row] = f2bf(sl * up);
         }
       }
     }
@@ -527,7 +528,8 @@ void gemm_graphsafe_cuda(const pk_bf16* W, const pk_bf16* X, pk_bf16* Y, int M, 
                          pk_stream stream) {
   using namespace pk;
   if (M <= 0 || N <= 0 || K <= 0) return;
-  if (N > 4) {
+  // rows too long to keep N of them beside the weight ring go to the tensor cores as well
+  if (N > 4 || (K % 8 == 0 && (size_t)N * K * 2 > 96 * 1024)) {
     launch_gemm((const bf16*)W, (const bf16*)X, (bf16*)Y, M, N, K, stream);
     return;
   }
@@ -557,7 +559,7 @@ int pk_b200_gemv_fused(const pk_b200_gemv_args* g, pk_stream stream) {
   if (!g || g->M <= 0 || g->K <= 0) return -1;
   if (!gemv_stream_supported(g->W, g->X, g->N, g->K)) return -1;
   if (g->x_mode >= 1 && (g->hidden_out == nullptr || g->hidden_out == g->X || g->K > 10240)) return -1;
-  if (g->x_mode < 0 || g->x_mode > 3 || g->epi < 0 || g->epi > 5) return -1;
+  if (g->x_mode < 0 || g->x_mode > 3 || g->epi < 0 || g->epi > 6 || (g->y_ld && g->y_ld < g->M)) return -1;
   GemvArgs a{};
   a.W = (const bf16*)g->W;
   a.X = (const bf16*)g->X;
@@ -578,6 +580,7 @@ int pk_b200_gemv_fused(const pk_b200_gemv_args* g, pk_stream stream) {
   a.hidden_out = (bf16*)g->hidden_out;
   a.normed_out = (bf16*)g->normed_out;
   a.epi = g->epi;
+  a.y_ld = g->y_ld ? g->y_ld : g->M;
   if (g->x_mode == 2 || g->epi == 2) {
     const pk_tp_comm* comm = static_cast<const pk_tp_comm*>(g->tp_comm);
     if (!comm) return -1;

@@ -4,11 +4,11 @@
 // host's table), a chunk-local causal mask (query at position p sees keys floor(p / chunk) * chunk .. p; chunk 0 = plain
 // causal) and a learned per-head sink that adds exp(sink) to the softmax denominator without a value.
 // Further options (pk_attn_extra): a sliding window (keys p - window + 1 .. p), a soft cap on the scaled score
-// (cap * tanh(score / cap)), a linear distance bias (head h subtracts 2^(-slope_log2 (h + 1) / heads) * (p - j)), an
-// element-wise logistic gate on the output, and -- in the append -- an unweighted RMS norm of every cached value head.
+// (cap * tanh(score / cap)), a linear distance bias (head h subtracts 2^(-slope_log2 (h + 1) / heads) * (p - j)), a
+// logistic gate on the output, element by element or one per head, and -- in the append -- an unweighted RMS norm of every cached value head.
 // A window may keep the first `keep_first` positions of the sequence visible for good (they keep their true positions).
-// gqa_norm_append_kernel is the append for designs that norm q and k (per head with one weight for all heads, or over the whole
-// projection at once) before rotating them, stretch the query by a factor that grows with the logarithm of the position, or
+// gqa_norm_append_kernel is the append for designs that norm q and k (per head with one weight for all heads or none, or over the whole
+// projection at once) beside rotating them (a layer that reads another layer's cache brings queries only), stretch the query by a factor that grows with the logarithm of the position, or
 // cache the keys as projected in the place of values.
 //
 // Cache: token at position p of a request lives in page pages[page_off[req] + p / page_size], slot p % page_size, at
@@ -78,8 +78,9 @@ __global__ void gqa_rope_append_kernel(const E* __restrict__ qkv, int ld, const 
 }
 
 // Append for designs that norm q and k before they rotate.  qkv [tokens, ld] = [q (H*dim) | k (G*dim) | v (G*vdim)]; with `v_from_k` there
-// is no v part and the cached values are the keys as projected (vdim == dim).  norm_kind 1: every head of q (of k) is divided by its own
-// root mean square and multiplied by qw (kw) [dim], one weight for all heads; 2: the whole q row (k row) is divided by ONE root mean
+// is no v part and the cached values are the keys as projected (vdim == dim); with `q_only` the row is q alone and nothing is cached.  norm_kind 1: every head of q (of k) is divided by its own
+// root mean square and multiplied by qw (kw) [dim], one weight for all heads (null: no weight; a rotation keeps
+// the root mean square, so dividing by it before or after the rotation is the same); 2: the whole q row (k row) is divided by ONE root mean
 // square and multiplied by qw [H*dim] (kw [G*dim]); 0: no norm.  Then the first `dims` entries of every head rotate, and q is
 // multiplied by 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1) (temp_every 0: not).  One CTA per token; the row lives in shared
 // memory as fp32; sums of squares are added per head by one warp and then in head order, so a row's result does not depend on timing.
@@ -88,8 +89,9 @@ __global__ void gqa_norm_append_kernel(const E* __restrict__ qkv, int ld, const 
                                        const int* __restrict__ page_off, const int* __restrict__ pages, E* __restrict__ q_out, E* __restrict__ cache,
                                        long page_stride, int page_size, int H, int G, int dim, int vdim, int dims, int interleaved,
                                        const float* __restrict__ freq, float mag, const E* __restrict__ qw, const E* __restrict__ kw, int norm_kind,
-                                       float eps, float temp_coef, int temp_every, int v_from_k) {
+                                       float eps, float temp_coef, int temp_every, int v_from_k, int q_only) {
   extern __shared__ float na_sm[];
+  if (q_only) G = 0;
   float* row = na_sm;             // [nq + nk]
   float* inv = row + (H + G) * dim;  // [H + G] sum of squares per head
   pdl_wait();
@@ -98,11 +100,11 @@ __global__ void gqa_norm_append_kernel(const E* __restrict__ qkv, int ld, const 
   const E* src = qkv + (size_t)t * ld;
   const int nq = H * dim, nk = G * dim, nv = G * vdim, half = dims >> 1;
   // the page lookup (three dependent loads) and the weights of the last phase travel while the row is loaded and summed
-  const int page = pages[page_off[req[t]] + p / page_size];
-  if (norm_kind)
+  const int page = q_only ? 0 : pages[page_off[req[t]] + p / page_size];
+  if (norm_kind && qw)
     for (int e = threadIdx.x * 64; e < (norm_kind == 1 ? dim : nq + nk); e += blockDim.x * 64)
       prefetch_l2(norm_kind == 1 ? (e < dim ? qw + e : kw + e - dim) : (e < nq ? qw + e : kw + e - nq));  // a line of 64 entries each
-  if (norm_kind == 1 && threadIdx.x * 64 < dim) prefetch_l2(kw + threadIdx.x * 64);
+  if (norm_kind == 1 && kw && threadIdx.x * 64 < dim) prefetch_l2(kw + threadIdx.x * 64);
   // 16-byte accesses where every piece of the row and of the slot starts on such a boundary (bf16, sizes multiples of 8)
   const bool vec = sizeof(E) == 2 && ((nq | nk | nv | ld | (int)(page_stride & 7)) & 7) == 0 &&
                    ((reinterpret_cast<uintptr_t>(qkv) | reinterpret_cast<uintptr_t>(cache)) & 15) == 0;
@@ -135,7 +137,7 @@ __global__ void gqa_norm_append_kernel(const E* __restrict__ qkv, int ld, const 
     ik = 1.f / sqrtf(sk / (float)nk + eps);
   }
   const float stretch = temp_every > 0 ? 1.f + temp_coef * logf((float)((p + 1) / temp_every) + 1.f) : 1.f;
-  E* slot = cache + (size_t)page * page_stride + (size_t)(p % page_size) * (nk + nv);
+  E* slot = q_only ? nullptr : cache + (size_t)page * page_stride + (size_t)(p % page_size) * (nk + nv);
   // norm, rotation and the query's factor head by head (a warp per head, lanes over its entries: no index arithmetic per entry)
   for (int hd = warp; hd < H + G; hd += nw) {
     const bool is_q = hd < H;
@@ -183,7 +185,15 @@ struct AttnExtra {
   long gate_ld;
   int max_kv_len;
   int keep_first;
+  int gate_per_head;
+  long out_ld;  // elements from one row of the output to the next
 };
+// logistic gate of entry (t, h, d); x.gate is not null
+template <typename E>
+__device__ __forceinline__ float out_gate(const AttnExtra& x, int t, int h, int d, int vdim) {
+  const int at = x.gate_per_head ? h : h * vdim + d;
+  return 1.f / (1.f + expf(-to_f(static_cast<const E*>(x.gate)[(size_t)t * x.gate_ld + at])));
+}
 __device__ __forceinline__ int first_visible(int p, int chunk, int window) {
   int lo = chunk > 0 ? (p / chunk) * chunk : 0;
   if (window > 0) lo = max(lo, p - window + 1);
@@ -287,8 +297,8 @@ __global__ void __launch_bounds__(kGqaWarps * 32) gqa_attention_kernel(const E* 
 #pragma unroll
     for (int w = 0; w < kGqaWarps; ++w) o += sm_acc[w * vdim + d] * cw[w];
     o /= den;
-    if (x.gate) o *= 1.f / (1.f + expf(-to_f(static_cast<const E*>(x.gate)[(size_t)t * x.gate_ld + h * vdim + d])));
-    out[((size_t)t * H + h) * vdim + d] = from_f<E>(o);
+    if (x.gate) o *= out_gate<E>(x, t, h, d, vdim);
+    out[(size_t)t * x.out_ld + h * vdim + d] = from_f<E>(o);
   }
 }
 
@@ -498,19 +508,23 @@ __global__ void __launch_bounds__(128, 3) gqa_attention_mma_kernel(const bf16* _
   const float mt_a = fmaxf(m_a, sk), mt_b = fmaxf(m_b, sk);
   const float f_a = m_a == -INFINITY ? 0.f : exp2f(m_a - mt_a), f_b = m_b == -INFINITY ? 0.f : exp2f(m_b - mt_b);
   const float d_a = l_a * f_a + (sink ? exp2f(sk - mt_a) : 0.f), d_b = l_b * f_b + (sink ? exp2f(sk - mt_b) : 0.f);
-  const float i_a = f_a / d_a, i_b = f_b / d_b;
+  float i_a = f_a / d_a, i_b = f_b / d_b;
+  if (x.gate && x.gate_per_head) {
+    if (req_a >= 0) i_a *= out_gate<bf16>(x, t0 + ra, h, 0, DV);
+    if (req_b >= 0) i_b *= out_gate<bf16>(x, t0 + rb, h, 0, DV);
+  }
 #pragma unroll
   for (int ni = 0; ni < DV / 8; ++ni) {
     const int c = ni * 8 + 2 * tq;
     float g0 = 1.f, g1 = 1.f, g2 = 1.f, g3 = 1.f;
-    if (x.gate) {
+    if (x.gate && !x.gate_per_head) {
       const bf16* ga = static_cast<const bf16*>(x.gate) + (size_t)(t0 + ra) * x.gate_ld + h * DV + c;
       const bf16* gb = static_cast<const bf16*>(x.gate) + (size_t)(t0 + rb) * x.gate_ld + h * DV + c;
       if (req_a >= 0) g0 = 1.f / (1.f + expf(-bf2f(ga[0]))), g1 = 1.f / (1.f + expf(-bf2f(ga[1])));
       if (req_b >= 0) g2 = 1.f / (1.f + expf(-bf2f(gb[0]))), g3 = 1.f / (1.f + expf(-bf2f(gb[1])));
     }
-    if (req_a >= 0) *reinterpret_cast<uint32_t*>(out + ((size_t)(t0 + ra) * H + h) * DV + c) = pack_bf16(oa[ni][0] * i_a * g0, oa[ni][1] * i_a * g1);
-    if (req_b >= 0) *reinterpret_cast<uint32_t*>(out + ((size_t)(t0 + rb) * H + h) * DV + c) = pack_bf16(oa[ni][2] * i_b * g2, oa[ni][3] * i_b * g3);
+    if (req_a >= 0) *reinterpret_cast<uint32_t*>(out + (size_t)(t0 + ra) * x.out_ld + h * DV + c) = pack_bf16(oa[ni][0] * i_a * g0, oa[ni][1] * i_a * g1);
+    if (req_b >= 0) *reinterpret_cast<uint32_t*>(out + (size_t)(t0 + rb) * x.out_ld + h * DV + c) = pack_bf16(oa[ni][2] * i_b * g2, oa[ni][3] * i_b * g3);
   }
 }
 
@@ -550,8 +564,8 @@ __global__ void gqa_attention_merge_kernel(const float* __restrict__ part_o, con
     }
     for (; sp < nsplit; ++sp) a4[0] = fmaf(part_o[((size_t)(h * nsplit + sp) * T + t) * vdim + d], wgt[sp], a4[0]);
     float o = (a4[0] + a4[1]) + (a4[2] + a4[3]);
-    if (x.gate) o *= 1.f / (1.f + expf(-bf2f(static_cast<const bf16*>(x.gate)[(size_t)t * x.gate_ld + h * vdim + d])));
-    out[((size_t)t * H + h) * vdim + d] = f2bf(o);
+    if (x.gate) o *= out_gate<bf16>(x, t, h, d, vdim);
+    out[(size_t)t * x.out_ld + h * vdim + d] = f2bf(o);
   }
 }
 
@@ -618,9 +632,10 @@ extern "C" int pk_gqa_rope_append_ex(const void* qkv, int ld, const void* bias, 
 extern "C" int pk_gqa_norm_append(const void* qkv, int ld, const int* positions, const int* req, const int* page_off, const int* pages, void* q_out,
                                   void* cache, long page_stride, int page_size, int heads, int kv_heads, int dim, int vdim, int dims, int interleaved,
                                   const float* freq, float mag, const pk_qk_prep* prep, int tokens, int f32, pk_stream st) {
-  if (!qkv || !positions || !req || !page_off || !pages || !q_out || !cache || !prep || tokens <= 0 || heads <= 0 || kv_heads <= 0 ||
+  if (!qkv || !positions || !q_out || !prep || (!prep->q_only && (!req || !page_off || !pages || !cache)) || tokens <= 0 || heads <= 0 || kv_heads <= 0 ||
       heads % kv_heads || dim <= 0 || vdim <= 0 || dims < 0 || dims > dim || (dims & 1) || (dims > 0 && !freq) || page_size <= 0 ||
-      prep->norm_kind < 0 || prep->norm_kind > 2 || (prep->norm_kind && (!prep->q_weight || !prep->k_weight)) || prep->temp_every < 0 ||
+      prep->norm_kind < 0 || prep->norm_kind > 2 || (prep->norm_kind == 2 && (!prep->q_weight || !prep->k_weight)) ||
+      (prep->norm_kind == 1 && (!prep->q_weight != !prep->k_weight)) || prep->temp_every < 0 ||
       (prep->values_are_keys && vdim != dim))
     return -1;
   const size_t smem = ((size_t)(heads + kv_heads) * dim + heads + kv_heads) * sizeof(float);
@@ -631,7 +646,8 @@ extern "C" int pk_gqa_norm_append(const void* qkv, int ld, const int* positions,
     if (smem > 48 * 1024) cudaFuncSetAttribute(gqa_norm_append_kernel<E>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);                \
     launch(gqa_norm_append_kernel<E>, dim3(tokens), dim3(threads), smem, st, true, (const E*)qkv, ld, positions, req, page_off, pages, (E*)q_out,  \
            (E*)cache, page_stride, page_size, heads, kv_heads, dim, vdim, dims, interleaved, freq, mag, (const E*)prep->q_weight,                  \
-           (const E*)prep->k_weight, prep->norm_kind, prep->eps, prep->temp_coef, prep->temp_every, prep->values_are_keys);                        \
+           (const E*)prep->k_weight, prep->norm_kind, prep->eps, prep->temp_coef, prep->temp_every, prep->values_are_keys,                      \
+           prep->q_only);                        \
   } while (0)
   if (f32) PK_NA(float);
   else PK_NA(bf16);
@@ -652,14 +668,17 @@ extern "C" int pk_gqa_attention_ex(const void* q, const void* cache, const void*
   if (!q || !cache || !positions || !req || !page_off || !pages || !out || tokens <= 0 || heads <= 0 || kv_heads <= 0 || heads % kv_heads ||
       dim <= 0 || vdim <= 0 || chunk < 0 || page_size <= 0)
     return -1;
-  AttnExtra x{0, 0.f, 0.f, nullptr, 0, 0, 0};
+  AttnExtra x{0, 0.f, 0.f, nullptr, 0, 0, 0, 0, (long)heads * vdim};
   if (extra) {
-    if (extra->window < 0 || extra->softcap < 0.f || extra->slope_log2 < 0.f || extra->max_kv_len < 0 || extra->keep_first < 0) return -1;
-    x = AttnExtra{extra->window, extra->softcap, extra->slope_log2, extra->gate, extra->gate_ld, extra->max_kv_len, extra->window > 0 ? extra->keep_first : 0};
+    if (extra->window < 0 || extra->softcap < 0.f || extra->slope_log2 < 0.f || extra->max_kv_len < 0 || extra->keep_first < 0 ||
+        (extra->out_ld && extra->out_ld < (long)heads * vdim))
+      return -1;
+    x = AttnExtra{extra->window,     extra->softcap,    extra->slope_log2, extra->gate, extra->gate_ld,
+                  extra->max_kv_len, extra->window > 0 ? extra->keep_first : 0, extra->gate_per_head, extra->out_ld ? extra->out_ld : (long)heads * vdim};
   }
   if (dim > 32 * kGqaMaxPerLane || vdim > 32 * kGqaMaxPerLane) return -2;
   const bool aligned = ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(out)) & 15) == 0 &&
-                       page_stride % 8 == 0;
+                       page_stride % 8 == 0 && x.out_ld % 2 == 0;
   // bf16 prompt portions always; single decoded tokens too when the caller asked through the _ex entry (the key axis is then split)
   if (!f32 && (tokens >= 32 || extra) && aligned && dim == vdim && (dim == 64 || dim == 128 || dim == 32 || dim == 96) && (dim * kv_heads) % 8 == 0) {
 #define PK_GQA_MMA(D) \

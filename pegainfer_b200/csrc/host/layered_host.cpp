@@ -1,5 +1,5 @@
-// C++ host of the decoder designs whose checkpoint configuration lists the layers one by one (Vamadra, Risolorn, Nagosun, Goguzen, Rilonex),
-// on an fp32 residual stream.  A layer is a mixer plus an optional feed-forward, put together in one of five block forms:
+// C++ host of the decoder designs whose checkpoint configuration lists the layers one by one (Vamadra, Risolorn, Nagosun, Goguzen, Rilonex, Vegodra),
+// on an fp32 residual stream.  A layer is a mixer plus an optional feed-forward, put together in one of six block forms:
 //   block 0  sequential sublayers with the norm on each sublayer's OUTPUT:  x += norm(mixer(x));  x += norm(ff(x))
 //   block 1  parallel sublayers under one Dynamic-Tanh pre-norm:            h = dyt(x);  x += mixer(h) + ff(h)
 //   block 2  "sandwich": a grouped RMS norm before AND after each sublayer, the sublayer's result gated by a logistic
@@ -8,6 +8,8 @@
 //            a layer may run with another layer's weights (and a cache / state of its own); logits are scaled and soft-capped
 //   block 4  pre-norm sequential sublayers over a residual of parallel streams (hyper-connections): a sublayer reads u = sum_s in[s] x_s,
 //            h = rms(u) w, and its result y goes back as x_t <- sum_s mix[s][t] x_s + out[t] y   (mixers 2, 5 and 6)
+//   block 5  parallel sublayers under one layer norm (weight and bias):     h = ln(x);  x += mixer(h) + ff(h)   (mixers 0, 1 and 7); the embedding
+//            passes a norm of its own.  Both sublayers' inner results lie side by side, so one output projection makes their sum
 // Mixers: 0 latent attention (compressed paged cache, shared rotated key part, per-head sink, logistic output gate, optional
 // reuse of an earlier layer's cache); 1 grouped-query attention with biases, rotary embedding from a frequency table, a
 // chunk-local causal mask and a sink, over a paged K/V cache (block 2 adds: sliding window, score soft cap, linear distance
@@ -15,12 +17,13 @@
 // convolutions; 3 xLSTM matrix memory; 4 two branches side by side on the same input -- grouped-query attention and a state-space layer
 // (scalar decay per head, short causal convolution, gated group-normed read-out) -- each branch's result RMS-normed over the width, the
 // mixer's result their mean; 5 real-gated linear recurrent unit behind a short convolution, times a GELU branch; 6 two branches side by
-// side -- grouped-query attention with mixed scores, logistic weights and a gate per head, and a gated delta rule -- summed with constants.
+// side -- grouped-query attention with mixed scores, logistic weights and a gate per head, and a gated delta rule -- summed with constants; 7 gated linear attention (a decay per key channel from a low-rank projection).
 // In block 4 the delta rule may decay per head and key channel and its read-out gate may be logistic, both through low-rank projections.
-// Block 3 gives the attention (mixer 1 and the attention branch of 4) further options: RMS norm of q and k per
+// Block 5 gives the latent attention queries through a normed latent and an element-wise output gate, and the grouped-query attention unit-RMS
+// queries and keys, a gate per head and another layer's keys and values (kv_from).  Block 3 gives the attention (mixer 1 and the attention branch of 4) further options: RMS norm of q and k per
 // head or over the whole projection, a query factor that grows with the logarithm of the position, values that are the keys as projected,
-// a window that keeps the first positions visible, rotary frequencies rescaled by wavelength.  Mixers 2 to 6 keep an fp32 state per
-// request in numbered state slots.  Feed-forward: dense SwiGLU, dense with a ReLU gate, or a mixture of experts (softmax or logistic router or plain top logits;
+// a window that keeps the first positions visible, rotary frequencies rescaled by wavelength.  Mixers 2 to 7 keep an fp32 state per
+// request in numbered state slots.  Feed-forward: dense SwiGLU, dense with a ReLU or GELU gate, or a mixture of experts (softmax or logistic router or plain top logits;
 // relu^2, gated-SiLU or clamped gated experts; a shared expert with or without a gate).
 //
 // Same structure as the other hosts in this folder: kernels are reached only through the C ABI
@@ -76,11 +79,11 @@ struct LayerCfg {  // mirrored by ctypes in pegainfer_b200/layered.py
   float slope_log2;          // 1: head h subtracts 2^(-slope_log2 (h + 1) / heads) * distance from the score
   int value_norm;            // 1: cached values are divided by their root mean square per head (eps of the model, no weight)
   int sink_kind;             // 0 learned per-head sink 'mix.sink', 1 none, 2 a sink of score zero (one added to the softmax denominator)
-  int out_gate;              // 1: 1 = heads' outputs times logistic(W_g h) element by element ('mix.g' [heads * vdim, width])
+  int out_gate;              // 1 = heads' outputs times logistic(W_g h) element by element ('mix.g' [heads * vdim, width]); block 5: also 2 = one per head ('mix.g' [heads, width])
   int proj_bias;             // 1: q, k, v and o projections carry biases ('.b')
   // options read by block 3 (all off when zero)
   int keep_first;            // attention with a window: the first keep_first positions stay visible
-  int qk_norm;               // 1: RMS norm of q and k per head, weights 'q.norm' / 'k.norm' [dim]; 2: over the whole projection, weights [heads*dim] / [kv_heads*dim]
+  int qk_norm;               // 1: RMS norm of q and k per head, weights 'q.norm' / 'k.norm' [dim]; 2: over the whole projection, weights [heads*dim] / [kv_heads*dim]; 3 (block 5): per head, no weights
   float q_temp_coef;         // q *= 1 + q_temp_coef * ln(floor((p + 1) / q_temp_every) + 1)
   int q_temp_every;
   int values_are_keys;       // 1: no value projection, a head's values are its keys as projected
@@ -96,13 +99,16 @@ struct LayerCfg {  // mirrored by ctypes in pegainfer_b200/layered.py
   float left_scale, right_scale;  // 6: factors of the attention's and the delta rule's result
   int lru_width, lru_blocks;      // 5
   float lru_rate;                 // 5: log a = -lru_rate * r * softplus(lam)
-  int mlp_act;               // dense feed-forward: 0 SiLU gate, 1 ReLU gate
+  int mlp_act;               // dense feed-forward: 0 SiLU gate, 1 ReLU gate, 2 GELU gate (tanh form)
+  // options read by block 5
+  int q_rank;                // 0: size of the latent the queries pass ('dq' [q_rank, width], 'dq.norm', 'uq')
+  float tau;                 // 7: decay = logistic(.)^(1 / tau); rank of the decay's projection in decay_rank
 };
 struct ModelCfg {
   int vocab, width, n_layers;
   float eps;
   int f32, page_size, num_pages, max_requests, device, enable_pdl;
-  int block_kind;  // 0 sequential sublayers, offset RMS norm on their outputs; 1 parallel sublayers under a Dynamic-Tanh pre-norm; 2 sandwich
+  int block_kind;  // 0 sequential sublayers, offset RMS norm on their outputs; 1 parallel sublayers under a Dynamic-Tanh pre-norm; 2 sandwich; 3 .. 5 see above
   float embed_scale, logit_scale;
   int norm_groups;        // block 2: parts of a row that are normed separately
   float residual_mult;    // block 2: multiplier of every sublayer's normed result
@@ -118,7 +124,7 @@ struct Lib {
   X(cuda_set_device) X(cublas_init) X(cublas_destroy) X(gemm_cuda) X(flashinfer_top1_cuda) X(pk_b200_set_pdl) X(pk_b200_launch_count)      \
   X(pk_res32_skinny_proj) X(pk_convert) X(pk_gemm_strided) X(pk_proj_rows_f32out) X(pk_scale_to_f32) X(pk_top1_rows_f32)
 #define PV_MOE(X) X(pk_moe_down_combine) X(pk_moe_grouped_workspace_bytes) X(pk_moe_up_act_p) X(pk_moe_grouped_act_p)
-#define PV_DENSE(X) X(pk_act) X(pk_b200_gemv_fused) X(pk_b200_gemm_gated)
+#define PV_DENSE(X) X(pk_act) X(pk_act_ex) X(pk_b200_gemv_fused) X(pk_b200_gemm_gated_ex)
 #define PV_BLOCK0(X)                                                                                                                        \
   X(pk_res32_embed) X(pk_res32_offset_norm_add) X(pk_res32_offset_norm_rows) X(pk_rope_slice) X(pk_latent_kv_append) X(pk_latent_attention) \
   X(pk_router_grouped_topk)
@@ -126,21 +132,29 @@ struct Lib {
   X(pk_res32_embed_scaled) X(pk_res32_add_dyt) X(pk_res32_dyt_rows) X(pk_gqa_rope_append) X(pk_gqa_attention) X(pk_causal_conv_silu)       \
   X(pk_mlstm_seq) X(pk_router_topk_ex)
 #define PV_BLOCK13(X) X(pk_head_norm_gate)
-#define PV_BLOCK23(X) X(pk_res32_gnorm_rows) X(pk_gqa_attention_ex)
+#define PV_BLOCK23(X) X(pk_res32_gnorm_rows)
+#define PV_BLOCK235(X) X(pk_gqa_attention_ex)
+#define PV_BLOCK25(X) X(pk_latent_attention_ex)
+#define PV_BLOCK35(X) X(pk_gqa_norm_append)
+#define PV_BLOCK45(X) X(pk_head_norm_gate_ex) X(pk_gemm_strided_f32out)
 #define PV_BLOCK3(X)                                                                                                                        \
-  X(pk_res32_embed_scaled_norm) X(pk_res32_branches_add_norm) X(pk_logits_scale_cap) X(pk_act_clamped) X(pk_gqa_norm_append)               \
+  X(pk_res32_embed_scaled_norm) X(pk_res32_branches_add_norm) X(pk_logits_scale_cap) X(pk_act_clamped)                                      \
   X(pk_causal_conv_silu_bias) X(pk_ssd_seq) X(pk_router_topk_logits)
 #define PV_BLOCK2(X)                                                                                                                        \
   X(pk_res32_embed_gnorm) X(pk_res32_gated_gnorm_add) X(pk_rope_slice_ex)   \
-  X(pk_latent_kv_append_ex) X(pk_latent_attention_ex) X(pk_b200_gemm_segments)
+  X(pk_latent_kv_append_ex) X(pk_b200_gemm_segments)
 #define PV_BLOCK14(X) X(pk_gated_delta_seq)
 #define PV_BLOCK24(X) X(pk_gqa_rope_append_ex)
 #define PV_BLOCK4(X)                                                                                                                        \
   X(pk_res32_streams_embed) X(pk_res32_streams_step) X(pk_res32_streams_rows) X(pk_gqa_mixed_attention) X(pk_causal_conv)                  \
-  X(pk_channel_decay) X(pk_channel_delta_seq) X(pk_lru_seq) X(pk_head_norm_gate_ex) X(pk_gemm_strided_f32out)
+  X(pk_channel_decay) X(pk_channel_delta_seq) X(pk_lru_seq)
+#define PV_BLOCK5(X)                                                                                                                        \
+  X(pk_res32_embed_lnorm) X(pk_res32_add_lnorm) X(pk_res32_lnorm_rows) X(pk_latent_prep) X(pk_latent_query) X(pk_gemm_strided_gated)       \
+  X(pk_gla_seq) X(pk_logistic_decay)
 #define PV_FN(name) decltype(&::name) name = nullptr;
   PV_COMMON(PV_FN) PV_MOE(PV_FN) PV_DENSE(PV_FN) PV_BLOCK0(PV_FN) PV_BLOCK1(PV_FN) PV_BLOCK2(PV_FN) PV_BLOCK3(PV_FN) PV_BLOCK4(PV_FN)
-  PV_BLOCK13(PV_FN) PV_BLOCK14(PV_FN) PV_BLOCK23(PV_FN) PV_BLOCK24(PV_FN)
+  PV_BLOCK13(PV_FN) PV_BLOCK14(PV_FN) PV_BLOCK23(PV_FN) PV_BLOCK24(PV_FN) PV_BLOCK235(PV_FN) PV_BLOCK25(PV_FN) PV_BLOCK35(PV_FN) PV_BLOCK45(PV_FN)
+  PV_BLOCK5(PV_FN)
 #undef PV_FN
   // a library built for one design need not hold the other block form's kernels: only what `block_kind` runs is required
   std::string load(const std::string& p, int block_kind) {
@@ -156,11 +170,13 @@ struct Lib {
     } else if (block_kind == 1) {
       PV_MOE(PV_REQ) PV_BLOCK1(PV_REQ) PV_BLOCK13(PV_REQ) PV_BLOCK14(PV_REQ)
     } else if (block_kind == 2) {  // the sandwich block form has no mixture of experts
-      PV_DENSE(PV_REQ) PV_BLOCK2(PV_REQ) PV_BLOCK23(PV_REQ) PV_BLOCK24(PV_REQ)
+      PV_DENSE(PV_REQ) PV_BLOCK2(PV_REQ) PV_BLOCK23(PV_REQ) PV_BLOCK24(PV_REQ) PV_BLOCK235(PV_REQ) PV_BLOCK25(PV_REQ)
     } else if (block_kind == 4) {  // no mixture of experts either
-      PV_DENSE(PV_REQ) PV_BLOCK4(PV_REQ) PV_BLOCK14(PV_REQ) PV_BLOCK24(PV_REQ)
+      PV_DENSE(PV_REQ) PV_BLOCK4(PV_REQ) PV_BLOCK14(PV_REQ) PV_BLOCK24(PV_REQ) PV_BLOCK45(PV_REQ)
+    } else if (block_kind == 5) {  // nor here
+      PV_DENSE(PV_REQ) PV_BLOCK5(PV_REQ) PV_BLOCK235(PV_REQ) PV_BLOCK25(PV_REQ) PV_BLOCK35(PV_REQ) PV_BLOCK45(PV_REQ)
     } else {
-      PV_MOE(PV_REQ) PV_BLOCK3(PV_REQ) PV_BLOCK13(PV_REQ) PV_BLOCK23(PV_REQ)
+      PV_MOE(PV_REQ) PV_BLOCK3(PV_REQ) PV_BLOCK13(PV_REQ) PV_BLOCK23(PV_REQ) PV_BLOCK235(PV_REQ) PV_BLOCK35(PV_REQ)
     }
 #undef PV_REQ
     return missing.empty() ? "" : "kernel library " + p + " lacks:" + missing;
@@ -188,6 +204,7 @@ struct Layer {
   DeviceBuf alpha32, corr32, p0_32, p1_32, p2_32;          // float copies of small parameter vectors (made in finalize)
   Mat alpha, corr, p0, p1, p2;
   Mat qn, kn, conv_b, o2, lout, rout;                      // block 3: q / k norm weights; mixer 4: convolution bias, second output projection, branch norms
+  Mat uq, dq_norm;                                         // block 5: second factor and norm weight of the queries' latent (the first is stacked into qkv)
   Mat a2, g2, gates, conv_in_b, r_bias, i_bias, talk, hc[2][3];  // block 4: low-rank second factors; linear unit; score mixing; stream weights in / out / mix
   DeviceBuf hc32[2][3];
   int wsrc = 0;                                            // the layer whose weights this layer runs with (itself unless the configuration says otherwise)
@@ -208,7 +225,7 @@ struct Model {
   int es = 2;  // element size
   Mat embed, head, final_norm, final_b, final_alpha;
   DeviceBuf final_alpha32;
-  Mat embed_norm;                // block 2: norm of the embedding
+  Mat embed_norm, embed_norm_b;  // blocks 2 and 5: norm of the embedding
   DeviceBuf zero_sink;           // block 2: [heads] zeros, the sink of score zero
   DeviceBuf rgbuf;               // block 2: gate pre-activations [tokens, width]
   DeviceBuf cache, state;        // paged cache pool; recurrent state, one slot per request id
@@ -224,7 +241,8 @@ struct Model {
   DeviceBuf ao2, mix2;                       // mixer 4: the state-space branch's gated read-out and its projection
   DeviceBuf attn_ws;                         // block 4: partial sums of the attention's key shares
   long attn_ws_bytes = 0;
-  DeviceBuf zc, gbuf, one32;                 // block 4: fp32 decay / gate pre-activations, low-rank read-out gate; the constant 1 (weights of a single stream)
+  DeviceBuf cq;                              // block 5: normed latents of the queries
+  DeviceBuf zc, gbuf, one32;                 // blocks 4, 5: fp32 decay / gate pre-activations, low-rank read-out gate; the constant 1 (weights of a single stream)
   DeviceBuf x, xa, q, dkv, qa, gate, olat, ao, mix, gu, act, z, ids, wts, hid, yf, sgl, sh, xr, logits_e, logits_f, logits_bf, sampled_d, top1_val,
       top1_states, trail, moe_ws;
   DeviceBuf meta_d;
@@ -240,7 +258,7 @@ struct Model {
   std::set<GraphKey> seen;
   bool use_graph = true;
   // widest layer
-  int mx_big = 0, mx_conv = 0, mx_small = 0, mx_inner = 0, mx_zc = 0, mx_gbuf = 0, mx_attn = 0, n_streams = 1;
+  int mx_big = 0, mx_conv = 0, mx_small = 0, mx_inner = 0, mx_zc = 0, mx_gbuf = 0, mx_attn = 0, mx_cq = 0, n_streams = 1;
   int mx_q = 0, mx_dkv = 0, mx_qa = 0, mx_h = 0, mx_olat = 0, mx_ao = 0, mx_gu = 0, mx_act = 0, mx_e = 0, mx_top = 0, mx_hid = 0;
 
   bool fail(const std::string& m) {
@@ -282,7 +300,10 @@ struct Model {
   bool run_streams_layer(int li, int T, int max_kv, const int* M, int n);
   bool delta_branch(const Layer& L, const char* rows, int nbig, const float* small, int nsmall, float* slot0, void* out, int ld_out, float factor, int T,
                     const int* M, int n);
-  bool gated_ff(const Layer& L, int T);
+  bool run_lnorm_layer(int li, int T, int max_kv, const int* M, int n);
+  bool configure_lnorm_layer(int i, int64_t* off, int64_t* soff);
+  bool load_lnorm_tensor(Layer& L, const std::string& sub, const std::string& name, const void* data, int rows, int cols, bool* known);
+  bool gated_ff(const Layer& L, int T, void* out, int ld_out);
   bool load_streams_tensor(Layer& L, const std::string& sub, const std::string& name, const void* data, int rows, int cols, bool* known);
   bool put_cols(Mat& m, int rows, int cols, int col0, const void* src, int src_cols, const std::string& name, int got_rows, int got_cols);
   bool lin_segments(const Mat& W, const void* X, void* const* Y, const int* seg_rows, int N);
@@ -308,13 +329,89 @@ struct DeltaDims {
   int64_t state(int taps) const { return (int64_t)H * D * V + (int64_t)std::max(taps - 1, 0) * C; }
 };
 
+// layout of a block 5 layer's stacked projection and of its sublayers' inner results (side by side in ao, as their output projections are in o)
+struct LnormDims {
+  int nq, nk, nv;      // 1, 7: q, k, v columns (k and v: 0 when the layer borrows them);  0: latent of the queries, latent + shared rotated part, 0
+  int ng, na;          // output gate; first factor of the decay
+  int big, wo, ff, ld; // padded columns of the projection; the mixer's inner result, the feed-forward's, both
+  explicit LnormDims(const LayerCfg& a) {
+    const bool latent = a.mixer_kind == 0, own = a.kv_from < 0;
+    nq = latent ? a.q_rank : a.heads * a.dim;
+    nk = latent ? a.kv_rank + a.rot_dim : a.mixer_kind == 7 ? a.heads * a.dim : own ? a.kv_heads * a.dim : 0;
+    nv = latent ? 0 : a.mixer_kind == 7 ? a.heads * a.vdim : own ? a.kv_heads * a.vdim : 0;
+    ng = a.mixer_kind == 7 || a.out_gate == 1 ? a.heads * a.vdim : a.out_gate == 2 ? a.heads : 0;
+    na = a.mixer_kind == 7 ? a.decay_rank : 0;
+    big = (nq + nk + nv + ng + na + 7) / 8 * 8;  // rows of zeros at the end keep every row of the result 16-byte aligned
+    wo = a.heads * a.vdim;
+    ff = a.mlp_kind == 1 ? a.ff : 0;
+    ld = wo + ff;
+  }
+  int gate_at() const { return nq + nk + nv; }
+  int decay_at() const { return nq + nk + nv + ng; }
+};
+
 static std::string lname(int i, const char* s) { return "l" + std::to_string(i) + "." + s; }
+
+bool Model::configure_lnorm_layer(int i, int64_t* off, int64_t* soff) {
+  Layer& L = layers[i];
+  const LayerCfg& a = L.c;
+  if (a.mixer_kind != 0 && a.mixer_kind != 1 && a.mixer_kind != 7) return fail(lname(i, "mixer: not available in this block form"));
+  if (a.heads <= 0 || a.dim <= 0 || a.vdim <= 0 || a.out_gate < 0 || a.out_gate > 2 || (a.sink_kind != 0 && a.sink_kind != 1))
+    return fail(lname(i, "mixer: inconsistent sizes or options"));
+  L.wsrc = i;
+  L.owner = i;
+  if (a.mixer_kind == 0) {
+    if (a.kv_rank <= 0 || a.q_rank <= 0 || a.rot_dim < 0 || a.kv_from >= 0 || a.out_gate != 1 || a.sink_kind != 1)
+      return fail(lname(i, "mixer: inconsistent latent attention"));
+    if (a.rot_dims < 0 || a.rot_dims > a.rot_dim || (a.rot_dims & 1)) return fail(lname(i, "mixer: rot.dims must be even and at most rot_dim"));
+    if (a.kv_rank > 1024) return fail(lname(i, "mixer: kv_rank above 1024 is outside the attention kernel's range"));
+    L.cache_off = *off;
+    *off += (int64_t)c.page_size * (a.kv_rank + a.rot_dim);
+    mx_cq = std::max(mx_cq, a.q_rank);
+    mx_q = std::max(mx_q, a.heads * (a.dim + a.rot_dim));
+    mx_qa = std::max(mx_qa, a.heads * (a.kv_rank + a.rot_dim));
+    mx_olat = std::max(mx_olat, a.heads * a.kv_rank);
+  } else if (a.mixer_kind == 1) {
+    if (a.kv_heads <= 0 || a.heads % a.kv_heads) return fail(lname(i, "mixer: heads must be a multiple of kv_heads"));
+    if (a.dim > 256 || a.vdim > 256) return fail(lname(i, "mixer: head sizes above 256 are outside the kernels' range"));
+    if (a.rot_dims < 0 || a.rot_dims > a.dim || (a.rot_dims & 1)) return fail(lname(i, "mixer: rot.dims must be even and at most dim"));
+    if (a.chunk < 0 || a.window < 0 || (a.qk_norm != 0 && a.qk_norm != 3)) return fail(lname(i, "mixer: inconsistent attention options"));
+    if (a.kv_from >= 0) {
+      if (a.kv_from >= i || layers[a.kv_from].c.mixer_kind != 1 || layers[a.kv_from].c.kv_from >= 0)
+        return fail(lname(i, "mixer: kv_from must name an earlier attention layer with keys and values of its own"));
+      const LayerCfg& o = layers[a.kv_from].c;
+      if (o.kv_heads != a.kv_heads || o.dim != a.dim || o.vdim != a.vdim) return fail(lname(i, "mixer: key / value sizes differ from the layer it borrows from"));
+      L.owner = a.kv_from;
+      L.cache_off = layers[a.kv_from].cache_off;
+    } else {
+      L.cache_off = *off;
+      *off += (int64_t)c.page_size * a.kv_heads * (a.dim + a.vdim);
+    }
+    mx_q = std::max(mx_q, a.heads * a.dim);
+  } else {
+    if (a.decay_rank <= 0 || !(a.tau > 0.f) || a.kv_from >= 0) return fail(lname(i, "mixer: inconsistent gated linear attention"));
+    if (a.dim > 256) return fail(lname(i, "mixer: head sizes above 256 are outside the kernels' range"));
+    L.state_off = *soff;
+    *soff += (int64_t)a.heads * a.dim * a.vdim;
+    *soff = (*soff + 3) / 4 * 4;
+    mx_zc = std::max(mx_zc, a.heads * a.dim);
+    mx_inner = std::max(mx_inner, a.heads * a.vdim);
+  }
+  *off = (*off + 7) / 8 * 8;  // every layer's block starts 16-byte aligned in both element types
+  if (a.mlp_kind != 0 && a.mlp_kind != 1) return fail(lname(i, "mlp: this block form has dense feed-forwards only"));
+  if (a.mlp_kind == 1 && (a.ff <= 0 || a.mlp_act < 0 || a.mlp_act > 2)) return fail(lname(i, "mlp: ff must be positive"));
+  const LnormDims d(a);
+  mx_big = std::max(mx_big, d.big);
+  mx_ao = std::max(mx_ao, d.ld);
+  if (d.ff) mx_gu = std::max(mx_gu, 2 * d.ff);
+  return true;
+}
 
 bool Model::configure(const ModelCfg& mc, const LayerCfg* lc) {
   c = mc;
   es = c.f32 ? 4 : 2;
   if (c.vocab <= 0 || c.width <= 0 || c.n_layers <= 0) return fail("vocab, width and the number of layers must be positive");
-  if (c.block_kind < 0 || c.block_kind > 4) return fail("unknown block form");
+  if (c.block_kind < 0 || c.block_kind > 5) return fail("unknown block form");
   if (c.streams < 0 || c.streams > 16) return fail("streams: 1 to 16 parallel rows of the residual");
   n_streams = c.block_kind == 4 ? std::max(c.streams, 1) : 1;
   if (c.block_kind == 3 && c.logit_softcap < 0.f) return fail("logit_softcap must not be negative");
@@ -327,7 +424,11 @@ bool Model::configure(const ModelCfg& mc, const LayerCfg* lc) {
     Layer& L = layers[i];
     L.c = lc[i];
     const LayerCfg& a = L.c;
-    if (a.mixer_kind < 0 || a.mixer_kind > 6) return fail(lname(i, "mixer: unknown kind"));
+    if (a.mixer_kind < 0 || a.mixer_kind > 7) return fail(lname(i, "mixer: unknown kind"));
+    if (c.block_kind == 5) {
+      if (!configure_lnorm_layer(i, &off, &soff)) return false;
+      continue;
+    }
     if (c.block_kind == 4) {
       if (a.mixer_kind != 2 && a.mixer_kind < 5) return fail(lname(i, "mixer: not available in this block form"));
       L.wsrc = i;
@@ -629,14 +730,56 @@ bool Model::load_streams_tensor(Layer& L, const std::string& sub, const std::str
   return false;
 }
 
+// a tensor of a block 5 layer; *known = false: not one of this layer's.  The mixer's projections are stacked
+//   mixer 0  [q latent | kv latent, shared rotated part | g]        mixer 1  [q (| k | v) | g]        mixer 7  [q | k | v | g | a1]
+// and its output projection lies beside the feed-forward's along the contraction axis.
+bool Model::load_lnorm_tensor(Layer& L, const std::string& sub, const std::string& name, const void* data, int rows, int cols, bool* known) {
+  const LayerCfg& a = L.c;
+  const LnormDims d(a);
+  const int W = c.width, H = a.heads, mk = a.mixer_kind;
+  *known = true;
+  if (sub == "norm1") return put(L.norm1, 1, W, 0, data, 1, name, rows, cols);
+  if (sub == "norm1.b") return put(L.nb, 1, W, 0, data, 1, name, rows, cols);
+  if (d.ff) {
+    if (sub == "mlp.gate") return put(L.gate_up, 2 * d.ff, W, 0, data, d.ff, name, rows, cols);
+    if (sub == "mlp.up") return put(L.gate_up, 2 * d.ff, W, d.ff, data, d.ff, name, rows, cols);
+    if (sub == "mlp.down") return put_cols(L.o, W, d.ld, d.wo, data, d.ff, name, rows, cols);
+  }
+  if (sub == "mix.o") return put_cols(L.o, W, d.ld, 0, data, d.wo, name, rows, cols);
+  if (d.ng && sub == "mix.g") return put(L.qkv, d.big, W, d.gate_at(), data, d.ng, name, rows, cols);
+  if (mk == 0) {
+    if (sub == "mix.dq") return put(L.qkv, d.big, W, 0, data, d.nq, name, rows, cols);
+    if (sub == "mix.dkv") return put(L.qkv, d.big, W, d.nq, data, d.nk, name, rows, cols);
+    if (sub == "mix.dq.norm") return put(L.dq_norm, 1, a.q_rank, 0, data, 1, name, rows, cols);
+    if (sub == "mix.dkv.norm") return put(L.dkv_norm, 1, a.kv_rank, 0, data, 1, name, rows, cols);
+    if (sub == "mix.uq") return put(L.uq, H * (a.dim + a.rot_dim), a.q_rank, 0, data, H * (a.dim + a.rot_dim), name, rows, cols);
+    if (sub == "mix.uk") return put_uk(L, data, name, rows, cols);
+    if (sub == "mix.uv") return put(L.uv, H * a.vdim, a.kv_rank, 0, data, H * a.vdim, name, rows, cols);
+  } else {
+    if (sub == "mix.q") return put(L.qkv, d.big, W, 0, data, d.nq, name, rows, cols);
+    if (d.nk && sub == "mix.k") return put(L.qkv, d.big, W, d.nq, data, d.nk, name, rows, cols);
+    if (d.nv && sub == "mix.v") return put(L.qkv, d.big, W, d.nq + d.nk, data, d.nv, name, rows, cols);
+    if (mk == 1 && a.sink_kind == 0 && sub == "mix.sink") return put(L.sink, 1, H, 0, data, 1, name, rows, cols);
+    if (mk == 7) {
+      if (sub == "mix.a1") return put(L.qkv, d.big, W, d.decay_at(), data, d.na, name, rows, cols);
+      if (sub == "mix.a2") return put(L.a2, H * a.dim, a.decay_rank, 0, data, H * a.dim, name, rows, cols);
+      if (sub == "mix.a2.b") return put(L.p1, 1, H * a.dim, 0, data, 1, name, rows, cols);
+      if (sub == "mix.norm") return put(L.hnorm, 1, a.vdim, 0, data, 1, name, rows, cols);
+    }
+  }
+  *known = false;
+  return false;
+}
+
 bool Model::load_tensor(const std::string& name, const void* data, int rows, int cols, int is_f32) {
   if ((is_f32 != 0) != (c.f32 != 0)) return fail(name + ": element type differs from the model's");
   const int W = c.width;
   if (name == "embed") return put(embed, c.vocab, W, 0, data, c.vocab, name, rows, cols);
-  if (c.block_kind == 2 && name == "embed.norm") return put(embed_norm, 1, W, 0, data, 1, name, rows, cols);
+  if ((c.block_kind == 2 || c.block_kind == 5) && name == "embed.norm") return put(embed_norm, 1, W, 0, data, 1, name, rows, cols);
   if (name == "head") return put(head, c.vocab, W, 0, data, c.vocab, name, rows, cols);
   if (name == "final.norm") return put(final_norm, 1, W, 0, data, 1, name, rows, cols);
-  if (c.block_kind == 1 && name == "final.norm.b") return put(final_b, 1, W, 0, data, 1, name, rows, cols);
+  if (c.block_kind == 5 && name == "embed.norm.b") return put(embed_norm_b, 1, W, 0, data, 1, name, rows, cols);
+  if ((c.block_kind == 1 || c.block_kind == 5) && name == "final.norm.b") return put(final_b, 1, W, 0, data, 1, name, rows, cols);
   if (c.block_kind == 1 && name == "final.norm.alpha") return put(final_alpha, 1, 1, 0, data, 1, name, rows, cols);
   if (name.size() < 3 || name[0] != 'l') return fail("unknown tensor " + name);
   const size_t dot = name.find('.');
@@ -647,9 +790,9 @@ bool Model::load_tensor(const std::string& name, const void* data, int rows, int
   const LayerCfg& a = L.c;
   const std::string sub = name.substr(dot + 1);
   bool ok;
-  if (c.block_kind == 4) {
+  if (c.block_kind == 4 || c.block_kind == 5) {
     bool known;
-    ok = load_streams_tensor(L, sub, name, data, rows, cols, &known);
+    ok = c.block_kind == 4 ? load_streams_tensor(L, sub, name, data, rows, cols, &known) : load_lnorm_tensor(L, sub, name, data, rows, cols, &known);
     if (!known) return fail("unknown tensor " + name + " for the configuration of layer " + std::to_string(li));
     if (ok) L.got.insert(sub);
     return ok;
@@ -881,7 +1024,8 @@ static void rotary_table(const LayerCfg& a, std::vector<float>* f, float* mag) {
 
 bool Model::finalize() {
   if (!embed.d.ptr || !head.d.ptr || !final_norm.d.ptr) return fail("embed / head / final.norm missing");
-  if (c.block_kind == 2 && !embed_norm.d.ptr) return fail("embed.norm missing");
+  if ((c.block_kind == 2 || c.block_kind == 5) && !embed_norm.d.ptr) return fail("embed.norm missing");
+  if (c.block_kind == 5 && (!embed_norm_b.d.ptr || !final_b.d.ptr)) return fail("embed.norm.b / final.norm.b missing");
   if (c.block_kind == 2 && !zero_sink.alloc_zeros((size_t)std::max(mx_h, 1) * es)) return fail("allocation failed");
   if (c.block_kind == 1 && (!final_b.d.ptr || !final_alpha.d.ptr || !to_f32(final_alpha, &final_alpha32))) return fail("final.norm.b / final.norm.alpha missing");
   if (c.block_kind == 4) {
@@ -894,7 +1038,15 @@ bool Model::finalize() {
     Layer& L = layers[i];
     const LayerCfg& a = L.c;
     std::vector<std::string> need;
-    if (c.block_kind == 4) {
+    if (c.block_kind == 5) {
+      need = {"norm1", "norm1.b", "mix.o"};
+      if (LnormDims(a).ng) need.push_back("mix.g");
+      if (a.mixer_kind == 0) need.insert(need.end(), {"mix.dq", "mix.dq.norm", "mix.uq", "mix.dkv", "mix.dkv.norm", "mix.uk", "mix.uv"});
+      else need.push_back("mix.q");
+      if (a.mixer_kind != 0 && a.kv_from < 0) need.insert(need.end(), {"mix.k", "mix.v"});
+      if (a.mixer_kind == 1 && a.sink_kind == 0) need.push_back("mix.sink");
+      if (a.mixer_kind == 7) need.insert(need.end(), {"mix.a1", "mix.a2", "mix.a2.b", "mix.norm"});
+    } else if (c.block_kind == 4) {
       need = {"norm1"};
       if (a.mlp_kind) need.push_back("norm2");
       for (int q = 0; q < (c.streams > 0 ? (a.mlp_kind ? 2 : 1) : 0); ++q)
@@ -976,6 +1128,10 @@ bool Model::finalize() {
       if (a.mixer_kind == 6 && !to_f32(L.p2, &L.p2_32)) return false;
       if (a.mixer_kind != 6) continue;  // only the attention rotates
     }
+    if (c.block_kind == 5 && a.mixer_kind == 7) {
+      if (!to_f32(L.p1, &L.p1_32)) return false;
+      continue;
+    }
     if (c.block_kind >= 2 && a.rot_dims == 0) continue;  // nothing rotates
     std::vector<float> f;
     rotary_table(a, &f, &L.mag);
@@ -1023,6 +1179,9 @@ bool Model::ensure_scratch(int T, int R) {
       attn_ws_bytes = (long)(n <= 256 ? std::min<size_t>(128 * n, 4096) : 4 * n) * mx_attn * 4;
       ok = attn_ws.alloc_uninit((size_t)attn_ws_bytes);
     }
+    if (ok && c.block_kind == 5)
+      ok = big.alloc_uninit(n * std::max(mx_big, 1) * es) && cq.alloc_uninit(n * std::max(mx_cq, 1) * es) && zc.alloc_uninit(n * std::max(mx_zc, 1) * 4) &&
+           orec.alloc_uninit(n * std::max(mx_inner, 1) * 4);
     if (ok && c.block_kind == 2) ok = big.alloc_uninit(n * std::max(mx_big, 1) * es) && rgbuf.alloc_uninit(n * W * es);
     if (ok && c.block_kind == 3)
       ok = h32.alloc_uninit(n * W * 4) && big.alloc_uninit(n * std::max(mx_big, 1) * es) && convo.alloc_uninit(n * std::max(mx_conv, 1) * es) &&
@@ -1101,7 +1260,7 @@ bool Model::run_layer(int li, int T, int max_kv, const int* d_pos, const int* d_
   if (!rc(k.pk_res32_offset_norm_add(mix.ptr, f32, L.norm1.d.ptr, (float*)x.ptr, xa.ptr, W, T, c.eps, f32, st), "norm1")) return false;
   // ---- feed-forward
   if (a.mlp_kind == 1) {
-    if (!gated_ff(L, T)) return false;
+    if (!gated_ff(L, T, act.ptr, a.ff)) return false;
     if (!lin(L.down, act.ptr, mix.ptr, T)) return false;
     if (!rc(k.pk_res32_offset_norm_add(mix.ptr, f32, L.norm2.d.ptr, (float*)x.ptr, xa.ptr, W, T, c.eps, f32, st), "norm2")) return false;
   } else if (a.mlp_kind == 2) {
@@ -1125,28 +1284,30 @@ bool Model::run_layer(int li, int T, int max_kv, const int* d_pos, const int* d_
   return true;
 }
 
-// dense gated feed-forward up to its hidden activations: act = f(W_gate xa) * (W_up xa), f SiLU or ReLU.  bf16: gate | up projection with the
+// dense gated feed-forward up to its hidden activations: out = f(W_gate xa) * (W_up xa), f SiLU, ReLU or GELU, rows of stride ld_out.  bf16: gate | up projection with the
 // activation in its epilogue (the library's fused GEMV for <= 4 tokens, its tensor-core GEMM above; the same rounding points as the two
 // launches they replace, which remain the fallback)
-bool Model::gated_ff(const Layer& L, int T) {
+bool Model::gated_ff(const Layer& L, int T, void* out, int ld_out) {
   const LayerCfg& a = L.c;
   bool fused = false;
   if (!c.f32 && T <= 4) {
     pk_b200_gemv_args g{};
     g.W = (const pk_bf16*)L.gate_up.d.ptr;
     g.X = (const pk_bf16*)xa.ptr;
-    g.Y[0] = (pk_bf16*)act.ptr;
+    g.Y[0] = (pk_bf16*)out;
     g.seg_rows[0] = a.ff;
     g.M = a.ff;
     g.N = T;
     g.K = c.width;
-    g.epi = a.mlp_act == 1 ? 5 : 1;
+    g.epi = a.mlp_act == 2 ? 6 : a.mlp_act == 1 ? 5 : 1;
+    g.y_ld = ld_out;
     fused = k.pk_b200_gemv_fused(&g, st) == 0;
   } else if (!c.f32) {
-    fused = k.pk_b200_gemm_gated((const pk_bf16*)L.gate_up.d.ptr, (const pk_bf16*)xa.ptr, (pk_bf16*)act.ptr, a.ff, T, c.width, a.mlp_act, st) == 0;
+    fused = k.pk_b200_gemm_gated_ex((const pk_bf16*)L.gate_up.d.ptr, (const pk_bf16*)xa.ptr, (pk_bf16*)out, a.ff, T, c.width, ld_out, a.mlp_act, st) == 0;
   }
   if (fused) return true;
-  return lin(L.gate_up, xa.ptr, gu.ptr, T) && rc(k.pk_act(gu.ptr, act.ptr, a.ff, T, a.mlp_act == 1 ? 2 : 0, c.f32, st), "gated activation");
+  const int kind = a.mlp_act == 2 ? 3 : a.mlp_act == 1 ? 2 : 0;
+  return lin(L.gate_up, xa.ptr, gu.ptr, T) && rc(k.pk_act_ex(gu.ptr, out, ld_out, a.ff, T, kind, c.f32, st), "gated activation");
 }
 
 // routed experts of one layer for the tokens in xa: router logits are in zs (block 1) or z (block 0); result in yf (fp32)
@@ -1336,7 +1497,7 @@ bool Model::run_sandwich_layer(int li, int T, int max_kv, const int* M) {
           "mixer result: gate, norm, residual"))
     return false;
   if (a.mlp_kind == 1) {
-    if (!gated_ff(L, T)) return false;
+    if (!gated_ff(L, T, act.ptr, a.ff)) return false;
     if (rg && !lin(L.rg2, xa.ptr, rgbuf.ptr, T)) return false;
     if (!lin(L.down, act.ptr, mix.ptr, T)) return false;
     if (!rc(k.pk_res32_gated_gnorm_add(mix.ptr, f32, nullptr, rg ? rgbuf.ptr : nullptr, W, rg ? L.rg2_bias.d.ptr : nullptr, L.norm2b.d.ptr, c.residual_mult,
@@ -1544,12 +1705,82 @@ bool Model::run_streams_layer(int li, int T, int max_kv, const int* M, int n) {
   if (!write_streams(0, "mixer result: streams, next norm")) return false;
   // ---- feed-forward
   if (a.mlp_kind == 1) {
-    if (!gated_ff(L, T) || !lin(L.down, act.ptr, mix.ptr, T)) return false;
+    if (!gated_ff(L, T, act.ptr, a.ff) || !lin(L.down, act.ptr, mix.ptr, T)) return false;
     if (!write_streams(1, "feed-forward result: streams, next norm")) return false;
   }
   if (keep_trail)
     return rc(k.pk_res32_streams_rows((const float*)x.ptr, nullptr, nullptr, nullptr, (float*)trail.ptr + (size_t)li * T * W, W, S, c.eps, T, f32, st), "trail");
   return true;
+}
+
+// Parallel block under one layer norm: on entry xa holds ln(x) of this layer; on exit mix holds the sum of both sublayers' results -- the caller
+// adds it to the residual together with the next norm.
+bool Model::run_lnorm_layer(int li, int T, int max_kv, const int* M, int n) {
+  Layer& L = layers[li];
+  const LayerCfg& a = L.c;
+  const LnormDims d(a);
+  const int f32 = c.f32, H = a.heads, G = a.kv_heads;
+  const int *d_pos = M + T, *d_req = M + 2 * T, *d_poff = M + 3 * T, *d_slot = M + 3 * T + n, *d_row0 = M + 3 * T + 2 * n, *d_len = M + 3 * T + 3 * n;
+  const int* d_pages = M + pages_at;
+  char* pool_base = (char*)cache.ptr + (size_t)L.cache_off * es;
+  const char* gate = (const char*)big.ptr + (size_t)d.gate_at() * es;
+  if (!lin(L.qkv, xa.ptr, big.ptr, T)) return false;
+  if (a.mixer_kind == 0) {
+    const int r = a.kv_rank, rd = a.rot_dim;
+    if (!rc(k.pk_latent_prep(big.ptr, d.big, 0, a.q_rank, L.dq_norm.d.ptr, cq.ptr, d.nq, L.dkv_norm.d.ptr, d_pos, d_req, d_poff, d_pages, pool_base, page_stride,
+                             c.page_size, r, rd, a.rot_dims, a.rot_interleaved, (const float*)L.freq.ptr, L.mag, c.eps, T, f32, st),
+            "latent norms + cache append"))
+      return false;
+    if (!lin(L.uq, cq.ptr, q.ptr, T)) return false;
+    if (!rc(k.pk_latent_query(q.ptr, L.uk_t.d.ptr, qa.ptr, d_pos, T, H, a.dim, r, rd, a.rot_dims, a.rot_interleaved, (const float*)L.freq.ptr, L.mag, f32, st),
+            "query fold + rotation"))
+      return false;
+    if (!rc(k.pk_latent_attention_ex(qa.ptr, pool_base, nullptr, d_pos, d_req, d_poff, d_pages, olat.ptr, page_stride, c.page_size, T, H, r, rd, a.scale,
+                                     a.window, max_kv, f32, st),
+            "latent attention"))
+      return false;
+    if (!rc(k.pk_gemm_strided_gated(olat.ptr, L.uv.d.ptr, ao.ptr, gate, T, a.vdim, r, (long)H * r, r, d.ld, H, r, (long)a.vdim * r, a.vdim, d.big, a.vdim, f32,
+                                    st),
+            "value expansion + output gate"))
+      return false;
+  } else if (a.mixer_kind == 1) {
+    pk_qk_prep prep{};
+    prep.norm_kind = a.qk_norm == 3 ? 1 : 0;
+    prep.eps = c.eps;
+    prep.q_only = a.kv_from >= 0;
+    if (!rc(k.pk_gqa_norm_append(big.ptr, d.big, d_pos, d_req, d_poff, d_pages, q.ptr, pool_base, page_stride, c.page_size, H, G, a.dim, a.vdim, a.rot_dims,
+                                 a.rot_interleaved, (const float*)L.freq.ptr, L.mag, &prep, T, f32, st),
+            "q / k norm + rotation + cache append"))
+      return false;
+    pk_attn_extra ex{};
+    ex.window = a.window;
+    ex.gate = d.ng ? gate : nullptr;
+    ex.gate_ld = d.big;
+    ex.gate_per_head = a.out_gate == 2;
+    ex.max_kv_len = max_kv;
+    ex.out_ld = d.ld;
+    if (!rc(k.pk_gqa_attention_ex(q.ptr, pool_base, a.sink_kind == 0 ? L.sink.d.ptr : nullptr, d_pos, d_req, d_poff, d_pages, ao.ptr, page_stride, c.page_size, T,
+                                  H, G, a.dim, a.vdim, a.scale, a.chunk, &ex, f32, st),
+            "attention"))
+      return false;
+  } else {
+    if (!rc(k.pk_gemm_strided_f32out((const char*)big.ptr + (size_t)d.decay_at() * es, L.a2.d.ptr, (float*)zc.ptr, T, H * a.dim, d.na, d.big, d.na,
+                                     (long)H * a.dim, 1, 0, 0, 0, f32, st),
+            "decay projection"))
+      return false;
+    const int ready = T >= kGroupedMinTokens;  // a prompt portion makes its decays once, a few tokens inside the recurrence
+    if (ready && !rc(k.pk_logistic_decay((float*)zc.ptr, (const float*)L.p1_32.ptr, a.tau, T, H * a.dim, st), "decays")) return false;
+    if (!rc(k.pk_gla_seq(big.ptr, d.big, 0, d.nq, d.nq + d.nk, (const float*)zc.ptr, H * a.dim, ready, (const float*)L.p1_32.ptr, a.tau,
+                         (float*)state.ptr + L.state_off, slot_stride, d_slot, d_row0, d_len, (float*)orec.ptr, H, a.dim, a.vdim, n, f32, st),
+            "gated linear attention"))
+      return false;
+    if (!rc(k.pk_head_norm_gate_ex((const float*)orec.ptr, nullptr, L.hnorm.d.ptr, 0, big.ptr, d.big, d.gate_at(), ao.ptr, d.ld, 1.f, T, H, a.vdim, c.eps, 0,
+                                   f32, st),
+            "read-out norm"))
+      return false;
+  }
+  if (d.ff && !gated_ff(L, T, (char*)ao.ptr + (size_t)d.wo * es, d.ld)) return false;
+  return lin(L.o, ao.ptr, mix.ptr, T);
 }
 
 // everything between the metadata upload and the final synchronisation: launches only (no allocation, no synchronisation)
@@ -1562,6 +1793,20 @@ bool Model::forward(int T, int n, int n_rows, int max_kv, int want_sample) {
     if (!rc(k.pk_res32_embed(embed.d.ptr, d_tok, (float*)x.ptr, xa.ptr, W, T, c.f32, st), "embedding")) return false;
     for (int li = 0; li < c.n_layers; ++li)
       if (!run_layer(li, T, max_kv, d_pos, d_req, d_poff, d_pages)) return false;
+  } else if (c.block_kind == 5) {
+    if (!rc(k.pk_res32_embed_lnorm(embed.d.ptr, d_tok, embed_norm.d.ptr, embed_norm_b.d.ptr, (float*)x.ptr, layers[0].norm1.d.ptr, layers[0].nb.d.ptr, xa.ptr, W,
+                                   c.eps, T, c.f32, st),
+            "embedding"))
+      return false;
+    for (int li = 0; li < c.n_layers; ++li) {
+      const Layer* next = li + 1 < c.n_layers ? &layers[li + 1] : nullptr;
+      if (!run_lnorm_layer(li, T, max_kv, M, n)) return false;
+      if (!rc(k.pk_res32_add_lnorm(mix.ptr, (float*)x.ptr, next ? next->norm1.d.ptr : nullptr, next ? next->nb.d.ptr : nullptr, xa.ptr, W, c.eps, T, c.f32, st),
+              "residual sum + norm"))
+        return false;
+      if (keep_trail && !cu(cudaMemcpyAsync((char*)trail.ptr + (size_t)li * T * W * 4, x.ptr, (size_t)T * W * 4, cudaMemcpyDeviceToDevice, st), "trail copy"))
+        return false;
+    }
   } else if (c.block_kind == 4) {
     if (!rc(k.pk_res32_streams_embed(embed.d.ptr, d_tok, (const float*)(c.streams > 0 ? layers[0].hc32[0][0].ptr : one32.ptr), (float*)x.ptr,
                                      layers[0].norm1.d.ptr, xa.ptr, (float*)h32.ptr, W, n_streams, c.eps, T, c.f32, st),
@@ -1601,6 +1846,8 @@ bool Model::forward(int T, int n, int n_rows, int max_kv, int want_sample) {
   if (n_rows > 0) {
     if (c.block_kind == 0) {
       if (!rc(k.pk_res32_offset_norm_rows((const float*)x.ptr, d_rows, final_norm.d.ptr, xr.ptr, W, n_rows, c.eps, c.f32, st), "final norm")) return false;
+    } else if (c.block_kind == 5) {
+      if (!rc(k.pk_res32_lnorm_rows((const float*)x.ptr, d_rows, final_norm.d.ptr, final_b.d.ptr, xr.ptr, W, c.eps, n_rows, c.f32, st), "final norm")) return false;
     } else if (c.block_kind == 4) {
       if (!rc(k.pk_res32_streams_rows((const float*)x.ptr, d_rows, final_norm.d.ptr, xr.ptr, nullptr, W, n_streams, c.eps, n_rows, c.f32, st), "final norm"))
         return false;

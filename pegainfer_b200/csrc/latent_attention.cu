@@ -88,6 +88,70 @@ __global__ void latent_kv_append_kernel(const E* __restrict__ dkv, const E* __re
   }
 }
 
+// The append for designs whose queries pass a latent too, with that latent's norm beside it.  rows [tokens, ld]: q latent at q_off, [kv latent |
+// shared rotated part] at kv_off.  grid (token, 2): one CTA norms the q latent into cq, the other appends to the cache.
+template <typename E>
+__global__ void latent_prep_kernel(const E* __restrict__ rows, int ld, int q_off, int q_rank, const E* __restrict__ q_norm_w, E* __restrict__ cq, int kv_off,
+                                   const E* __restrict__ kv_norm_w, const int* __restrict__ pos, const int* __restrict__ req,
+                                   const int* __restrict__ page_off, const int* __restrict__ pages, E* __restrict__ cache, long page_stride, int page_size,
+                                   int rank, int rot, int dims, int interleaved, const float* __restrict__ freq, float mag, float eps) {
+  __shared__ float red[33];
+  pdl_wait();
+  pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
+  const int t = blockIdx.x;
+  const bool kv = blockIdx.y == 1;
+  const E* d = rows + (size_t)t * ld + (kv ? kv_off : q_off);
+  const E* w = kv ? kv_norm_w : q_norm_w;
+  const int n = kv ? rank : q_rank, p = pos[t];
+  E* dst = kv ? cache + (size_t)pages[page_off[req[t]] + p / page_size] * page_stride + (size_t)(p % page_size) * (rank + rot) : cq + (size_t)t * q_rank;
+  float v[4], ss = 0.f;  // the first four entries of a thread stay in registers
+#pragma unroll
+  for (int u = 0; u < 4; ++u) {
+    const int i = threadIdx.x + u * blockDim.x;
+    v[u] = i < n ? to_f(d[i]) : 0.f;
+    ss = fmaf(v[u], v[u], ss);
+  }
+  for (int i = threadIdx.x + 4 * blockDim.x; i < n; i += blockDim.x) ss = fmaf(to_f(d[i]), to_f(d[i]), ss);
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)n + eps);
+#pragma unroll
+  for (int u = 0; u < 4; ++u) {
+    const int i = threadIdx.x + u * blockDim.x;
+    if (i < n) dst[i] = from_f<E>(v[u] * inv * to_f(w[i]));
+  }
+  for (int i = threadIdx.x + 4 * blockDim.x; i < n; i += blockDim.x) dst[i] = from_f<E>(to_f(d[i]) * inv * to_f(w[i]));
+  if (!kv) return;
+  for (int i = threadIdx.x; i < rot; i += blockDim.x) {
+    const float r = i < dims ? rotate_entry([&](int k) { return to_f(d[rank + k]); }, i, dims, interleaved, (float)p, freq, mag) : to_f(d[rank + i]);
+    dst[rank + i] = from_f<E>(r);
+  }
+}
+
+// A few tokens' queries in one launch: grid (token, head, slice); the last slice rotates the head's rotated part, the others fold slices of the
+// unrotated part onto the latent (qa[:rank] = q[:dim] W_uk, uk_t [heads][rank][dim]; every warp streams whole rows of uk_t).
+template <typename E>
+__global__ void latent_query_rows_kernel(const E* __restrict__ q, const E* __restrict__ uk_t, E* __restrict__ qa, const int* __restrict__ pos, int heads,
+                                         int dim, int rank, int rot, int dims, int interleaved, const float* __restrict__ freq, float mag) {
+  extern __shared__ __align__(16) float q_sm[];
+  pdl_wait();
+  pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
+  const int t = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  const E* src = q + ((size_t)t * heads + h) * (dim + rot);
+  E* dst = qa + ((size_t)t * heads + h) * (rank + rot);
+  if (blockIdx.z == gridDim.z - 1) {
+    for (int i = threadIdx.x; i < rot; i += blockDim.x) {
+      const float r = i < dims ? rotate_entry([&](int k) { return to_f(src[dim + k]); }, i, dims, interleaved, (float)pos[t], freq, mag) : to_f(src[dim + i]);
+      dst[rank + i] = from_f<E>(r);
+    }
+    return;
+  }
+  for (int k = threadIdx.x; k < dim; k += blockDim.x) q_sm[k] = to_f(src[k]);
+  __syncthreads();
+  for (int j = blockIdx.z * nw + warp; j < rank; j += (gridDim.z - 1) * nw) {
+    const float acc = warp_dot(uk_t + ((size_t)h * rank + j) * dim, q_sm, dim, lane);
+    if (lane == 0) dst[j] = from_f<E>(acc);
+  }
+}
+
 constexpr int kLatentMaxPerLane = 32;  // rank <= 1024
 
 // Generic-width kernel: one block per (query row, head); warps stride over the visible keys with an online softmax each,
@@ -240,4 +304,44 @@ extern "C" int pk_latent_attention_ex(const void* qa, const void* cache, const v
     launch(latent_attention_kernel<bf16>, dim3(tokens, heads), dim3(threads), smem, st, true, (const bf16*)qa, (const bf16*)cache, (const bf16*)sink,
            positions, req, page_off, pages, (bf16*)out, page_stride, page_size, heads, rank, rot, scale, window);
   return (int)cudaGetLastError();
+}
+
+extern "C" int pk_latent_prep(const void* rows, int ld, int q_off, int q_rank, const void* q_norm_w, void* cq, int kv_off, const void* kv_norm_w,
+                              const int* positions, const int* req, const int* page_off, const int* pages, void* cache, long page_stride, int page_size,
+                              int rank, int rot, int dims, int interleaved, const float* freq, float mag, float eps, int tokens, int f32, pk_stream st) {
+  if (!rows || !q_norm_w || !cq || !kv_norm_w || !positions || !req || !page_off || !pages || !cache || (dims > 0 && !freq) || tokens <= 0 || q_rank <= 0 ||
+      q_off < 0 || kv_off < 0 || ld < q_off + q_rank || ld < kv_off + rank + rot || rank <= 0 || rot < 0 || dims < 0 || dims > rot || (dims & 1) ||
+      page_size <= 0)
+    return -1;
+  const int widest = q_rank > rank ? q_rank : rank, threads = widest <= 256 ? 64 : widest <= 1024 || tokens > 64 ? 128 : 256;
+  const dim3 g(tokens, 2);
+  if (f32)
+    launch(latent_prep_kernel<float>, g, dim3(threads), 0, st, true, (const float*)rows, ld, q_off, q_rank, (const float*)q_norm_w, (float*)cq, kv_off,
+           (const float*)kv_norm_w, positions, req, page_off, pages, (float*)cache, page_stride, page_size, rank, rot, dims, interleaved, freq, mag, eps);
+  else
+    launch(latent_prep_kernel<bf16>, g, dim3(threads), 0, st, true, (const bf16*)rows, ld, q_off, q_rank, (const bf16*)q_norm_w, (bf16*)cq, kv_off,
+           (const bf16*)kv_norm_w, positions, req, page_off, pages, (bf16*)cache, page_stride, page_size, rank, rot, dims, interleaved, freq, mag, eps);
+  return (int)cudaGetLastError();
+}
+
+extern "C" int pk_latent_query(const void* q, const void* uk_t, void* qa, const int* positions, int tokens, int heads, int dim, int rank, int rot, int dims,
+                               int interleaved, const float* freq, float mag, int f32, pk_stream st) {
+  if (!q || !uk_t || !qa || !positions || (dims > 0 && !freq) || tokens <= 0 || heads <= 0 || dim <= 0 || rank <= 0 || rot < 0 || dims < 0 || dims > rot ||
+      (dims & 1))
+    return -1;
+  if (tokens <= 8 && dim <= 8192) {
+    const dim3 g(tokens, heads, (rank + 31) / 32 + 1);
+    const size_t sm = (size_t)dim * sizeof(float);
+    if (f32)
+      launch(latent_query_rows_kernel<float>, g, dim3(256), sm, st, true, (const float*)q, (const float*)uk_t, (float*)qa, positions, heads, dim, rank, rot,
+             dims, interleaved, freq, mag);
+    else
+      launch(latent_query_rows_kernel<bf16>, g, dim3(256), sm, st, true, (const bf16*)q, (const bf16*)uk_t, (bf16*)qa, positions, heads, dim, rank, rot, dims,
+             interleaved, freq, mag);
+    return (int)cudaGetLastError();
+  }
+  const int rc = pk_gemm_strided(q, uk_t, qa, nullptr, tokens, rank, dim, (long)heads * (dim + rot), 1, dim, (long)heads * (rank + rot), heads, dim + rot,
+                                 (long)dim * rank, rank + rot, 0, 0, f32, st);
+  if (rc != 0 || rot == 0) return rc;
+  return pk_rope_slice_ex(q, qa, positions, freq, mag, tokens, heads, dim + rot, dim, rank + rot, rank, rot, dims, interleaved, f32, st);
 }

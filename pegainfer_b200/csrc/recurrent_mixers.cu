@@ -2,6 +2,7 @@
 //   * short causal convolution (+ SiLU) over time per channel, with the last taps - 1 inputs of every request as state;
 //   * gated delta rule:   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q        (q, k unit vectors per head)
 //     with one decay g per head, or one per head and key channel (g then scales the rows of S);
+//   * gated linear attention:   S <- diag(a) S + k v^T;  o = S^T q     (one decay per head and key channel, a = logistic(.)^(1 / tau));
 //   * real-gated linear recurrent unit, one scalar per channel:  S <- a S + sqrt(1 - a^2) i u,  log a = -rate r softplus(lam),
 //     r and i logistic gates;  the read-out is multiplied by a GELU branch.  Affine maps compose, so a portion is scanned in parallel.
 //   * xLSTM matrix memory: m' = max(f + m, i);  S <- e^(f + m - m') S + e^(i - m') k v^T;  n likewise with k alone;
@@ -15,8 +16,8 @@
 // Step layout: entry e of the step owns rows [row0[e], row0[e] + len[e]) of every [tokens, features] buffer (a portion
 // of a prompt or one decoded token) and the state slot slot[e]; a slot's state is `state + slot * slot_stride` floats.
 // Sequence kernels: one CTA per (entry, head, slice of value columns); a column of S lives in the registers of DK / 16
-// neighbouring lanes (key size padded to the template's DK), tokens run one after the other.  The delta rule has a kernel of its
-// own, delta_seq_kernel; in recurrent_seq_kernel (matrix memory, state space) all threads first bring q, k, v and the gate inputs of a
+// neighbouring lanes (key size padded to the template's DK), tokens run one after the other.  The delta rule and the gated linear attention
+// have a kernel of their own, delta_seq_kernel; in recurrent_seq_kernel (matrix memory, state space) all threads first bring q, k, v and the gate inputs of a
 // block of 32 tokens into shared memory.  The matrix memory's normaliser n is one more column with value 1.  Latency-bound per token
 // (48 FMAs and two shuffle reductions per thread, one warp per scheduler).
 #include <algorithm>
@@ -107,6 +108,7 @@ struct SeqArgs {
   const float* zc;     // delta rule with a decay per key channel: [tokens, ld_zc], pre-activation of (head, channel) at h * dim + d; p1 = dt_bias [H * dim]
   int ld_zc;
   int zc_ready;        // 1: zc holds the decays themselves
+  float inv_tau;       // gated linear attention: decay = logistic(zc + p1)^inv_tau
 };
 
 // MODE 1: xLSTM matrix memory.  MODE 2: state-space duality (q = C, k = B, v = x; dim = state size).
@@ -276,12 +278,14 @@ __global__ void __launch_bounds__(160) recurrent_seq_kernel(SeqArgs a) {
   }
 }
 
-// ---- gated delta rule.  CTA = (entry, head, COLS value columns), warp-specialised: warps 0-3 run the recurrence, warps 4-7 prepare the next
+// ---- gated delta rule, gated linear attention.  CTA = (entry, head, COLS value columns), warp-specialised: warps 0-3 run the recurrence, warps 4-7 prepare the next
 // TB tokens meanwhile (unit vectors, gates, k . q) in the other of two shared-memory stages; one barrier per TB tokens.
 // Recurrence: KS = DK / 16 neighbouring lanes share one state column, 16 entries each as eight packed pairs (two-wide fp32 arithmetic), entry
 // (m * KS + ks) * 4 + e for m < 4, e < 4, so that the lanes' 16-byte shared-memory reads fall on consecutive banks.  Both products of a
 // token are taken on the decayed state before the write, o = S^T q = (g S)^T q + (k . q) u, so that their reductions over the lanes overlap and
-// only one of them is on the path to the next token.  CH: one decay per key channel (a third vector per token), else one per head.
+// only one of them is on the path to the next token.  FORM: delta rule with one decay per head (kHeadDecay) or per key channel
+// (kChannelDecay: a third vector per token); kLinear: gated linear attention, a decay per key channel and no correction of the value -- the write
+// waits for no reduction, q and k are used as projected.
 struct F2 {  // a packed pair of floats
   unsigned long long v;
 };
@@ -311,14 +315,17 @@ __device__ __forceinline__ float2 f2_unpack(F2 a) {
   return r;
 }
 
+constexpr int kHeadDecay = 0, kChannelDecay = 1, kLinear = 2;
+__device__ __forceinline__ float logistic_decay(float z, float inv_tau) { return expf(logsigmoidf_(z) * inv_tau); }
 constexpr int kDeltaTB = 16;  // tokens per stage
-template <int DK, bool CH>
+template <int DK, int FORM>
 constexpr int delta_stage_floats() {
-  return kDeltaTB * (2 * DK + 128 / (DK / 16) + (CH ? DK : 0) + 4);
+  return kDeltaTB * (2 * DK + 128 / (DK / 16) + (FORM != kHeadDecay ? DK : 0) + 4);
 }
 
-template <typename E, int DK, bool CH>
+template <typename E, int DK, int FORM>
 __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
+  constexpr bool CH = FORM != kHeadDecay, LIN = FORM == kLinear;
   constexpr int KS = DK / 16, COLS = 128 / KS, TB = kDeltaTB, NV = DK / 32, TW = TB / 4;  // TW: tokens a preparing warp handles per stage
   extern __shared__ __align__(16) float ds_sm[];
   pdl_wait();
@@ -326,13 +333,13 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
   const int e = blockIdx.x, h = blockIdx.y, kvh = h / (a.H / a.G), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int n = a.len[e], r0 = a.row0[e], dim = a.dim, vdim = a.vdim, col0 = blockIdx.z * COLS;
   const int n_stages = (n + TB - 1) / TB;
-  auto ks_of = [&](int b) { return ds_sm + (b & 1) * delta_stage_floats<DK, CH>(); };  // k [TB][DK] | q [TB][DK] | v [TB][COLS] | scalars [4][TB] | decays [TB][DK]
+  auto ks_of = [&](int b) { return ds_sm + (b & 1) * delta_stage_floats<DK, FORM>(); };  // k [TB][DK] | q [TB][DK] | v [TB][COLS] | scalars [4][TB] | decays [TB][DK]
   constexpr int QO = TB * DK, VO = 2 * TB * DK, SO = VO + TB * COLS, GO = SO + 4 * TB;
   if (warp >= 4) {
     // ---- preparation
     const E* X = static_cast<const E*>(a.qkv);
     const int qo = a.q_off + kvh * dim, ko = a.k_off + kvh * dim, vo = a.v_off + h * vdim + col0, pw = warp - 4, d0 = lane * NV;
-    const float qscale = 1.f / sqrtf((float)dim), rate = expf(a.p0[h]);
+    const float qscale = 1.f / sqrtf((float)dim), rate = LIN ? 0.f : expf(a.p0[h]);
     // Raw inputs of a stage wait in registers from one barrier to the next, so that their loads' latency is hidden: fetch() issues the loads
     // of a stage, finish() turns them into what the recurrence reads.
     constexpr int NW = sizeof(E) == 2 ? (NV + 1) / 2 : NV, VPT = TB * COLS / 128;  // 32-bit words per head row and lane; values per thread
@@ -384,7 +391,7 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
         const int at = pt + 128 * i, tt = min(at / COLS, nb - 1), c = at % COLS;
         vr[i] = col0 + c < vdim ? X[(size_t)(r0 + t0 + tt) * a.ld + vo + c] : from_f<E>(0.f);
       }
-      if (pw == 0 && lane < nb) {
+      if (!LIN && pw == 0 && lane < nb) {
         const float* z = a.z + (size_t)(r0 + t0 + lane) * a.ldz;
         if (!CH) za = z[a.za_off + h];
         zb = z[a.zb_off + h];
@@ -394,7 +401,7 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
       float* sm = ks_of(b);
       float qq[TW], kk[TW], kq[TW];
 #pragma unroll
-      for (int i = 0; i < TW; ++i) {
+      for (int i = 0; i < TW && !LIN; ++i) {
         qq[i] = kk[i] = kq[i] = 0.f;
 #pragma unroll
         for (int j = 0; j < NV; ++j) {
@@ -405,7 +412,7 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
         }
       }
 #pragma unroll
-      for (int o = 16; o > 0; o >>= 1)
+      for (int o = 16; o > 0 && !LIN; o >>= 1)
 #pragma unroll
         for (int i = 0; i < TW; ++i) {
           qq[i] += __shfl_xor_sync(0xffffffffu, qq[i], o);
@@ -415,8 +422,8 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
 #pragma unroll
       for (int i = 0; i < TW; ++i) {
         const int tt = pw + 4 * i;
-        const float qf = qscale / sqrtf(qq[i] + 1e-6f), kf = 1.f / sqrtf(kk[i] + 1e-6f);
-        if (lane == 0) sm[SO + 2 * TB + tt] = kq[i] * qf * kf;
+        const float qf = LIN ? qscale : qscale / sqrtf(qq[i] + 1e-6f), kf = LIN ? 1.f : 1.f / sqrtf(kk[i] + 1e-6f);
+        if (!LIN && lane == 0) sm[SO + 2 * TB + tt] = kq[i] * qf * kf;
         float kd[NV], qd[NV];
 #pragma unroll
         for (int j = 0; j < NV; ++j) {
@@ -429,7 +436,10 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
           for (int j = 0; j < NV; ++j) {
             gd[j] = gr[i][j];
             if (d0 + j >= dim) gd[j] = 1.f;
-            else if (!a.zc_ready) gd[j] = expf(-rate * softplusf_(gd[j] + a.p1[h * dim + d0 + j]));
+            else if (!a.zc_ready) {
+              const float z = gd[j] + a.p1[h * dim + d0 + j];
+              gd[j] = LIN ? logistic_decay(z, a.inv_tau) : expf(-rate * softplusf_(z));
+            }
           }
         }
         if constexpr (NV >= 4) {
@@ -450,7 +460,7 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
       }
 #pragma unroll
       for (int i = 0; i < VPT; ++i) sm[VO + pt + 128 * i] = to_f(vr[i]);
-      if (pw == 0 && lane < TB) {
+      if (!LIN && pw == 0 && lane < TB) {
         if (!CH) sm[SO + lane] = expf(-rate * softplusf_(za + a.p1[h]));
         sm[SO + TB + lane] = sigmoidf_(zb);
       }
@@ -488,7 +498,26 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
       const ulonglong2* kp = reinterpret_cast<const ulonglong2*>(sm + tt * DK) + ksi;
       const ulonglong2* qp = reinterpret_cast<const ulonglong2*>(sm + QO + tt * DK) + ksi;
       const ulonglong2* gp = reinterpret_cast<const ulonglong2*>(sm + GO + tt * DK) + ksi;
-      const float vt = sm[VO + tt * COLS + cl], beta = sm[SO + TB + tt], kq = sm[SO + 2 * TB + tt];
+      const float vt = sm[VO + tt * COLS + cl];
+      if constexpr (LIN) {
+        const F2 v2 = f2_pack(vt, vt);
+        F2 o0{0}, o1{0};
+#pragma unroll
+        for (int m = 0; m < 4; ++m) {
+          const ulonglong2 k2 = kp[m * KS], q2 = qp[m * KS], g2 = gp[m * KS];
+          S[2 * m] = f2_fma(F2{k2.x}, v2, f2_mul(S[2 * m], F2{g2.x}));
+          S[2 * m + 1] = f2_fma(F2{k2.y}, v2, f2_mul(S[2 * m + 1], F2{g2.y}));
+          o0 = f2_fma(S[2 * m], F2{q2.x}, o0);
+          o1 = f2_fma(S[2 * m + 1], F2{q2.y}, o1);
+        }
+        const float2 o2 = f2_unpack(f2_add(o0, o1));
+        float o = o2.x + o2.y;
+#pragma unroll
+        for (int s = 1; s < KS; s <<= 1) o += __shfl_xor_sync(0xffffffffu, o, s);
+        if (on && ksi == 0) out[(size_t)(b * TB + tt) * out_ld] = o;
+        continue;
+      }
+      const float beta = sm[SO + TB + tt], kq = sm[SO + 2 * TB + tt];
       const F2 g1 = CH ? F2{0} : f2_pack(sm[SO + tt], sm[SO + tt]);
       F2 kk[8], c0{0}, c1{0}, o0{0}, o1{0};
 #pragma unroll
@@ -534,28 +563,28 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
   }
 }
 
-template <typename E, int DK, bool CH>
+template <typename E, int DK, int FORM>
 static void launch_delta_t(const SeqArgs& a, int entries, cudaStream_t st) {
   constexpr int COLS = 128 / (DK / 16);
-  constexpr size_t need = 2 * delta_stage_floats<DK, CH>() * sizeof(float), apart = 116 * 1024;
+  constexpr size_t need = 2 * delta_stage_floats<DK, FORM>() * sizeof(float), apart = 116 * 1024;
   const dim3 g(entries, a.H, (a.vdim + COLS - 1) / COLS);
   // the chain of tokens sets the time, so two CTAs never share an SM while there is one for each: a programmatic launch would otherwise place
   // them wherever the previous kernel's CTAs have just left
   const size_t smem = (long)g.x * g.y * g.z <= sm_count() ? (need > apart ? need : apart) : need;
   static bool attr_set = false;  // per template instance
   if (!attr_set) {
-    cudaFuncSetAttribute(delta_seq_kernel<E, DK, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(need > apart ? need : apart));
+    cudaFuncSetAttribute(delta_seq_kernel<E, DK, FORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(need > apart ? need : apart));
     attr_set = true;
   }
-  launch(delta_seq_kernel<E, DK, CH>, g, dim3(256), smem, st, true, a);
+  launch(delta_seq_kernel<E, DK, FORM>, g, dim3(256), smem, st, true, a);
 }
-template <typename E, bool CH>
+template <typename E, int FORM>
 static int launch_delta(const SeqArgs& a, int entries, cudaStream_t st) {
   if (a.dim > 256) return -2;
-  if (a.dim <= 32) launch_delta_t<E, 32, CH>(a, entries, st);
-  else if (a.dim <= 64) launch_delta_t<E, 64, CH>(a, entries, st);
-  else if (a.dim <= 128) launch_delta_t<E, 128, CH>(a, entries, st);
-  else launch_delta_t<E, 256, CH>(a, entries, st);
+  if (a.dim <= 32) launch_delta_t<E, 32, FORM>(a, entries, st);
+  else if (a.dim <= 64) launch_delta_t<E, 64, FORM>(a, entries, st);
+  else if (a.dim <= 128) launch_delta_t<E, 128, FORM>(a, entries, st);
+  else launch_delta_t<E, 256, FORM>(a, entries, st);
   return (int)cudaGetLastError();
 }
 
@@ -567,6 +596,14 @@ __global__ void channel_decay_kernel(float* __restrict__ z, const float* __restr
     const int c = (int)(i % C);
     z[i] = expf(-expf(a_log[c / dim]) * softplusf_(z[i] + dt_bias[c]));
   }
+}
+
+// z <- logistic(z + bias)^inv_tau in place, C entries per token
+__global__ void logistic_decay_kernel(float* __restrict__ z, const float* __restrict__ bias, float inv_tau, long total, int C) {
+  pdl_wait();
+  pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
+  for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x)
+    z[i] = logistic_decay(z[i] + bias[i % C], inv_tau);
 }
 
 // out[t, h, j] = E( (o[t,h,j] / den[t,h]) / sqrt(mean_j(.^2) + eps) * w[h * w_stride + j] * act(gate[t, gate_off + h*vdim + j]) )
@@ -816,7 +853,7 @@ extern "C" int pk_gated_delta_seq(const void* qkv, int ld, int q_off, int k_off,
   if (!seq_args_ok(qkv, z, a_log, dt_bias, state, slot, row0, len, out, heads, kv_heads, dim, vdim, entries)) return -1;
   SeqArgs a{qkv, ld, q_off, k_off, v_off, z, ldz, decay_off, beta_off, a_log, dt_bias, state, slot_stride, slot, row0, len, out, nullptr,
             heads, kv_heads, dim, vdim, 0.f};
-  return f32 ? launch_delta<float, false>(a, entries, st) : launch_delta<bf16, false>(a, entries, st);
+  return f32 ? launch_delta<float, kHeadDecay>(a, entries, st) : launch_delta<bf16, kHeadDecay>(a, entries, st);
 }
 
 extern "C" int pk_channel_delta_seq(const void* qkv, int ld, int q_off, int k_off, int v_off, const float* z, int ldz, int beta_off, const float* decay,
@@ -826,7 +863,7 @@ extern "C" int pk_channel_delta_seq(const void* qkv, int ld, int q_off, int k_of
   if (!seq_args_ok(qkv, z, a_log, dt_bias, state, slot, row0, len, out, heads, kv_heads, dim, vdim, entries) || !decay || ld_decay < heads * dim) return -1;
   SeqArgs a{qkv, ld, q_off, k_off, v_off, z, ldz, 0, beta_off, a_log, dt_bias, state, slot_stride, slot, row0, len, out, nullptr,
             heads, kv_heads, dim, vdim, 0.f, nullptr, 0, 0, nullptr, decay, ld_decay, decay_ready};
-  return f32 ? launch_delta<float, true>(a, entries, st) : launch_delta<bf16, true>(a, entries, st);
+  return f32 ? launch_delta<float, kChannelDecay>(a, entries, st) : launch_delta<bf16, kChannelDecay>(a, entries, st);
 }
 
 extern "C" int pk_mlstm_seq(const void* qkv, int ld, int q_off, int k_off, int v_off, const float* z, int ldz, int forget_off, int input_off,
@@ -902,5 +939,23 @@ extern "C" int pk_channel_decay(float* z, const float* a_log, const float* dt_bi
   if (!z || !a_log || !dt_bias || tokens <= 0 || heads <= 0 || dim <= 0) return -1;
   const long total = (long)tokens * heads * dim;
   launch(channel_decay_kernel, dim3((unsigned)std::min<long>((total + 255) / 256, 148L * 8)), dim3(256), 0, st, true, z, a_log, dt_bias, total, heads * dim, dim);
+  return (int)cudaGetLastError();
+}
+
+extern "C" int pk_gla_seq(const void* qkv, int ld, int q_off, int k_off, int v_off, const float* decay, int ld_decay, int decay_ready, const float* bias,
+                          float tau, float* state, long slot_stride, const int* slot, const int* row0, const int* len, float* out, int heads, int dim,
+                          int vdim, int entries, int f32, pk_stream st) {
+  if (!qkv || !decay || !bias || !state || !slot || !row0 || !len || !out || heads <= 0 || dim <= 0 || vdim <= 0 || entries <= 0 ||
+      ld_decay < heads * dim || !(tau > 0.f))
+    return -1;
+  SeqArgs a{qkv, ld, q_off, k_off, v_off, nullptr, 0, 0, 0, nullptr, bias, state, slot_stride, slot, row0, len, out, nullptr,
+            heads, heads, dim, vdim, 0.f, nullptr, 0, 0, nullptr, decay, ld_decay, decay_ready, 1.f / tau};
+  return f32 ? launch_delta<float, kLinear>(a, entries, st) : launch_delta<bf16, kLinear>(a, entries, st);
+}
+
+extern "C" int pk_logistic_decay(float* z, const float* bias, float tau, int tokens, int channels, pk_stream st) {
+  if (!z || !bias || tokens <= 0 || channels <= 0 || !(tau > 0.f)) return -1;
+  const long total = (long)tokens * channels;
+  launch(logistic_decay_kernel, dim3((unsigned)std::min<long>((total + 255) / 256, 148L * 8)), dim3(256), 0, st, true, z, bias, 1.f / tau, total, channels);
   return (int)cudaGetLastError();
 }

@@ -80,9 +80,9 @@ __global__ void skinny_proj_kernel(const E* __restrict__ W, const float* __restr
 
 // kind 0: out[t][f] = silu(in[t][f]) * in[t][F + f]   (in is [T, 2F]: gate rows stacked over up rows)
 // kind 1: out[t][f] = relu(in[t][f])^2                (in is [T, F])
-// kind 2: out[t][f] = relu(in[t][f]) * in[t][F + f]   (in is [T, 2F])
+// kind 2: out[t][f] = relu(in[t][f]) * in[t][F + f]   (in is [T, 2F]);  kind 3: the same with gelu in its tanh form
 template <typename E>
-__global__ void act_kernel(const E* __restrict__ in, E* __restrict__ out, int F, long total, int kind) {
+__global__ void act_kernel(const E* __restrict__ in, E* __restrict__ out, int ld_out, int F, long total, int kind) {
   pdl_wait();
   pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
   for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x) {
@@ -90,12 +90,12 @@ __global__ void act_kernel(const E* __restrict__ in, E* __restrict__ out, int F,
     float r;
     if (kind != 1) {
       const float g = to_f(in[t * 2 * F + f]), u = to_f(in[t * 2 * F + F + f]);
-      r = (kind == 2 ? fmaxf(g, 0.f) : g / (1.f + expf(-g))) * u;
+      r = (kind == 2 ? fmaxf(g, 0.f) : kind == 3 ? gelu_tanh_gate(g) : g / (1.f + expf(-g))) * u;
     } else {
       const float u = fmaxf(to_f(in[i]), 0.f);
       r = u * u;
     }
-    out[i] = from_f<E>(r);
+    out[t * ld_out + f] = from_f<E>(r);
   }
 }
 
@@ -108,10 +108,11 @@ __global__ void convert_kernel(const A* __restrict__ in, B* __restrict__ out, lo
 
 // C[b][i][j] = (sum_k A[b*bsA + i*lda + k] * B[b*bsB + k*sbk + j*sbn]) * f(row_scale[i*ld_scale + b])
 // f = identity (scale_kind 1) or logistic (scale_kind 2); no scale when row_scale is null.  64 x 64 output tile, 256 threads, 4 x 4 each.
+// gate (may be null): the result is multiplied by logistic(gate[b * bs_gate + i * ld_gate + j]).
 template <typename E, typename O>
 __global__ void gemm_strided_kernel(const E* __restrict__ A, const E* __restrict__ B, O* __restrict__ C, const float* __restrict__ row_scale,
                                     int rows, int cols, int K, long lda, long sbk, long sbn, long ldc, long bsA, long bsB, long bsC,
-                                    int ld_scale, int scale_kind) {
+                                    int ld_scale, int scale_kind, const E* __restrict__ gate, long ld_gate, long bs_gate) {
   constexpr int TL = 64, KT = 16;
   __shared__ float as[KT][TL + 1], bs[KT][TL + 1];
   pdl_wait();
@@ -167,7 +168,9 @@ __global__ void gemm_strided_kernel(const E* __restrict__ A, const E* __restrict
 #pragma unroll
     for (int v = 0; v < 4; ++v) {
       const int j = j0 + tx * 4 + v;
-      if (j < cols) C[(size_t)i * ldc + j] = from_f<O>(acc[u][v] * s);
+      if (j >= cols) continue;
+      const float g = gate ? 1.f / (1.f + expf(-to_f(gate[(size_t)b * bs_gate + (size_t)i * ld_gate + j]))) : 1.f;
+      C[(size_t)i * ldc + j] = from_f<O>(acc[u][v] * s * g);
     }
   }
 }
@@ -176,7 +179,8 @@ __global__ void gemm_strided_kernel(const E* __restrict__ A, const E* __restrict
 // is staged as fp32 in shared memory and every warp streams whole B rows.
 template <typename E, typename O>
 __global__ void gemm_strided_rows_kernel(const E* __restrict__ A, const E* __restrict__ B, O* __restrict__ C, const float* __restrict__ row_scale,
-                                         int cols, int K, long lda, long sbn, long ldc, long bsA, long bsB, long bsC, int ld_scale, int scale_kind) {
+                                         int cols, int K, long lda, long sbn, long ldc, long bsA, long bsB, long bsC, int ld_scale, int scale_kind,
+                                         const E* __restrict__ gate, long ld_gate, long bs_gate) {
   extern __shared__ __align__(16) float a_s[];
   pdl_wait();
   pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
@@ -191,7 +195,10 @@ __global__ void gemm_strided_rows_kernel(const E* __restrict__ A, const E* __res
   }
   for (int j = blockIdx.z * nw + warp; j < cols; j += gridDim.z * nw) {
     const float acc = warp_dot(B + (size_t)b * bsB + (size_t)j * sbn, a_s, K, lane);
-    if (lane == 0) C[(size_t)b * bsC + (size_t)i * ldc + j] = from_f<O>(acc * s);
+    if (lane == 0) {
+      const float g = gate ? 1.f / (1.f + expf(-to_f(gate[(size_t)b * bs_gate + (size_t)i * ld_gate + j]))) : 1.f;
+      C[(size_t)b * bsC + (size_t)i * ldc + j] = from_f<O>(acc * s * g);
+    }
   }
 }
 
@@ -199,7 +206,8 @@ __global__ void gemm_strided_rows_kernel(const E* __restrict__ A, const E* __res
 int launch_gemm_batched_mma_f32(const bf16* A, const bf16* B, float* C, int rows, int cols, int K, long lda, long ldb, long ldc, int batch, long bsA,
                                 long bsB, long bsC, cudaStream_t st);
 int launch_gemm_batched_mma(const bf16* A, const bf16* B, bf16* C, const float* row_scale, int rows, int cols, int K, long lda, long ldb, long ldc,
-                            int batch, long bsA, long bsB, long bsC, int ld_scale, int scale_kind, cudaStream_t st);
+                            int batch, long bsA, long bsB, long bsC, int ld_scale, int scale_kind, const bf16* gate, long ld_gate, long bs_gate,
+                            cudaStream_t st);
 
 static inline int grid_1d(long n, int block) {
   long g = (n + block - 1) / block;
@@ -688,6 +696,118 @@ __global__ void streams_rows_kernel(const float* __restrict__ x, const int* __re
   for (int i = threadIdx.x; i < width; i += blockDim.x) out[(size_t)r * width + i] = from_f<E>(row[i] * inv * to_f(w[i]));
 }
 
+// ---- layer norm with weight and bias, the one norm of a block whose sublayers run side by side:
+//   x <- x + y (the sum of both sublayers' results);   h = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b
+// One CTA per token; the row lives in shared memory as fp32 and every thread meets the entries it wrote itself; the mean comes first, then
+// the squared deviations, both summed in a fixed order.
+
+// row[i] over this thread's entries and their sum -> the row's mean and reciprocal deviation
+template <int V>
+__device__ __forceinline__ float2 lnorm_stats(const float* row, float sum, int width, float eps, float* red) {
+  const float mean = block_sum2(sum, 0.f, red).x / (float)width;
+  float ss = 0.f;
+  for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+    float r[V];
+    ldv<V>(row + i, r);
+#pragma unroll
+    for (int k = 0; k < V; ++k) ss = fmaf(r[k] - mean, r[k] - mean, ss);
+  }
+  return make_float2(mean, 1.f / sqrtf(block_sum2(ss, 0.f, red).x / (float)width + eps));
+}
+template <int V, typename E>
+__device__ __forceinline__ void lnorm_apply(const float* row, float2 st, const E* __restrict__ w, const E* __restrict__ b, int i, float* r) {
+  float wv[V], bv[V];
+  ldv<V>(row + i, r);
+  ldv<V>(w + i, wv);
+  ldv<V>(b + i, bv);
+#pragma unroll
+  for (int k = 0; k < V; ++k) r[k] = fmaf((r[k] - st.x) * st.y, wv[k], bv[k]);
+}
+
+// y null: the row starts as ln_0(embed[ids[t]]) instead.  w null: no h (after the last layer).
+template <typename E, int V>
+__global__ void __launch_bounds__(512) lnorm_step_kernel(const E* __restrict__ y, const E* __restrict__ embed, const int* __restrict__ ids,
+                                                         const E* __restrict__ w0, const E* __restrict__ b0, float* __restrict__ x, const E* __restrict__ w,
+                                                         const E* __restrict__ b, E* __restrict__ h, int width, float eps) {
+  extern __shared__ __align__(16) float gn_sm[];
+  float* row = gn_sm;
+  float* red = row + width;  // 64 floats
+  pdl_wait();
+  pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
+  const int t = blockIdx.x;
+  float* xt = x + (size_t)t * width;
+  if (w)  // what the last phase reads, on its way while the sums are made
+    for (int i = threadIdx.x * 64; i < width; i += blockDim.x * 64) {
+      prefetch_l2(w + i);
+      prefetch_l2(b + i);
+    }
+  float sum = 0.f;
+  if (y) {
+    for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+      float r[V], yv[V];
+      ldv<V>(xt + i, r);
+      ldv<V>(y + (size_t)t * width + i, yv);
+#pragma unroll
+      for (int k = 0; k < V; ++k) {
+        r[k] += yv[k];
+        sum += r[k];
+      }
+      stv<V>(xt + i, r);
+      stv<V>(row + i, r);
+    }
+  } else {
+    const E* src = embed + (size_t)ids[t] * width;
+    float s0 = 0.f;
+    for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+      float r[V];
+      ldv<V>(src + i, r);
+#pragma unroll
+      for (int k = 0; k < V; ++k) s0 += r[k];
+      stv<V>(row + i, r);
+    }
+    const float2 st0 = lnorm_stats<V>(row, s0, width, eps, red);
+    for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+      float r[V];
+      lnorm_apply<V>(row, st0, w0, b0, i, r);
+#pragma unroll
+      for (int k = 0; k < V; ++k) sum += r[k];
+      stv<V>(xt + i, r);
+      stv<V>(row + i, r);
+    }
+  }
+  if (!w) return;
+  const float2 st = lnorm_stats<V>(row, sum, width, eps, red);
+  for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+    float r[V];
+    lnorm_apply<V>(row, st, w, b, i, r);
+    stv<V>(h + (size_t)t * width + i, r);
+  }
+}
+
+// out[r] = ln(x[rows[r]]) in the element type (rows null: every row)
+template <typename E>
+__global__ void lnorm_rows_kernel(const float* __restrict__ x, const int* __restrict__ rows, const E* __restrict__ w, const E* __restrict__ b,
+                                  E* __restrict__ out, int width, float eps) {
+  extern __shared__ __align__(16) float gn_sm[];
+  float* row = gn_sm;
+  float* red = row + width;
+  pdl_wait();
+  pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
+  const int r = blockIdx.x;
+  const float* xt = x + (size_t)(rows ? rows[r] : r) * width;
+  float sum = 0.f;
+  for (int i = threadIdx.x; i < width; i += blockDim.x) {
+    row[i] = xt[i];
+    sum += xt[i];
+  }
+  const float2 st = lnorm_stats<1>(row, sum, width, eps, red);
+  for (int i = threadIdx.x; i < width; i += blockDim.x) {
+    float v[1];
+    lnorm_apply<1>(row, st, w, b, i, v);
+    out[(size_t)r * width + i] = from_f<E>(v[0]);
+  }
+}
+
 // out = cap * tanh(float(in) * scale / cap)  (cap 0: float(in) * scale)
 template <typename A>
 __global__ void logits_scale_cap_kernel(const A* __restrict__ in, float* __restrict__ out, long n, float scale, float cap) {
@@ -748,6 +868,25 @@ static int launch_streams(const E* y, const E* embed, const int* ids, const floa
   return (int)cudaGetLastError();
 }
 
+template <typename E>
+static int launch_lnorm(const E* y, const E* embed, const int* ids, const E* w0, const E* b0, float* x, const E* w, const E* b, E* h, int width, float eps,
+                        int tokens, cudaStream_t st) {
+  const size_t sm = (size_t)(width + 64) * sizeof(float);
+  auto al = [](const void* p, int n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)) == 0; };
+  const int n = 4 * sizeof(E);
+  const bool vec = width % 4 == 0 && al(x, 16) && al(y, n) && al(embed, n) && al(w0, n) && al(b0, n) && al(w, n) && al(b, n) && al(h, n);
+  const int v = vec ? 4 : 1, thr = std::min(tokens > 64 ? 256 : 512, std::max(32, (width / v + 31) / 32 * 32));
+#define PK_LN(V)                                                                                                                               \
+  do {                                                                                                                                         \
+    if (!gnorm_fits(lnorm_step_kernel<E, V>, sm)) return -2;                                                                                   \
+    launch(lnorm_step_kernel<E, V>, dim3(tokens), dim3(thr), sm, st, true, y, embed, ids, w0, b0, x, w, b, h, width, eps);                     \
+  } while (0)
+  if (vec) PK_LN(4);
+  else PK_LN(1);
+#undef PK_LN
+  return (int)cudaGetLastError();
+}
+
 }  // namespace pk
 
 using namespace pk;
@@ -799,10 +938,14 @@ extern "C" int pk_res32_skinny_proj(const void* W, const float* x, float* out, i
 }
 
 extern "C" int pk_act(const void* in, void* out, int F, int tokens, int kind, int f32, pk_stream st) {
-  if (!in || !out || F <= 0 || tokens <= 0 || kind < 0 || kind > 2) return -1;
+  return pk_act_ex(in, out, F, F, tokens, kind, f32, st);
+}
+
+extern "C" int pk_act_ex(const void* in, void* out, int ld_out, int F, int tokens, int kind, int f32, pk_stream st) {
+  if (!in || !out || F <= 0 || ld_out < F || tokens <= 0 || kind < 0 || kind > 3) return -1;
   const long total = (long)F * tokens;
-  PK_BY_TYPE(f32, launch(act_kernel<float>, dim3(grid_1d(total, 256)), dim3(256), 0, st, true, (const float*)in, (float*)out, F, total, kind),
-             launch(act_kernel<bf16>, dim3(grid_1d(total, 256)), dim3(256), 0, st, true, (const bf16*)in, (bf16*)out, F, total, kind));
+  PK_BY_TYPE(f32, launch(act_kernel<float>, dim3(grid_1d(total, 256)), dim3(256), 0, st, true, (const float*)in, (float*)out, ld_out, F, total, kind),
+             launch(act_kernel<bf16>, dim3(grid_1d(total, 256)), dim3(256), 0, st, true, (const bf16*)in, (bf16*)out, ld_out, F, total, kind));
   return (int)cudaGetLastError();
 }
 
@@ -816,31 +959,43 @@ extern "C" int pk_convert(const void* in, int in_f32, void* out, int out_f32, lo
   return (int)cudaGetLastError();
 }
 
-extern "C" int pk_gemm_strided(const void* A, const void* B, void* C, const float* row_scale, int rows, int cols, int K, long lda, long sbk,
-                               long sbn, long ldc, int batch, long bsA, long bsB, long bsC, int ld_scale, int scale_kind, int f32, pk_stream st) {
+template <typename E>
+static int gemm_strided(const E* A, const E* B, E* C, const float* row_scale, int rows, int cols, int K, long lda, long sbk, long sbn, long ldc, int batch,
+                        long bsA, long bsB, long bsC, int ld_scale, int scale_kind, const E* gate, long ld_gate, long bs_gate, cudaStream_t st) {
   if (!A || !B || !C || rows <= 0 || cols <= 0 || K <= 0 || batch <= 0) return -1;
   if (rows <= 8 && sbk == 1 && K <= 8192) {
-    const dim3 gr(rows, batch, (cols + 31) / 32), br(256);
-    const size_t sm = (size_t)K * sizeof(float);
-    PK_BY_TYPE(f32,
-               launch(gemm_strided_rows_kernel<float, float>, gr, br, sm, st, true, (const float*)A, (const float*)B, (float*)C, row_scale, cols, K, lda, sbn,
-                      ldc, bsA, bsB, bsC, ld_scale, scale_kind),
-               launch(gemm_strided_rows_kernel<bf16, bf16>, gr, br, sm, st, true, (const bf16*)A, (const bf16*)B, (bf16*)C, row_scale, cols, K, lda, sbn, ldc,
-                      bsA, bsB, bsC, ld_scale, scale_kind));
+    launch(gemm_strided_rows_kernel<E, E>, dim3(rows, batch, (cols + 31) / 32), dim3(256), (size_t)K * sizeof(float), st, true, A, B, C, row_scale, cols, K,
+           lda, sbn, ldc, bsA, bsB, bsC, ld_scale, scale_kind, gate, ld_gate, bs_gate);
     return (int)cudaGetLastError();
   }
-  if (!f32 && sbk == 1 && rows >= 32) {  // many rows in bf16: the tensor-core kernel when the operands are laid out for it
-    const int rc = launch_gemm_batched_mma((const bf16*)A, (const bf16*)B, (bf16*)C, row_scale, rows, cols, K, lda, sbn, ldc, batch, bsA, bsB, bsC,
-                                           ld_scale, scale_kind, st);
-    if (rc != -2) return rc;
+  if constexpr (sizeof(E) == 2) {
+    if (sbk == 1 && rows >= 32) {  // many rows in bf16: the tensor-core kernel when the operands are laid out for it
+      const int rc = launch_gemm_batched_mma(A, B, C, row_scale, rows, cols, K, lda, sbn, ldc, batch, bsA, bsB, bsC, ld_scale, scale_kind, gate, ld_gate,
+                                             bs_gate, st);
+      if (rc != -2) return rc;
+    }
   }
-  const dim3 g((cols + 63) / 64, (rows + 63) / 64, batch), b(256);
-  PK_BY_TYPE(f32,
-             launch(gemm_strided_kernel<float, float>, g, b, 0, st, true, (const float*)A, (const float*)B, (float*)C, row_scale, rows, cols, K, lda, sbk,
-                    sbn, ldc, bsA, bsB, bsC, ld_scale, scale_kind),
-             launch(gemm_strided_kernel<bf16, bf16>, g, b, 0, st, true, (const bf16*)A, (const bf16*)B, (bf16*)C, row_scale, rows, cols, K, lda, sbk, sbn,
-                    ldc, bsA, bsB, bsC, ld_scale, scale_kind));
+  launch(gemm_strided_kernel<E, E>, dim3((cols + 63) / 64, (rows + 63) / 64, batch), dim3(256), 0, st, true, A, B, C, row_scale, rows, cols, K, lda, sbk, sbn,
+         ldc, bsA, bsB, bsC, ld_scale, scale_kind, gate, ld_gate, bs_gate);
   return (int)cudaGetLastError();
+}
+
+extern "C" int pk_gemm_strided(const void* A, const void* B, void* C, const float* row_scale, int rows, int cols, int K, long lda, long sbk,
+                               long sbn, long ldc, int batch, long bsA, long bsB, long bsC, int ld_scale, int scale_kind, int f32, pk_stream st) {
+  if (f32)
+    return gemm_strided<float>((const float*)A, (const float*)B, (float*)C, row_scale, rows, cols, K, lda, sbk, sbn, ldc, batch, bsA, bsB, bsC, ld_scale,
+                               scale_kind, nullptr, 0, 0, st);
+  return gemm_strided<bf16>((const bf16*)A, (const bf16*)B, (bf16*)C, row_scale, rows, cols, K, lda, sbk, sbn, ldc, batch, bsA, bsB, bsC, ld_scale, scale_kind,
+                            nullptr, 0, 0, st);
+}
+
+extern "C" int pk_gemm_strided_gated(const void* A, const void* B, void* C, const void* gate, int rows, int cols, int K, long lda, long ldb, long ldc,
+                                     int batch, long bsA, long bsB, long bsC, long ld_gate, long bs_gate, int f32, pk_stream st) {
+  if (f32)
+    return gemm_strided<float>((const float*)A, (const float*)B, (float*)C, nullptr, rows, cols, K, lda, 1, ldb, ldc, batch, bsA, bsB, bsC, 0, 0,
+                               (const float*)gate, ld_gate, bs_gate, st);
+  return gemm_strided<bf16>((const bf16*)A, (const bf16*)B, (bf16*)C, nullptr, rows, cols, K, lda, 1, ldb, ldc, batch, bsA, bsB, bsC, 0, 0, (const bf16*)gate,
+                            ld_gate, bs_gate, st);
 }
 
 extern "C" int pk_gemm_strided_f32out(const void* A, const void* B, float* C, int rows, int cols, int K, long lda, long ldb, long ldc, int batch, long bsA,
@@ -851,9 +1006,9 @@ extern "C" int pk_gemm_strided_f32out(const void* A, const void* B, float* C, in
     const size_t sm = (size_t)K * sizeof(float);
     PK_BY_TYPE(f32,
                launch(gemm_strided_rows_kernel<float, float>, gr, br, sm, st, true, (const float*)A, (const float*)B, C, (const float*)nullptr, cols, K, lda,
-                      ldb, ldc, bsA, bsB, bsC, 0, 0),
+                      ldb, ldc, bsA, bsB, bsC, 0, 0, (const float*)nullptr, 0L, 0L),
                launch(gemm_strided_rows_kernel<bf16, float>, gr, br, sm, st, true, (const bf16*)A, (const bf16*)B, C, (const float*)nullptr, cols, K, lda, ldb,
-                      ldc, bsA, bsB, bsC, 0, 0));
+                      ldc, bsA, bsB, bsC, 0, 0, (const bf16*)nullptr, 0L, 0L));
     return (int)cudaGetLastError();
   }
   if (!f32) {
@@ -863,9 +1018,9 @@ extern "C" int pk_gemm_strided_f32out(const void* A, const void* B, float* C, in
   const dim3 g((cols + 63) / 64, (rows + 63) / 64, batch), b(256);
   PK_BY_TYPE(f32,
              launch(gemm_strided_kernel<float, float>, g, b, 0, st, true, (const float*)A, (const float*)B, C, (const float*)nullptr, rows, cols, K, lda, 1L,
-                    ldb, ldc, bsA, bsB, bsC, 0, 0),
+                    ldb, ldc, bsA, bsB, bsC, 0, 0, (const float*)nullptr, 0L, 0L),
              launch(gemm_strided_kernel<bf16, float>, g, b, 0, st, true, (const bf16*)A, (const bf16*)B, C, (const float*)nullptr, rows, cols, K, lda, 1L, ldb,
-                    ldc, bsA, bsB, bsC, 0, 0));
+                    ldc, bsA, bsB, bsC, 0, 0, (const bf16*)nullptr, 0L, 0L));
   return (int)cudaGetLastError();
 }
 
@@ -1028,5 +1183,35 @@ extern "C" int pk_res32_streams_rows(const float* x, const int* rows, const void
   const dim3 g(n_rows), b(gnorm_threads(width, n_rows));
   PK_BY_TYPE(f32, launch(streams_rows_kernel<float>, g, b, sm, st, true, x, rows, (const float*)w, (float*)out, out32, width, streams, eps),
              launch(streams_rows_kernel<bf16>, g, b, sm, st, true, x, rows, (const bf16*)w, (bf16*)out, out32, width, streams, eps));
+  return (int)cudaGetLastError();
+}
+
+extern "C" int pk_res32_embed_lnorm(const void* embed, const int* token_ids, const void* w0, const void* b0, float* x, const void* w_next, const void* b_next,
+                                    void* h, int width, float eps, int tokens, int f32, pk_stream st) {
+  if (!embed || !token_ids || !w0 || !b0 || !x || (w_next && (!b_next || !h)) || width <= 0 || tokens <= 0) return -1;
+  if (f32)
+    return launch_lnorm<float>(nullptr, (const float*)embed, token_ids, (const float*)w0, (const float*)b0, x, (const float*)w_next, (const float*)b_next,
+                               (float*)h, width, eps, tokens, st);
+  return launch_lnorm<bf16>(nullptr, (const bf16*)embed, token_ids, (const bf16*)w0, (const bf16*)b0, x, (const bf16*)w_next, (const bf16*)b_next, (bf16*)h,
+                            width, eps, tokens, st);
+}
+
+extern "C" int pk_res32_add_lnorm(const void* y, float* x, const void* w_next, const void* b_next, void* h, int width, float eps, int tokens, int f32,
+                                  pk_stream st) {
+  if (!y || !x || (w_next && (!b_next || !h)) || width <= 0 || tokens <= 0) return -1;
+  if (f32)
+    return launch_lnorm<float>((const float*)y, nullptr, nullptr, nullptr, nullptr, x, (const float*)w_next, (const float*)b_next, (float*)h, width, eps, tokens,
+                               st);
+  return launch_lnorm<bf16>((const bf16*)y, nullptr, nullptr, nullptr, nullptr, x, (const bf16*)w_next, (const bf16*)b_next, (bf16*)h, width, eps, tokens, st);
+}
+
+extern "C" int pk_res32_lnorm_rows(const float* x, const int* rows, const void* w, const void* b, void* out, int width, float eps, int n_rows, int f32,
+                                   pk_stream st) {
+  if (!x || !w || !b || !out || width <= 0 || n_rows <= 0) return -1;
+  const size_t sm = (size_t)(width + 64) * sizeof(float);
+  if (!(f32 ? gnorm_fits(lnorm_rows_kernel<float>, sm) : gnorm_fits(lnorm_rows_kernel<bf16>, sm))) return -2;
+  const dim3 g(n_rows), bl(gnorm_threads(width, n_rows));
+  PK_BY_TYPE(f32, launch(lnorm_rows_kernel<float>, g, bl, sm, st, true, x, rows, (const float*)w, (const float*)b, (float*)out, width, eps),
+             launch(lnorm_rows_kernel<bf16>, g, bl, sm, st, true, x, rows, (const bf16*)w, (const bf16*)b, (bf16*)out, width, eps));
   return (int)cudaGetLastError();
 }

@@ -19,7 +19,7 @@ class GemvArgs(C.Structure):
     """pk_b200_gemv_args (include/pegainfer_kernels.h)."""
     _fields_ = [("W", vp), ("X", vp), ("Y", vp * 3), ("seg_rows", i32 * 3), ("M", i32), ("N", i32),
                 ("K", i32), ("x_mode", i32), ("residual", vp), ("norm_w", vp), ("eps", f32),
-                ("hidden_out", vp), ("normed_out", vp), ("epi", i32), ("tp_comm", vp), ("tp_step", vp), ("tp_op", i32)]
+                ("hidden_out", vp), ("normed_out", vp), ("epi", i32), ("tp_comm", vp), ("tp_step", vp), ("tp_op", i32), ("y_ld", i32)]
 
 
 class PrefetchSpan(C.Structure):
@@ -114,14 +114,14 @@ i64l = C.c_long
 class AttnExtra(C.Structure):
     """pk_attn_extra: options of pk_gqa_attention_ex (a zero / NULL field switches its option off)."""
     _fields_ = [("window", i32), ("softcap", f32), ("slope_log2", f32), ("gate", vp), ("gate_ld", i64l), ("max_kv_len", i32),
-                ("keep_first", i32)]
+                ("keep_first", i32), ("gate_per_head", i32), ("out_ld", i64l)]
 
 
 class QkPrep(C.Structure):
     """pk_qk_prep: what pk_gqa_norm_append does to q and k (norm per head or over the whole projection, the query's factor that grows with
     the logarithm of the position, keys cached in the place of values)."""
     _fields_ = [("norm_kind", i32), ("q_weight", vp), ("k_weight", vp), ("eps", f32), ("temp_coef", f32), ("temp_every", i32),
-                ("values_are_keys", i32)]
+                ("values_are_keys", i32), ("q_only", i32)]
 
 
 RES32_SIGNATURES = {
@@ -188,6 +188,17 @@ RES32_SIGNATURES = {
     "pk_head_norm_gate_ex": (i32, [vp, vp, vp, i32, vp, i32, i32, vp, i32, f32, i32, i32, i32, f32, i32, i32, vp]),
     "pk_gemm_strided_f32out": (i32, [vp, vp, vp] + [i32] * 3 + [i64l] * 3 + [i32] + [i64l] * 3 + [i32, vp]),
     "pk_b200_gemm_gated": (i32, [vp, vp, vp, i32, i32, i32, i32, vp]),
+    # parallel blocks under a layer norm, latent queries, gated linear attention
+    "pk_b200_gemm_gated_ex": (i32, [vp, vp, vp] + [i32] * 5 + [vp]),
+    "pk_res32_embed_lnorm": (i32, [vp] * 8 + [i32, f32, i32, i32, vp]),
+    "pk_res32_add_lnorm": (i32, [vp] * 5 + [i32, f32, i32, i32, vp]),
+    "pk_res32_lnorm_rows": (i32, [vp] * 5 + [i32, f32, i32, i32, vp]),
+    "pk_act_ex": (i32, [vp, vp] + [i32] * 5 + [vp]),
+    "pk_latent_prep": (i32, [vp, i32, i32, i32, vp, vp, i32] + [vp] * 6 + [i64l] + [i32] * 5 + [vp, f32, f32, i32, i32, vp]),
+    "pk_latent_query": (i32, [vp] * 4 + [i32] * 7 + [vp, f32, i32, vp]),
+    "pk_gemm_strided_gated": (i32, [vp] * 4 + [i32] * 3 + [i64l] * 3 + [i32] + [i64l] * 5 + [i32, vp]),
+    "pk_gla_seq": (i32, [vp, i32, i32, i32, i32, vp, i32, i32, vp, f32, vp, i64l, vp, vp, vp, vp] + [i32] * 5 + [vp]),
+    "pk_logistic_decay": (i32, [vp, vp, f32, i32, i32, vp]),
 }
 
 

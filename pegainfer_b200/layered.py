@@ -31,7 +31,7 @@ class LayerCfg(C.Structure):
                [(n, C.c_float) for n in ("act_limit", "act_slope", "shared_limit")] + [("weights_of", C.c_int)] + \
                [(n, C.c_int) for n in ("d_heads", "d_kv_heads", "d_dim", "d_vdim", "decay_rank", "gate_rank")] + \
                [("left_scale", C.c_float), ("right_scale", C.c_float), ("lru_width", C.c_int), ("lru_blocks", C.c_int), ("lru_rate", C.c_float),
-                ("mlp_act", C.c_int)]
+                ("mlp_act", C.c_int), ("q_rank", C.c_int), ("tau", C.c_float)]
 
 
 class ModelCfg(C.Structure):

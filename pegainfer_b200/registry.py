@@ -38,6 +38,11 @@ def _load_rilonex(path, dtype, max_tokens, max_requests, **kw):
     return RilonexModel.from_pretrained(path, dtype=dtype, max_tokens=max_tokens, max_requests=max_requests, **kw)
 
 
+def _load_vegodra(path, dtype, max_tokens, max_requests, **kw):
+    from .vegodra import VegodraModel
+    return VegodraModel.from_pretrained(path, dtype=dtype, max_tokens=max_tokens, max_requests=max_requests, **kw)
+
+
 def _load_qwen3(path, dtype, max_tokens, max_requests, **kw):
     from .config import PAGE_SIZE
     from .model import ModelRuntimeConfig, Qwen3Model
@@ -54,11 +59,12 @@ ARCHITECTURES = {
     "Nagosun": _load_nagosun,
     "Goguzen": _load_goguzen,
     "Rilonex": _load_rilonex,
+    "Vegodra": _load_vegodra,
     "Qwen3ForCausalLM": _load_qwen3,
     "qwen3": _load_qwen3,
 }
 # designs whose kernels run with every product in fp32 as well
-FLOAT32_CAPABLE = {"Vamadra", "Risolorn", "Nagosun", "Goguzen", "Rilonex"}
+FLOAT32_CAPABLE = {"Vamadra", "Risolorn", "Nagosun", "Goguzen", "Rilonex", "Vegodra"}
 
 
 def architecture_of(model_path: str) -> str:
