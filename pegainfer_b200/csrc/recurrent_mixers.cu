@@ -16,13 +16,14 @@
 // Step layout: entry e of the step owns rows [row0[e], row0[e] + len[e]) of every [tokens, features] buffer (a portion
 // of a prompt or one decoded token) and the state slot slot[e]; a slot's state is `state + slot * slot_stride` floats.
 // Sequence kernels: one CTA per (entry, head, slice of value columns); a column of S lives in the registers of DK / 16
-// neighbouring lanes (key size padded to the template's DK), tokens run one after the other.  The delta rule and the gated linear attention
-// have a kernel of their own, delta_seq_kernel; in recurrent_seq_kernel (matrix memory, state space) all threads first bring q, k, v and the gate inputs of a
+// neighbouring lanes (key size padded to the template's DK), tokens run one after the other.  The delta rule and the gated linear
+// attention have kernels of their own, delta_seq_kernel and gla_seq_kernel; in recurrent_seq_kernel (matrix memory, state space) all threads first bring q, k, v and the gate inputs of a
 // block of 32 tokens into shared memory.  The matrix memory's normaliser n is one more column with value 1.  Latency-bound per token
 // (48 FMAs and two shuffle reductions per thread, one warp per scheduler).
 #include <algorithm>
 
 #include "common.cuh"
+#include "mma.cuh"
 #include "typed.cuh"
 
 namespace pk {
@@ -108,7 +109,6 @@ struct SeqArgs {
   const float* zc;     // delta rule with a decay per key channel: [tokens, ld_zc], pre-activation of (head, channel) at h * dim + d; p1 = dt_bias [H * dim]
   int ld_zc;
   int zc_ready;        // 1: zc holds the decays themselves
-  float inv_tau;       // gated linear attention: decay = logistic(zc + p1)^inv_tau
 };
 
 // MODE 1: xLSTM matrix memory.  MODE 2: state-space duality (q = C, k = B, v = x; dim = state size).
@@ -278,14 +278,12 @@ __global__ void __launch_bounds__(160) recurrent_seq_kernel(SeqArgs a) {
   }
 }
 
-// ---- gated delta rule, gated linear attention.  CTA = (entry, head, COLS value columns), warp-specialised: warps 0-3 run the recurrence, warps 4-7 prepare the next
+// ---- gated delta rule.  CTA = (entry, head, COLS value columns), warp-specialised: warps 0-3 run the recurrence, warps 4-7 prepare the next
 // TB tokens meanwhile (unit vectors, gates, k . q) in the other of two shared-memory stages; one barrier per TB tokens.
 // Recurrence: KS = DK / 16 neighbouring lanes share one state column, 16 entries each as eight packed pairs (two-wide fp32 arithmetic), entry
 // (m * KS + ks) * 4 + e for m < 4, e < 4, so that the lanes' 16-byte shared-memory reads fall on consecutive banks.  Both products of a
 // token are taken on the decayed state before the write, o = S^T q = (g S)^T q + (k . q) u, so that their reductions over the lanes overlap and
-// only one of them is on the path to the next token.  FORM: delta rule with one decay per head (kHeadDecay) or per key channel
-// (kChannelDecay: a third vector per token); kLinear: gated linear attention, a decay per key channel and no correction of the value -- the write
-// waits for no reduction, q and k are used as projected.
+// only one of them is on the path to the next token.  CH: one decay per key channel (a third vector per token), else one per head.
 struct F2 {  // a packed pair of floats
   unsigned long long v;
 };
@@ -315,17 +313,14 @@ __device__ __forceinline__ float2 f2_unpack(F2 a) {
   return r;
 }
 
-constexpr int kHeadDecay = 0, kChannelDecay = 1, kLinear = 2;
-__device__ __forceinline__ float logistic_decay(float z, float inv_tau) { return expf(logsigmoidf_(z) * inv_tau); }
 constexpr int kDeltaTB = 16;  // tokens per stage
-template <int DK, int FORM>
+template <int DK, bool CH>
 constexpr int delta_stage_floats() {
-  return kDeltaTB * (2 * DK + 128 / (DK / 16) + (FORM != kHeadDecay ? DK : 0) + 4);
+  return kDeltaTB * (2 * DK + 128 / (DK / 16) + (CH ? DK : 0) + 4);
 }
 
-template <typename E, int DK, int FORM>
+template <typename E, int DK, bool CH>
 __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
-  constexpr bool CH = FORM != kHeadDecay, LIN = FORM == kLinear;
   constexpr int KS = DK / 16, COLS = 128 / KS, TB = kDeltaTB, NV = DK / 32, TW = TB / 4;  // TW: tokens a preparing warp handles per stage
   extern __shared__ __align__(16) float ds_sm[];
   pdl_wait();
@@ -333,13 +328,13 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
   const int e = blockIdx.x, h = blockIdx.y, kvh = h / (a.H / a.G), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int n = a.len[e], r0 = a.row0[e], dim = a.dim, vdim = a.vdim, col0 = blockIdx.z * COLS;
   const int n_stages = (n + TB - 1) / TB;
-  auto ks_of = [&](int b) { return ds_sm + (b & 1) * delta_stage_floats<DK, FORM>(); };  // k [TB][DK] | q [TB][DK] | v [TB][COLS] | scalars [4][TB] | decays [TB][DK]
+  auto ks_of = [&](int b) { return ds_sm + (b & 1) * delta_stage_floats<DK, CH>(); };  // k [TB][DK] | q [TB][DK] | v [TB][COLS] | scalars [4][TB] | decays [TB][DK]
   constexpr int QO = TB * DK, VO = 2 * TB * DK, SO = VO + TB * COLS, GO = SO + 4 * TB;
   if (warp >= 4) {
     // ---- preparation
     const E* X = static_cast<const E*>(a.qkv);
     const int qo = a.q_off + kvh * dim, ko = a.k_off + kvh * dim, vo = a.v_off + h * vdim + col0, pw = warp - 4, d0 = lane * NV;
-    const float qscale = 1.f / sqrtf((float)dim), rate = LIN ? 0.f : expf(a.p0[h]);
+    const float qscale = 1.f / sqrtf((float)dim), rate = expf(a.p0[h]);
     // Raw inputs of a stage wait in registers from one barrier to the next, so that their loads' latency is hidden: fetch() issues the loads
     // of a stage, finish() turns them into what the recurrence reads.
     constexpr int NW = sizeof(E) == 2 ? (NV + 1) / 2 : NV, VPT = TB * COLS / 128;  // 32-bit words per head row and lane; values per thread
@@ -391,7 +386,7 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
         const int at = pt + 128 * i, tt = min(at / COLS, nb - 1), c = at % COLS;
         vr[i] = col0 + c < vdim ? X[(size_t)(r0 + t0 + tt) * a.ld + vo + c] : from_f<E>(0.f);
       }
-      if (!LIN && pw == 0 && lane < nb) {
+      if (pw == 0 && lane < nb) {
         const float* z = a.z + (size_t)(r0 + t0 + lane) * a.ldz;
         if (!CH) za = z[a.za_off + h];
         zb = z[a.zb_off + h];
@@ -401,7 +396,7 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
       float* sm = ks_of(b);
       float qq[TW], kk[TW], kq[TW];
 #pragma unroll
-      for (int i = 0; i < TW && !LIN; ++i) {
+      for (int i = 0; i < TW; ++i) {
         qq[i] = kk[i] = kq[i] = 0.f;
 #pragma unroll
         for (int j = 0; j < NV; ++j) {
@@ -412,7 +407,7 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
         }
       }
 #pragma unroll
-      for (int o = 16; o > 0 && !LIN; o >>= 1)
+      for (int o = 16; o > 0; o >>= 1)
 #pragma unroll
         for (int i = 0; i < TW; ++i) {
           qq[i] += __shfl_xor_sync(0xffffffffu, qq[i], o);
@@ -422,8 +417,8 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
 #pragma unroll
       for (int i = 0; i < TW; ++i) {
         const int tt = pw + 4 * i;
-        const float qf = LIN ? qscale : qscale / sqrtf(qq[i] + 1e-6f), kf = LIN ? 1.f : 1.f / sqrtf(kk[i] + 1e-6f);
-        if (!LIN && lane == 0) sm[SO + 2 * TB + tt] = kq[i] * qf * kf;
+        const float qf = qscale / sqrtf(qq[i] + 1e-6f), kf = 1.f / sqrtf(kk[i] + 1e-6f);
+        if (lane == 0) sm[SO + 2 * TB + tt] = kq[i] * qf * kf;
         float kd[NV], qd[NV];
 #pragma unroll
         for (int j = 0; j < NV; ++j) {
@@ -436,10 +431,7 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
           for (int j = 0; j < NV; ++j) {
             gd[j] = gr[i][j];
             if (d0 + j >= dim) gd[j] = 1.f;
-            else if (!a.zc_ready) {
-              const float z = gd[j] + a.p1[h * dim + d0 + j];
-              gd[j] = LIN ? logistic_decay(z, a.inv_tau) : expf(-rate * softplusf_(z));
-            }
+            else if (!a.zc_ready) gd[j] = expf(-rate * softplusf_(gd[j] + a.p1[h * dim + d0 + j]));
           }
         }
         if constexpr (NV >= 4) {
@@ -460,7 +452,7 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
       }
 #pragma unroll
       for (int i = 0; i < VPT; ++i) sm[VO + pt + 128 * i] = to_f(vr[i]);
-      if (!LIN && pw == 0 && lane < TB) {
+      if (pw == 0 && lane < TB) {
         if (!CH) sm[SO + lane] = expf(-rate * softplusf_(za + a.p1[h]));
         sm[SO + TB + lane] = sigmoidf_(zb);
       }
@@ -498,26 +490,7 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
       const ulonglong2* kp = reinterpret_cast<const ulonglong2*>(sm + tt * DK) + ksi;
       const ulonglong2* qp = reinterpret_cast<const ulonglong2*>(sm + QO + tt * DK) + ksi;
       const ulonglong2* gp = reinterpret_cast<const ulonglong2*>(sm + GO + tt * DK) + ksi;
-      const float vt = sm[VO + tt * COLS + cl];
-      if constexpr (LIN) {
-        const F2 v2 = f2_pack(vt, vt);
-        F2 o0{0}, o1{0};
-#pragma unroll
-        for (int m = 0; m < 4; ++m) {
-          const ulonglong2 k2 = kp[m * KS], q2 = qp[m * KS], g2 = gp[m * KS];
-          S[2 * m] = f2_fma(F2{k2.x}, v2, f2_mul(S[2 * m], F2{g2.x}));
-          S[2 * m + 1] = f2_fma(F2{k2.y}, v2, f2_mul(S[2 * m + 1], F2{g2.y}));
-          o0 = f2_fma(S[2 * m], F2{q2.x}, o0);
-          o1 = f2_fma(S[2 * m + 1], F2{q2.y}, o1);
-        }
-        const float2 o2 = f2_unpack(f2_add(o0, o1));
-        float o = o2.x + o2.y;
-#pragma unroll
-        for (int s = 1; s < KS; s <<= 1) o += __shfl_xor_sync(0xffffffffu, o, s);
-        if (on && ksi == 0) out[(size_t)(b * TB + tt) * out_ld] = o;
-        continue;
-      }
-      const float beta = sm[SO + TB + tt], kq = sm[SO + 2 * TB + tt];
+      const float vt = sm[VO + tt * COLS + cl], beta = sm[SO + TB + tt], kq = sm[SO + 2 * TB + tt];
       const F2 g1 = CH ? F2{0} : f2_pack(sm[SO + tt], sm[SO + tt]);
       F2 kk[8], c0{0}, c1{0}, o0{0}, o1{0};
 #pragma unroll
@@ -563,29 +536,344 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(SeqArgs a) {
   }
 }
 
-template <typename E, int DK, int FORM>
+template <typename E, int DK, bool CH>
 static void launch_delta_t(const SeqArgs& a, int entries, cudaStream_t st) {
   constexpr int COLS = 128 / (DK / 16);
-  constexpr size_t need = 2 * delta_stage_floats<DK, FORM>() * sizeof(float), apart = 116 * 1024;
+  constexpr size_t need = 2 * delta_stage_floats<DK, CH>() * sizeof(float), apart = 116 * 1024;
   const dim3 g(entries, a.H, (a.vdim + COLS - 1) / COLS);
   // the chain of tokens sets the time, so two CTAs never share an SM while there is one for each: a programmatic launch would otherwise place
   // them wherever the previous kernel's CTAs have just left
   const size_t smem = (long)g.x * g.y * g.z <= sm_count() ? (need > apart ? need : apart) : need;
   static bool attr_set = false;  // per template instance
   if (!attr_set) {
-    cudaFuncSetAttribute(delta_seq_kernel<E, DK, FORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(need > apart ? need : apart));
+    cudaFuncSetAttribute(delta_seq_kernel<E, DK, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(need > apart ? need : apart));
     attr_set = true;
   }
-  launch(delta_seq_kernel<E, DK, FORM>, g, dim3(256), smem, st, true, a);
+  launch(delta_seq_kernel<E, DK, CH>, g, dim3(256), smem, st, true, a);
 }
-template <typename E, int FORM>
+template <typename E, bool CH>
 static int launch_delta(const SeqArgs& a, int entries, cudaStream_t st) {
   if (a.dim > 256) return -2;
-  if (a.dim <= 32) launch_delta_t<E, 32, FORM>(a, entries, st);
-  else if (a.dim <= 64) launch_delta_t<E, 64, FORM>(a, entries, st);
-  else if (a.dim <= 128) launch_delta_t<E, 128, FORM>(a, entries, st);
-  else launch_delta_t<E, 256, FORM>(a, entries, st);
+  if (a.dim <= 32) launch_delta_t<E, 32, CH>(a, entries, st);
+  else if (a.dim <= 64) launch_delta_t<E, 64, CH>(a, entries, st);
+  else if (a.dim <= 128) launch_delta_t<E, 128, CH>(a, entries, st);
+  else launch_delta_t<E, 256, CH>(a, entries, st);
   return (int)cudaGetLastError();
+}
+
+// ---- gated linear attention.  CTA = (entry, head, COLS value columns), warp-specialised: warps 0-3 run the recurrence over stages of TB tokens,
+// warps 4-7 keep kStages of them on their way into shared memory (as stored; cp.async where the rows are laid out for it) and add up read-outs.
+// Recurrence: KL = DK / RK neighbouring lanes share RC state columns, RK key entries of each (RK * RC = 16, packed pairs along the key axis), so
+// that every read of k, q and the decays from shared memory serves RC columns.  A read-out is a sum over those lanes that no later token waits
+// for: every thread leaves its share in shared memory, and warps 4-7 add the shares of a stage while the recurrence runs the next one.
+struct GlaArgs {
+  const void* qkv;     // [tokens, ld]: q at q_off + head * dim, k at k_off + head * dim, v at v_off + head * vdim
+  int ld, q_off, k_off, v_off;
+  const float* zc;     // [tokens, ld_zc]: pre-activation of the decay of (head, channel) at h * dim + d, or the decay itself (ready)
+  int ld_zc, ready;
+  const float* bias;   // [H * dim]
+  float inv_tau;
+  float* state;
+  long slot_stride;
+  const int *slot, *row0, *len;
+  float* out;          // [tokens, H * vdim]
+  int H, dim, vdim;
+};
+__device__ __forceinline__ float logistic_decay(float z, float inv_tau) { return expf(logsigmoidf_(z) * inv_tau); }
+
+template <typename E, int DK>
+struct GlaTile {
+  static constexpr int TB = 16, COLS = 128 / (DK / 16), RK = DK <= 128 ? 4 : 8, RC = 16 / RK, KL = DK / RK, kStages = sizeof(E) == 2 ? 4 : 3;
+  // bytes of a stage: k [TB][DK] | q [TB][DK] | v [TB][COLS] in the element type, decays [TB][DK] fp32
+  static constexpr int kQ = TB * DK * sizeof(E), kV = 2 * kQ, kG = kV + TB * COLS * sizeof(E), kStage = kG + TB * DK * 4;
+  static constexpr int kShares = TB * 128 * RC;  // floats of a stage's read-out shares: [TB][128 threads][RC]
+  static constexpr size_t kSmem = (size_t)kStages * kStage + 2 * kShares * sizeof(float);
+};
+// two packed pairs = four consecutive entries
+__device__ __forceinline__ void ld_pairs(const float* p, F2* o) {
+  const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(p);
+  o[0].v = v.x;
+  o[1].v = v.y;
+}
+__device__ __forceinline__ void ld_pairs(const bf16* p, F2* o) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  o[0] = f2_pack(bf16_lo(v.x), bf16_hi(v.x));
+  o[1] = f2_pack(bf16_lo(v.y), bf16_hi(v.y));
+}
+template <int N>
+__device__ __forceinline__ void ld_run(const float* p, float* o) {
+  if constexpr (N == 4) *reinterpret_cast<float4*>(o) = *reinterpret_cast<const float4*>(p);
+  else *reinterpret_cast<float2*>(o) = *reinterpret_cast<const float2*>(p);
+}
+template <int N>
+__device__ __forceinline__ void ld_run(const bf16* p, float* o) {
+  uint32_t u[N / 2];
+  if constexpr (N == 4) *reinterpret_cast<uint2*>(u) = *reinterpret_cast<const uint2*>(p);
+  else u[0] = *reinterpret_cast<const uint32_t*>(p);
+#pragma unroll
+  for (int i = 0; i < N / 2; ++i) {
+    o[2 * i] = bf16_lo(u[i]);
+    o[2 * i + 1] = bf16_hi(u[i]);
+  }
+}
+// GT tokens of the recurrence; their shares are stored after the last one, so that the loads of all of them may be under way together
+constexpr int kGlaGroup = 4;
+template <typename E, int DK, int GT>
+__device__ __forceinline__ void gla_tokens(F2 (&S)[GlaTile<E, DK>::RC][GlaTile<E, DK>::RK / 2], const unsigned char* sm, float* share, int t0, int ksl, int cl) {
+  typedef GlaTile<E, DK> L;
+  constexpr int RK = L::RK, RC = L::RC;
+  const E* ks = reinterpret_cast<const E*>(sm) + 4 * ksl;
+  const E* qs = reinterpret_cast<const E*>(sm + L::kQ) + 4 * ksl;
+  const E* vs = reinterpret_cast<const E*>(sm + L::kV) + cl;
+  const float* gs = reinterpret_cast<const float*>(sm + L::kG) + 4 * ksl;
+  float r[GT][RC];
+#pragma unroll
+  for (int t = 0; t < GT; ++t) {
+    const int tt = t0 + t;
+    F2 vc[RC];
+    float v[RC];
+    ld_run<RC>(vs + tt * L::COLS, v);
+#pragma unroll
+    for (int c = 0; c < RC; ++c) vc[c] = f2_pack(v[c], v[c]);
+    F2 o[RC];
+#pragma unroll
+    for (int m = 0; m < RK / 4; ++m) {
+      F2 k[2], q[2], g[2];
+      ld_pairs(ks + tt * DK + m * 4 * L::KL, k);
+      ld_pairs(qs + tt * DK + m * 4 * L::KL, q);
+      ld_pairs(gs + tt * DK + m * 4 * L::KL, g);
+#pragma unroll
+      for (int c = 0; c < RC; ++c) {
+        S[c][2 * m] = f2_fma(k[0], vc[c], f2_mul(S[c][2 * m], g[0]));
+        S[c][2 * m + 1] = f2_fma(k[1], vc[c], f2_mul(S[c][2 * m + 1], g[1]));
+        o[c] = f2_fma(S[c][2 * m + 1], q[1], m == 0 ? f2_mul(S[c][0], q[0]) : f2_fma(S[c][2 * m], q[0], o[c]));
+      }
+    }
+#pragma unroll
+    for (int c = 0; c < RC; ++c) {
+      const float2 p = f2_unpack(o[c]);
+      r[t][c] = p.x + p.y;
+    }
+  }
+#pragma unroll
+  for (int t = 0; t < GT; ++t) {
+    float* p = share + (t0 + t) * 128 * RC;
+    if constexpr (RC == 4) *reinterpret_cast<float4*>(p) = make_float4(r[t][0], r[t][1], r[t][2], r[t][3]);
+    else *reinterpret_cast<float2*>(p) = make_float2(r[t][0], r[t][1]);
+  }
+}
+// read-outs of the nb tokens of one stage, times `scale` (pt: 0 .. 127).  Item = (token, group of RC columns) with KL shares; P threads share an item
+// when there are fewer items than threads; every item starts at a share of its own, so that a quarter warp meets all banks.
+template <typename E, int DK>
+__device__ __forceinline__ void gla_read_out(const float* shares, int pt, int nb, float scale, float* out, size_t out_ld, int n_cols) {
+  typedef GlaTile<E, DK> L;
+  constexpr int RC = L::RC, KL = L::KL, GRP = 128 / KL, ITEMS = L::TB * GRP, P = ITEMS < 128 ? 128 / ITEMS : 1, N = KL / P;
+#pragma unroll
+  for (int it = pt / P; it < ITEMS; it += 128 / P) {
+    const int tt = it / GRP, g = it % GRP;
+    const float* p = shares + ((size_t)tt * 128 + g * KL + (pt % P) * N) * RC;
+    float s[RC];
+#pragma unroll
+    for (int c = 0; c < RC; ++c) s[c] = 0.f;
+    if (tt < nb) {
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        const float* x = p + ((i + it) % N) * RC;
+        if constexpr (RC == 4) {
+          const float4 v = *reinterpret_cast<const float4*>(x);
+          s[0] += v.x, s[1] += v.y, s[2] += v.z, s[3] += v.w;
+        } else {
+          const float2 v = *reinterpret_cast<const float2*>(x);
+          s[0] += v.x, s[1] += v.y;
+        }
+      }
+    }
+#pragma unroll
+    for (int c = 0; c < RC; ++c) {
+#pragma unroll
+      for (int d = 1; d < P; d <<= 1) s[c] += __shfl_xor_sync(0xffffffffu, s[c], d);
+      if (tt < nb && pt % P == 0 && g * RC + c < n_cols) out[(size_t)tt * out_ld + g * RC + c] = s[c] * scale;
+    }
+  }
+}
+
+template <typename E, int DK>
+__global__ void __launch_bounds__(256) gla_seq_kernel(GlaArgs a) {
+  typedef GlaTile<E, DK> L;
+  constexpr int TB = L::TB, COLS = L::COLS, RK = L::RK, RC = L::RC, KL = L::KL, NS = L::kStages;
+  extern __shared__ __align__(16) unsigned char gla_sm[];
+  float* const shares = reinterpret_cast<float*>(gla_sm + (size_t)NS * L::kStage);
+  const int e = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, dim = a.dim, vdim = a.vdim, col0 = blockIdx.z * COLS;
+  pdl_wait();
+  pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
+  const int n = a.len[e], r0 = a.row0[e], n_stages = (n + TB - 1) / TB;
+  const size_t out_ld = (size_t)a.H * vdim;
+  if (tid >= 128) {
+    const int pt = tid - 128;
+    const E* X = static_cast<const E*>(a.qkv) + (size_t)r0 * a.ld;
+    const float* Z = a.zc + (size_t)r0 * a.ld_zc + h * dim;
+    const int qo = a.q_off + h * dim, ko = a.k_off + h * dim, vo = a.v_off + h * vdim + col0;
+    constexpr int EP = 16 / sizeof(E), VP = COLS < EP ? COLS : EP;  // entries of a 16-byte piece; of a piece of v
+    // whole pieces of every row start on 16-byte boundaries (and heads end with a whole piece)
+    const bool rows_ok = ((a.ld | qo | ko | dim) % EP) == 0 && (reinterpret_cast<uintptr_t>(X) & 15) == 0;
+    const bool v_ok = ((a.ld | vo | vdim) % EP) == 0 && (reinterpret_cast<uintptr_t>(X) & 15) == 0 && COLS % EP == 0;
+    const bool z_ok = ((a.ld_zc | (h * dim) | dim) % 4) == 0 && (reinterpret_cast<uintptr_t>(Z) & 15) == 0;
+    auto load = [&](int b) {
+      unsigned char* st = gla_sm + (size_t)(b % NS) * L::kStage;
+      E* ks = reinterpret_cast<E*>(st);
+      E* qs = reinterpret_cast<E*>(st + L::kQ);
+      E* vs = reinterpret_cast<E*>(st + L::kV);
+      float* gs = reinterpret_cast<float*>(st + L::kG);
+      const int t0 = b * TB, nb = min(TB, n - t0);
+      if (rows_ok) {
+#pragma unroll
+        for (int i = pt; i < TB * (DK / EP); i += 128) {
+          const int tt = i / (DK / EP), d = (i % (DK / EP)) * EP;
+          if (tt < nb && d < dim) {
+            const E* row = X + (size_t)(t0 + tt) * a.ld;
+            cp_async16(ks + tt * DK + d, row + ko + d);
+            cp_async16(qs + tt * DK + d, row + qo + d);
+          }
+        }
+      } else {
+        for (int i = pt; i < nb * dim; i += 128) {
+          const int tt = i / dim, d = i % dim;
+          const E* row = X + (size_t)(t0 + tt) * a.ld;
+          ks[tt * DK + d] = row[ko + d];
+          qs[tt * DK + d] = row[qo + d];
+        }
+      }
+      if (v_ok) {
+#pragma unroll
+        for (int i = pt; i < TB * (COLS / VP); i += 128) {
+          const int tt = i / (COLS / VP), c = (i % (COLS / VP)) * VP;
+          if (tt < nb && col0 + c < vdim) cp_async16(vs + tt * COLS + c, X + (size_t)(t0 + tt) * a.ld + vo + c);
+        }
+      } else {
+        for (int i = pt; i < nb * COLS; i += 128) {
+          const int tt = i / COLS, c = i % COLS;
+          if (col0 + c < vdim) vs[tt * COLS + c] = X[(size_t)(t0 + tt) * a.ld + vo + c];
+        }
+      }
+      if (z_ok) {
+#pragma unroll
+        for (int i = pt; i < TB * (DK / 4); i += 128) {
+          const int tt = i / (DK / 4), d = (i % (DK / 4)) * 4;
+          if (tt < nb && d < dim) cp_async16(gs + tt * DK + d, Z + (size_t)(t0 + tt) * a.ld_zc + d);
+        }
+      } else {
+        for (int i = pt; i < nb * DK; i += 128) {
+          const int tt = i / DK, d = i % DK;
+          if (d < dim) gs[tt * DK + d] = Z[(size_t)(t0 + tt) * a.ld_zc + d];
+        }
+      }
+    };
+    // pre-activations -> decays in place: every thread turns the four-entry pieces that it brought itself
+    auto decays = [&](int b) {
+      float* gs = reinterpret_cast<float*>(gla_sm + (size_t)(b % NS) * L::kStage + L::kG);
+      const int nb = min(TB, n - b * TB);
+      if (z_ok) {
+        for (int i = pt; i < nb * (DK / 4); i += 128) {
+          const int tt = i / (DK / 4), d = (i % (DK / 4)) * 4;
+          if (d >= dim) continue;
+#pragma unroll
+          for (int u = 0; u < 4; ++u) gs[tt * DK + d + u] = logistic_decay(gs[tt * DK + d + u] + a.bias[h * dim + d + u], a.inv_tau);
+        }
+      } else {
+        for (int i = pt; i < nb * DK; i += 128) {
+          const int tt = i / DK, d = i % DK;
+          if (d < dim) gs[tt * DK + d] = logistic_decay(gs[tt * DK + d] + a.bias[h * dim + d], a.inv_tau);
+        }
+      }
+    };
+    const float qscale = 1.f / sqrtf((float)dim);
+    auto read_out = [&](int b) {
+      gla_read_out<E, DK>(shares + (b & 1) * L::kShares, pt, min(TB, n - b * TB), qscale, a.out + (size_t)(r0 + b * TB) * out_ld + h * vdim + col0, out_ld,
+                          vdim - col0);
+    };
+    if (dim < DK || col0 + COLS > vdim) {  // what no copy writes stays zero: padded key entries and columns contribute nothing
+      for (int i = pt * 16; i < NS * L::kStage; i += 128 * 16) *reinterpret_cast<uint4*>(gla_sm + i) = make_uint4(0, 0, 0, 0);
+      asm volatile("bar.sync 1, 128;" ::: "memory");
+    }
+#pragma unroll
+    for (int b = 0; b < NS - 1; ++b) {
+      if (b < n_stages) load(b);
+      cp_async_commit();
+    }
+    for (int b = 0; b < n_stages; ++b) {
+      asm volatile("cp.async.wait_group %0;" ::"n"(NS - 2) : "memory");
+      if (!a.ready) decays(b);
+      __syncthreads();  // stage b has landed; the recurrence is done with the stage before it, whose place the next load takes
+      if (b + NS - 1 < n_stages) load(b + NS - 1);
+      cp_async_commit();
+      if (b > 0) read_out(b - 1);
+    }
+    __syncthreads();  // the last stage's shares are complete
+    read_out(n_stages - 1);
+    return;
+  }
+  // ---- recurrence
+  const int ksl = tid % KL, cl = RC * (tid / KL), n_cols = vdim - col0 - cl;  // columns of this thread inside the head (may be none)
+  float* S_g = a.state + (size_t)a.slot[e] * a.slot_stride + (size_t)h * dim * vdim + col0 + cl;  // [dim][vdim]
+  auto key = [&](int j) { return ((j >> 1) * KL + ksl) * 4 + (j & 1) * 2; };                      // first key entry of pair j
+  F2 S[RC][RK / 2];
+#pragma unroll
+  for (int j = 0; j < RK / 2; ++j)
+#pragma unroll
+    for (int c = 0; c < RC; ++c) {
+      const int i = key(j);
+      S[c][j] = f2_pack(c < n_cols && i < dim ? S_g[(size_t)i * vdim + c] : 0.f, c < n_cols && i + 1 < dim ? S_g[(size_t)(i + 1) * vdim + c] : 0.f);
+    }
+  for (int b = 0; b < n_stages; ++b) {
+    __syncthreads();
+    const unsigned char* sm = gla_sm + (size_t)(b % NS) * L::kStage;
+    float* share = shares + (b & 1) * L::kShares + tid * RC;
+    const int nb = min(TB, n - b * TB);
+    int tt = 0;
+    for (; tt + kGlaGroup <= nb; tt += kGlaGroup) gla_tokens<E, DK, kGlaGroup>(S, sm, share, tt, ksl, cl);
+    for (; tt < nb; ++tt) gla_tokens<E, DK, 1>(S, sm, share, tt, ksl, cl);
+  }
+  __syncthreads();  // the last stage's shares are complete
+#pragma unroll
+  for (int j = 0; j < RK / 2; ++j)
+#pragma unroll
+    for (int c = 0; c < RC; ++c) {
+      const int i = key(j);
+      const float2 w = f2_unpack(S[c][j]);
+      if (c < n_cols && i < dim) S_g[(size_t)i * vdim + c] = w.x;
+      if (c < n_cols && i + 1 < dim) S_g[(size_t)(i + 1) * vdim + c] = w.y;
+    }
+}
+
+template <typename E, int DK>
+static void launch_gla_t(const GlaArgs& a, int entries, cudaStream_t st) {
+  constexpr size_t need = GlaTile<E, DK>::kSmem, apart = 116 * 1024, most = need > apart ? need : apart;
+  static_assert(most <= 227 * 1024, "stages exceed shared memory");
+  const dim3 g(entries, a.H, (a.vdim + GlaTile<E, DK>::COLS - 1) / GlaTile<E, DK>::COLS);
+  static bool attr_set = false;  // per template instance
+  if (!attr_set) {
+    cudaFuncSetAttribute(gla_seq_kernel<E, DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)most);
+    attr_set = true;
+  }
+  // as for the delta rule: two CTAs never share an SM while there is one for each
+  launch(gla_seq_kernel<E, DK>, g, dim3(256), (long)g.x * g.y * g.z <= sm_count() ? most : need, st, true, a);
+}
+template <typename E>
+static int launch_gla(const GlaArgs& a, int entries, cudaStream_t st) {
+  if (a.dim > 256) return -2;
+  if (a.dim <= 32) launch_gla_t<E, 32>(a, entries, st);
+  else if (a.dim <= 64) launch_gla_t<E, 64>(a, entries, st);
+  else if (a.dim <= 128) launch_gla_t<E, 128>(a, entries, st);
+  else launch_gla_t<E, 256>(a, entries, st);
+  return (int)cudaGetLastError();
+}
+
+// z <- logistic(z + bias)^inv_tau in place, C entries per token
+__global__ void logistic_decay_kernel(float* __restrict__ z, const float* __restrict__ bias, float inv_tau, long total, int C) {
+  pdl_wait();
+  pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
+  for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x)
+    z[i] = logistic_decay(z[i] + bias[i % C], inv_tau);
 }
 
 // z <- exp(-exp(a_log[head]) * softplus(z + dt_bias)) in place, C = heads * dim entries per token
@@ -596,14 +884,6 @@ __global__ void channel_decay_kernel(float* __restrict__ z, const float* __restr
     const int c = (int)(i % C);
     z[i] = expf(-expf(a_log[c / dim]) * softplusf_(z[i] + dt_bias[c]));
   }
-}
-
-// z <- logistic(z + bias)^inv_tau in place, C entries per token
-__global__ void logistic_decay_kernel(float* __restrict__ z, const float* __restrict__ bias, float inv_tau, long total, int C) {
-  pdl_wait();
-  pdl_launch_dependents();  // the next kernel may start its launch; it waits for this grid to finish before it reads
-  for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x)
-    z[i] = logistic_decay(z[i] + bias[i % C], inv_tau);
 }
 
 // out[t, h, j] = E( (o[t,h,j] / den[t,h]) / sqrt(mean_j(.^2) + eps) * w[h * w_stride + j] * act(gate[t, gate_off + h*vdim + j]) )
@@ -853,7 +1133,7 @@ extern "C" int pk_gated_delta_seq(const void* qkv, int ld, int q_off, int k_off,
   if (!seq_args_ok(qkv, z, a_log, dt_bias, state, slot, row0, len, out, heads, kv_heads, dim, vdim, entries)) return -1;
   SeqArgs a{qkv, ld, q_off, k_off, v_off, z, ldz, decay_off, beta_off, a_log, dt_bias, state, slot_stride, slot, row0, len, out, nullptr,
             heads, kv_heads, dim, vdim, 0.f};
-  return f32 ? launch_delta<float, kHeadDecay>(a, entries, st) : launch_delta<bf16, kHeadDecay>(a, entries, st);
+  return f32 ? launch_delta<float, false>(a, entries, st) : launch_delta<bf16, false>(a, entries, st);
 }
 
 extern "C" int pk_channel_delta_seq(const void* qkv, int ld, int q_off, int k_off, int v_off, const float* z, int ldz, int beta_off, const float* decay,
@@ -863,7 +1143,7 @@ extern "C" int pk_channel_delta_seq(const void* qkv, int ld, int q_off, int k_of
   if (!seq_args_ok(qkv, z, a_log, dt_bias, state, slot, row0, len, out, heads, kv_heads, dim, vdim, entries) || !decay || ld_decay < heads * dim) return -1;
   SeqArgs a{qkv, ld, q_off, k_off, v_off, z, ldz, 0, beta_off, a_log, dt_bias, state, slot_stride, slot, row0, len, out, nullptr,
             heads, kv_heads, dim, vdim, 0.f, nullptr, 0, 0, nullptr, decay, ld_decay, decay_ready};
-  return f32 ? launch_delta<float, kChannelDecay>(a, entries, st) : launch_delta<bf16, kChannelDecay>(a, entries, st);
+  return f32 ? launch_delta<float, true>(a, entries, st) : launch_delta<bf16, true>(a, entries, st);
 }
 
 extern "C" int pk_mlstm_seq(const void* qkv, int ld, int q_off, int k_off, int v_off, const float* z, int ldz, int forget_off, int input_off,
@@ -948,9 +1228,8 @@ extern "C" int pk_gla_seq(const void* qkv, int ld, int q_off, int k_off, int v_o
   if (!qkv || !decay || !bias || !state || !slot || !row0 || !len || !out || heads <= 0 || dim <= 0 || vdim <= 0 || entries <= 0 ||
       ld_decay < heads * dim || !(tau > 0.f))
     return -1;
-  SeqArgs a{qkv, ld, q_off, k_off, v_off, nullptr, 0, 0, 0, nullptr, bias, state, slot_stride, slot, row0, len, out, nullptr,
-            heads, heads, dim, vdim, 0.f, nullptr, 0, 0, nullptr, decay, ld_decay, decay_ready, 1.f / tau};
-  return f32 ? launch_delta<float, kLinear>(a, entries, st) : launch_delta<bf16, kLinear>(a, entries, st);
+  GlaArgs a{qkv, ld, q_off, k_off, v_off, decay, ld_decay, decay_ready, bias, 1.f / tau, state, slot_stride, slot, row0, len, out, heads, dim, vdim};
+  return f32 ? launch_gla<float>(a, entries, st) : launch_gla<bf16>(a, entries, st);
 }
 
 extern "C" int pk_logistic_decay(float* z, const float* bias, float tau, int tokens, int channels, pk_stream st) {
