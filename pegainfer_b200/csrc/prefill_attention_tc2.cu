@@ -64,7 +64,7 @@ __device__ __forceinline__ float ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-// {x0, x1} * s + c on the packed fp32 pipe (FFMA2, scalars broadcast)
+// {x0, x1} * s + c on the packed fp32 pipe (scalars broadcast)
 __device__ __forceinline__ void fma2(float& x0, float& x1, float s, float c) {
   unsigned long long v, sv, cv;
   asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(x0), "f"(x1));
@@ -73,7 +73,7 @@ __device__ __forceinline__ void fma2(float& x0, float& x1, float s, float c) {
   asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(v) : "l"(v), "l"(sv), "l"(cv));
   asm("mov.b64 {%0, %1}, %2;" : "=f"(x0), "=f"(x1) : "l"(v));
 }
-// acc0 += lo bf16 of pk, acc1 += hi bf16 of pk, exactly (fp32 accumulate of the ROUNDED values, FHADD.BF16: no unpack)
+// acc0 += lo bf16 of pk, acc1 += hi bf16 of pk, exactly (fp32 accumulate of the ROUNDED values: no unpack)
 __device__ __forceinline__ void add_bf16_pair(float& acc0, float& acc1, uint32_t pk) {
   asm("{\n\t.reg .b16 lo, hi;\n\tmov.b32 {lo, hi}, %2;\n\tadd.rn.f32.bf16 %0, lo, %0;\n\tadd.rn.f32.bf16 %1, hi, %1;\n\t}"
       : "+f"(acc0), "+f"(acc1)
@@ -453,7 +453,7 @@ prefill_attention_tc2_kernel(const __grid_constant__ CUtensorMap map_k, const __
         if (lane == 0) mbar_arrive(po_ready + i);
         continue;
       }
-      // ---- P = bf16(exp2(s * scale - ref)); the denominator sums the ROUNDED values (FHADD.BF16 straight off the pair) ----
+      // ---- P = bf16(exp2(s * scale - ref)); the denominator sums the ROUNDED values (straight off the pair) ----
       const float nref = -ref;
       float ds4[4] = {0.f, 0.f, 0.f, 0.f};
       auto p_pair = [&](uint32_t u0, uint32_t u1, int x) -> uint32_t {
